@@ -53,7 +53,7 @@ class SwiGluNames:
 class MoeNames:
     """Tensor names of a sparse block, after the spec's prefix; ``expert`` is a template over the expert's index."""
     router: str = "gate.weight"
-    shared_gate: str = "shared_expert_gate.weight"
+    shared_gate: Optional[str] = "shared_expert_gate.weight"
     shared: str = "shared_expert."
     expert: str = "experts.{e}."
     mlp: SwiGluNames = SwiGluNames()
@@ -104,7 +104,11 @@ class MoeFfnSpec:
     chosen among them returns its input (times its routing weight).  ``correction``: the name of a tensor with one
     number per router output that is added to the score for the choice only; the weights stay the scores.
     ``groups`` / ``keep_groups``: the router's outputs form that many equal groups of neighbours, a group's score is
-    its largest corrected score, and only experts of the best ``keep_groups`` groups can be chosen."""
+    its largest corrected score, and only experts of the best ``keep_groups`` groups can be chosen.
+    ``router_bias``: the name of a tensor with one number per router output that is added to the logits.
+    ``chosen_softmax``: the experts with the largest logits, their weights a softmax over the chosen logits alone.
+    ``glu`` / ``shared_glu``: (limit, alpha, shift) of gated units with clamped branches in place of SwiGLU, see
+    ``ClampedGluFfnSpec``.  ``names.shared_gate`` None: the shared expert is added without a gate."""
     hidden: int
     num_experts: int
     top_k: int
@@ -118,6 +122,10 @@ class MoeFfnSpec:
     correction: Optional[str] = None
     groups: int = 0
     keep_groups: int = 0
+    router_bias: Optional[str] = None
+    chosen_softmax: bool = False
+    glu: Optional[tuple] = None
+    shared_glu: Optional[tuple] = None
 
 
 @dataclass(frozen=True)
@@ -640,6 +648,62 @@ class SelectiveScanSpec:
     prefix: str
     kind: str = "selective_scan"
     names: SelectiveScanNames = SelectiveScanNames()
+
+
+@dataclass(frozen=True)
+class DifferentialAttentionNames:
+    q: str = "q"
+    k: str = "k"
+    v: str = "v"
+    o: str = "o"
+    q_norm: str = "q.norm"
+    k_norm: str = "k.norm"
+    head_gate: str = "g"
+    lambda_parts: tuple = ("lq1", "lk1", "lq2", "lk2")
+
+
+@dataclass(frozen=True)
+class DifferentialAttentionSpec:
+    """Softmax attention with two maps per head over the same values, the second taken off the first.  The query (key)
+    projection holds, head by head, ``key_dim`` channels for map one and as many for map two; queries and keys get an
+    RMS norm over the channels of a map (one weight vector for all heads and maps of a side), then the rotation
+    (``position``, split-half pairs) of the first channels of every map.  Scores are multiplied by ``scale`` as given and,
+    with ``softcap``, become softcap tanh(s / softcap).  Which keys a query sees: every earlier one, or (``chunk``) those
+    of its own block of ``chunk`` positions counted from the sequence's start.  Per head
+        o = a_1 - lambda a_2,  lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + diff  (one number for the layer),
+        o <- o / sqrt(mean(o^2) + eps) * (1 - diff)
+    and, with ``head_gate``, times the sigmoid of one number per token and head, a projection of the layer's input.
+    ``own_kv`` False: the layer has no keys and values and reads another layer's cache.  ``keep_window`` / ``keep_chunk``:
+    how far back the cache has to reach for every layer that reads it (both None: all the way)."""
+    hidden: int
+    num_heads: int
+    num_kv_heads: int
+    key_dim: int
+    value_dim: int
+    scale: float
+    softcap: Optional[float]
+    eps: float
+    diff: float
+    chunk: Optional[int]
+    position: Optional[ScaledRopeSpec]
+    own_kv: bool
+    keep_window: Optional[int]
+    keep_chunk: Optional[int]
+    prefix: str
+    head_gate: bool = True
+    kind: str = "attention_differential"
+    names: DifferentialAttentionNames = DifferentialAttentionNames()
+
+
+@dataclass(frozen=True)
+class OutputNormBlockSpec:
+    """x += norm(mixer(x)); x += norm(ffn(x)): the sublayers read the residual stream as it is and only their results
+    are normalised.  ``ffn`` None: the layer has a mixer only."""
+    mixer: Any
+    ffn: Any
+    mixer_post_norm: NormSpec
+    ffn_post_norm: Optional[NormSpec]
+    kind: str = "output_norm_residual"
 
 
 @dataclass(frozen=True)

@@ -11,6 +11,11 @@
 //
 // The query at position a sees key j iff j <= a and (window == 0 or a - j < window);
 // score = dot(q, k) / sqrt(hd).
+//
+// MAPS 2 is the differential form: every head has two attention maps over the same values, and a key head's row in the
+// cache holds the keys of both maps side by side.  A block's 16 rows are then up to eight heads times two maps; a
+// row's query is padded with zeros over the other map's channels, so both maps share the pages and the products of a
+// block, and the combine ends with the difference of the two, its norm and the head's gate (DiffParams).
 #include <cuda.h>
 
 #include "common.cuh"
@@ -84,20 +89,34 @@ __device__ __forceinline__ const bf16* tile_at(const bf16* tile, int r, int d) {
     return tile + (d >> 6) * (PAGE_KEYS * 64) + r * 64 + ((((d & 63) >> 3) ^ (r & 7)) << 3);
 }
 
-template <int HD>
+// The differential form's constants: scores s become softcap tanh(s / softcap) (0: as they are); per head
+// o = a_1 - lambda a_2, then o / sqrt(mean(o^2) + eps) * out_scale * sigmoid(gate[row * ldg + head]) (gate null: no gate).
+struct DiffParams {
+    int key_dim, value_dim;         // channels of one map's key, of a value; both multiples of 8
+    float softcap, lambda, eps, out_scale;
+    const float* gate;
+    long long ldg;
+};
+
+// cap * tanh(s / cap) by tanh(x) = 1 - 2 / (1 + e^(2x)): the absolute error is a few units of 2^-24 times cap
+__device__ __forceinline__ float softcap_score(float s, float cap) {
+    return cap - __fdividef(2.0f * cap, 1.0f + __expf(2.0f * s / cap));
+}
+
+template <int HDK, int HDV, int MAPS>
 __global__ void __launch_bounds__(THREADS)
 attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v,
                       const bf16* __restrict__ q, bf16* __restrict__ out, float* __restrict__ part_o, float* __restrict__ part_ml,
                       int* __restrict__ counters, const int* __restrict__ tok_seq, const int* __restrict__ tok_pos,
                       const int* __restrict__ seq_past, const int* __restrict__ block_table, int table_stride, int n_pages,
                       int page, int nh, int nkv, int window, int split_keys, int n_splits, float score_scale, int sink,
-                      const float* __restrict__ sink_vals, int chunk, int* __restrict__ status) {
+                      const float* __restrict__ sink_vals, int chunk, int* __restrict__ status, DiffParams df) {
     pdl_trigger();
-    constexpr int ITEM = PAGE_KEYS * HD;
-    constexpr int NBW = HD / 32;                   // 8-column blocks of the head that one warp accumulates
+    constexpr int ITEM_K = PAGE_KEYS * HDK, ITEM_V = PAGE_KEYS * HDV;
+    constexpr int NBW = HDV / 32;                   // 8-column blocks of the head that one warp accumulates
     constexpr int PLD = PAGE_KEYS + 8;             // row stride of the probabilities (bfloat16)
     extern __shared__ unsigned char dyn_raw[];
-    bf16* ring = reinterpret_cast<bf16*>((reinterpret_cast<uintptr_t>(dyn_raw) + 1023) & ~(uintptr_t)1023);   // [RING][ITEM]
+    bf16* ring = reinterpret_cast<bf16*>((reinterpret_cast<uintptr_t>(dyn_raw) + 1023) & ~(uintptr_t)1023);   // [ITEM_K + ITEM_V]: even items are keys, odd ones values
     __shared__ __align__(8) unsigned long long full_bar[RING];
     __shared__ float s_s[MMA_HEADS][PAGE_KEYS];
     __shared__ __align__(16) bf16 p_s[MMA_HEADS][PLD];
@@ -131,11 +150,17 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
         item_ok[slot] = ok ? 1 : 0;
         if (ok) {
             const int row0 = (pg * nkv + kvh) * PAGE_KEYS;       // the page's first row in the cache seen as [rows, HD]
-            mbar_expect_tx(&full_bar[slot], ITEM * 2);
+            if (item & 1) {
+                mbar_expect_tx(&full_bar[slot], ITEM_V * 2);
 #pragma unroll
-            for (int sub = 0; sub < HD / 64; sub++)
-                tma_load_2d(ring + (size_t)slot * ITEM + sub * (PAGE_KEYS * 64), (item & 1) ? &map_v : &map_k, sub * 64, row0,
-                            &full_bar[slot]);
+                for (int sub = 0; sub < HDV / 64; sub++)
+                    tma_load_2d(ring + ITEM_K + sub * (PAGE_KEYS * 64), &map_v, sub * 64, row0, &full_bar[slot]);
+            } else {
+                mbar_expect_tx(&full_bar[slot], ITEM_K * 2);
+#pragma unroll
+                for (int sub = 0; sub < HDK / 64; sub++)
+                    tma_load_2d(ring + sub * (PAGE_KEYS * 64), &map_k, sub * 64, row0, &full_bar[slot]);
+            }
         } else {
             mbar_arrive(&full_bar[slot]);
         }
@@ -151,12 +176,28 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
     }
     pdl_wait();
     // the query fragments of the block's heads (rows beyond ``heads`` are zero)
-    unsigned qa[HD / 16][4];
-    {
-        const bf16* q0 = q + ((size_t)n * nh + h0 + g8) * HD;
-        const bf16* q1 = q + ((size_t)n * nh + h0 + g8 + 8) * HD;
+    unsigned qa[HDK / 16][4];
+    if constexpr (MAPS == 2) {
+        // a row's channels lie where its map's keys lie in a key row (h0 is even: rows g8 and g8 + 8 belong to map g8 % 2)
+        const int kd = df.key_dim, off = (g8 & 1) * kd;
+        const bf16* q0 = q + ((size_t)n * nh + h0 + g8) * kd - off;
+        const bf16* q1 = q0 + (size_t)8 * kd;
+        auto piece = [&](const bf16* row, int c, bool live) {
+            return live && c >= off && c < off + kd ? *reinterpret_cast<const unsigned*>(row + c) : 0u;
+        };
 #pragma unroll
-        for (int kk = 0; kk < HD / 16; kk++) {
+        for (int kk = 0; kk < HDK / 16; kk++) {
+            const int c = kk * 16 + tg * 2;
+            qa[kk][0] = piece(q0, c, g8 < heads);
+            qa[kk][1] = piece(q1, c, g8 + 8 < heads);
+            qa[kk][2] = piece(q0, c + 8, g8 < heads);
+            qa[kk][3] = piece(q1, c + 8, g8 + 8 < heads);
+        }
+    } else {
+        const bf16* q0 = q + ((size_t)n * nh + h0 + g8) * HDK;
+        const bf16* q1 = q + ((size_t)n * nh + h0 + g8 + 8) * HDK;
+#pragma unroll
+        for (int kk = 0; kk < HDK / 16; kk++) {
             const int c = kk * 16 + tg * 2;
             qa[kk][0] = g8 < heads ? *reinterpret_cast<const unsigned*>(q0 + c) : 0u;
             qa[kk][1] = g8 + 8 < heads ? *reinterpret_cast<const unsigned*>(q1 + c) : 0u;
@@ -169,7 +210,7 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
         for (; issued < min(RING, n_items); issued++) issue(issued);
     }
 
-    const float root = sqrtf((float)HD);
+    const float root = sqrtf((float)HDK);
     float o[NBW][4];
 #pragma unroll
     for (int i = 0; i < NBW; i++)
@@ -181,7 +222,7 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
         const int key0 = (first_page + pi) * PAGE_KEYS;
         const int item_k = 2 * pi, slot_k = item_k % RING;
         if (__syncthreads_or(!mbar_wait(&full_bar[slot_k], (item_k / RING) & 1))) { failed = true; break; }
-        const bf16* kp = ring + (size_t)slot_k * ITEM;
+        const bf16* kp = ring;
         const bool page_ok = item_ok[slot_k] != 0;
         // ---- scores of keys 16*warp .. 16*warp+15 for all heads
         float sc[2][4];
@@ -190,7 +231,7 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
 #pragma unroll
             for (int j = 0; j < 4; j++) sc[i][j] = 0.f;
 #pragma unroll
-        for (int kk = 0; kk < HD / 16; kk++) {
+        for (int kk = 0; kk < HDK / 16; kk++) {
             unsigned kf[4];
             ldsm_x4(kf, tile_at(kp, warp * 16 + (lane & 7) + (lane >> 4) * 8, kk * 16 + ((lane >> 3) & 1) * 8));
             mma_16816(sc[0], qa[kk], kf[0], kf[1]);
@@ -202,7 +243,9 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
             for (int j = 0; j < 4; j++) {
                 const int t = warp * 16 + nb * 8 + tg * 2 + (j & 1), key = key0 + t;
                 const bool live = page_ok && key >= j0 && key <= j1;
-                if (g8 + (j >> 1) * 8 < heads) s_s[g8 + (j >> 1) * 8][t] = live ? (score_scale > 0.f ? sc[nb][j] * score_scale : sc[nb][j] / root) : -INFINITY;
+                float sv = score_scale > 0.f ? sc[nb][j] * score_scale : sc[nb][j] / root;
+                if (MAPS == 2 && df.softcap > 0.f) sv = softcap_score(sv, df.softcap);
+                if (g8 + (j >> 1) * 8 < heads) s_s[g8 + (j >> 1) * 8][t] = live ? sv : -INFINITY;
             }
         __syncthreads();                           // scores are written; the key buffer is free
         if (tid == 0 && issued < n_items) issue(issued++);
@@ -226,7 +269,7 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
         // ---- weighted values: this warp's quarter of the columns
         const int item_v = 2 * pi + 1, slot_v = item_v % RING;
         if (__syncthreads_or(!mbar_wait(&full_bar[slot_v], (item_v / RING) & 1))) { failed = true; break; }
-        const bf16* vp = ring + (size_t)slot_v * ITEM;
+        const bf16* vp = ring + ITEM_K;
         const float sc_lo = scale_s[g8], sc_hi = scale_s[g8 + 8];
 #pragma unroll
         for (int i = 0; i < NBW; i++) {
@@ -244,7 +287,7 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
                 for (int nb2 = 0; nb2 < NBW / 2; nb2++) {
                     unsigned vf[4];
                     ldsm_x4_trans(vf, tile_at(vp, kt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8,
-                                              warp * (HD / 4) + nb2 * 16 + (lane >> 4) * 8));
+                                              warp * (HDV / 4) + nb2 * 16 + (lane >> 4) * 8));
                     mma_16816(o[2 * nb2], pf, vf[0], vf[1]);
                     mma_16816(o[2 * nb2 + 1], pf, vf[2], vf[3]);
                 }
@@ -274,14 +317,14 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
     // ---- partial results: rows g8 and g8+8, this warp's columns
 #pragma unroll
     for (int i = 0; i < NBW; i++) {
-        const int d = warp * (HD / 4) + i * 8 + tg * 2;
+        const int d = warp * (HDV / 4) + i * 8 + tg * 2;
         if (g8 < heads) {
-            float* po = part_o + (((size_t)n * nh + h0 + g8) * n_splits + split) * HD + d;
+            float* po = part_o + (((size_t)n * nh + h0 + g8) * n_splits + split) * HDV + d;
             po[0] = o[i][0];
             po[1] = o[i][1];
         }
         if (g8 + 8 < heads) {
-            float* po = part_o + (((size_t)n * nh + h0 + g8 + 8) * n_splits + split) * HD + d;
+            float* po = part_o + (((size_t)n * nh + h0 + g8 + 8) * n_splits + split) * HDV + d;
             po[0] = o[i][2];
             po[1] = o[i][3];
         }
@@ -307,13 +350,14 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
     // The row's splits: a warp takes a head at a time.  The weight exp(m - max) and the sum of every split are worked
     // out once, a lane each, into the page buffers (free by now); then each lane adds up its columns over the splits
     // in ascending order, several loads in flight, so a result does not depend on how the work is shared out.
-    constexpr int WCH = RING * ITEM * (int)sizeof(bf16) / ((THREADS / 32) * 2 * (int)sizeof(float));   // splits a pass
-    constexpr int NV = HD / 64;                             // pairs of columns per lane: 64 j + 2 lane, + 1
+    constexpr int WCH = (ITEM_K + ITEM_V) * (int)sizeof(bf16) / ((THREADS / 32) * 2 * (int)sizeof(float));   // splits a pass
+    constexpr int NV = HDV / 64;                            // pairs of columns per lane: 64 j + 2 lane, + 1
     float* w_w = reinterpret_cast<float*>(ring) + (size_t)warp * 2 * WCH;
     float* l_w = w_w + WCH;
-    for (int g = warp; g < heads; g += THREADS / 32) {
+    // row ``g`` of the block, normalised: this lane's columns into ``res``
+    auto combine_row = [&](int g, float (&res)[NV][2]) {
         const float* ml = part_ml + ((size_t)n * nh + h0 + g) * n_splits * 2;
-        const float* po = part_o + ((size_t)n * nh + h0 + g) * n_splits * HD;
+        const float* po = part_o + ((size_t)n * nh + h0 + g) * n_splits * HDV;
         float mx = -INFINITY;
         for (int sp = s0 + lane; sp <= s1; sp += 32) mx = fmaxf(mx, __ldcg(ml + 2 * sp));
 #pragma unroll
@@ -333,25 +377,61 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
                 l_w[i] = __ldcg(ml + 2 * (c0 + i) + 1);
             }
             __syncwarp();
-            const float* pc = po + (size_t)c0 * HD + lane * 2;
+            const float* pc = po + (size_t)c0 * HDV + lane * 2;
 #pragma unroll 8
             for (int i = 0; i < cn; i++) {
                 const float w = w_w[i];
                 denom += l_w[i] * w;
 #pragma unroll
                 for (int j = 0; j < NV; j++) {
-                    const float2 v = __ldcg(reinterpret_cast<const float2*>(pc + (size_t)i * HD + j * 64));
+                    const float2 v = __ldcg(reinterpret_cast<const float2*>(pc + (size_t)i * HDV + j * 64));
                     num[j][0] += v.x * w;
                     num[j][1] += v.y * w;
                 }
             }
         }
-        bf16* orow = out + ((size_t)n * nh + h0 + g) * HD + lane * 2;
 #pragma unroll
-        for (int j = 0; j < NV; j++)
-            *reinterpret_cast<__nv_bfloat162*>(orow + j * 64) =
-                __nv_bfloat162(__float2bfloat16_rn(denom > 0.f ? num[j][0] / denom : 0.f),
-                               __float2bfloat16_rn(denom > 0.f ? num[j][1] / denom : 0.f));
+        for (int j = 0; j < NV; j++) {
+            res[j][0] = denom > 0.f ? num[j][0] / denom : 0.f;
+            res[j][1] = denom > 0.f ? num[j][1] / denom : 0.f;
+        }
+    };
+    if constexpr (MAPS == 2) {
+        // a warp takes a head: both maps' rows, their difference, its norm over the value channels (those beyond
+        // value_dim are zero) and the gate
+        for (int u = warp; 2 * u < heads; u += THREADS / 32) {
+            float o1[NV][2], o2[NV][2], ss = 0.f;
+            combine_row(2 * u, o1);
+            combine_row(2 * u + 1, o2);
+#pragma unroll
+            for (int j = 0; j < NV; j++)
+#pragma unroll
+                for (int e = 0; e < 2; e++) {
+                    o1[j][e] -= df.lambda * o2[j][e];
+                    ss = fmaf(o1[j][e], o1[j][e], ss);
+                }
+            ss = warp_sum(ss);
+            const int head = h0 / 2 + u;
+            float f = df.out_scale / sqrtf(ss / (float)df.value_dim + df.eps);
+            if (df.gate) f *= 1.0f / (1.0f + expf(-df.gate[(size_t)n * df.ldg + head]));
+            bf16* orow = out + ((size_t)n * (nh / 2) + head) * df.value_dim;
+#pragma unroll
+            for (int j = 0; j < NV; j++) {
+                const int d = j * 64 + lane * 2;
+                if (d < df.value_dim)
+                    *reinterpret_cast<__nv_bfloat162*>(orow + d) = __floats2bfloat162_rn(o1[j][0] * f, o1[j][1] * f);
+            }
+        }
+    } else {
+        for (int g = warp; g < heads; g += THREADS / 32) {
+            float res[NV][2];
+            combine_row(g, res);
+            bf16* orow = out + ((size_t)n * nh + h0 + g) * HDV + lane * 2;
+    #pragma unroll
+            for (int j = 0; j < NV; j++)
+                *reinterpret_cast<__nv_bfloat162*>(orow + j * 64) =
+                    __nv_bfloat162(__float2bfloat16_rn(res[j][0]), __float2bfloat16_rn(res[j][1]));
+        }
     }
 }
 
@@ -380,32 +460,33 @@ int make_cache_map(CUtensorMap* map, const void* base, unsigned long long rows, 
     return r == CUDA_SUCCESS ? 0 : (int)cudaErrorInvalidValue;
 }
 
-template <int HD>
+template <int HDK, int HDV, int MAPS>
 int launch_split_mma(int split, const bf16* q, const bf16* k, const bf16* v, bf16* out, float* po, float* pml, int* counters,
                      const int* tok_seq, const int* tok_pos, const int* seq_past, const int* table, int stride, int n_pages, int page,
                      int n_tokens, int nh, int nkv, int window, int n_splits, float score_scale, int sink,
                      const float* sink_vals, int chunk, int* status,
-                     cudaStream_t stream) {
+                     cudaStream_t stream, const DiffParams& df = DiffParams{}) {
     CUtensorMap map_k, map_v;
     const unsigned long long rows = (unsigned long long)n_pages * nkv * PAGE_KEYS;
-    int rc = make_cache_map(&map_k, k, rows, HD);
+    // heads narrower than the kernel's tiles are read with zeros behind them
+    int rc = make_cache_map(&map_k, k, rows, MAPS == 2 ? 2 * df.key_dim : HDK);
     if (rc) return rc;
-    rc = make_cache_map(&map_v, v, rows, HD);
+    rc = make_cache_map(&map_v, v, rows, MAPS == 2 ? df.value_dim : HDV);
     if (rc) return rc;
-    const size_t dyn = (size_t)RING * PAGE_KEYS * HD * sizeof(bf16) + 1024;
+    const size_t dyn = (size_t)PAGE_KEYS * (HDK + HDV) * sizeof(bf16) + 1024;
     static bool raised[64] = {false};              // per device: the attribute belongs to the device's context
     int device = 0;
     if (cudaGetDevice(&device) != cudaSuccess || device < 0 || device >= 64) return (int)cudaErrorInvalidDevice;
     if (!raised[device]) {
-        cudaError_t e = cudaFuncSetAttribute(attn_split_mma_kernel<HD>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)dyn);
+        cudaError_t e = cudaFuncSetAttribute(attn_split_mma_kernel<HDK, HDV, MAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)dyn);
         if (e != cudaSuccess) return (int)e;
         raised[device] = true;
     }
     const int group = nh / nkv;
     dim3 grid(n_tokens, nkv * ((group + MMA_HEADS - 1) / MMA_HEADS), n_splits);
-    esp_launch_pdl(ESP_PDL_ATTENTION, attn_split_mma_kernel<HD>, dim3(grid), dim3(THREADS), dyn, stream, map_k, map_v, q, out, po, pml,
+    esp_launch_pdl(ESP_PDL_ATTENTION, attn_split_mma_kernel<HDK, HDV, MAPS>, dim3(grid), dim3(THREADS), dyn, stream, map_k, map_v, q, out, po, pml,
                    counters, tok_seq, tok_pos, seq_past, table, stride, n_pages, page, nh, nkv, window, split, n_splits, score_scale,
-                   sink, sink_vals, chunk, status);
+                   sink, sink_vals, chunk, status, df);
     return esp_launch_status();
 }
 }  // namespace
@@ -427,7 +508,7 @@ ESP_API int esp_attn_decode(const void* q, const void* k_cache, const void* v_ca
     if (nkv <= 0 || nh % nkv != 0 || n_splits <= 0 || n_splits > 65535 || nh > 65535 || split < PAGE_KEYS || split % PAGE_KEYS != 0 ||
         page != PAGE_KEYS)
         return (int)cudaErrorInvalidValue;
-#define ESP_HD(HD) return launch_split_mma<HD>(split, (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache, (bf16*)out, part_o, \
+#define ESP_HD(HD) return launch_split_mma<HD, HD, 1>(split, (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache, (bf16*)out, part_o, \
                                                part_ml, counters, tok_seq, tok_pos, seq_past, block_table, table_stride, n_pages, \
                                                page, n_tokens, nh, nkv, window, n_splits, score_scale, sink, sink_vals, chunk, status, stream)
     switch (hd) {
@@ -438,6 +519,40 @@ ESP_API int esp_attn_decode(const void* q, const void* k_cache, const void* v_ca
     }
 #undef ESP_HD
     return (int)cudaErrorInvalidValue;
+}
+
+// The differential form (see the top of the file).  q [n_tokens, heads, 2, key_dim]; keys [pages, nkv, 64, 2 * key_dim]
+// (a row: the keys of map one, then of map two), values [pages, nkv, 64, value_dim]; out [n_tokens, heads, value_dim].
+// key_dim and value_dim: multiples of 8, at most 128 and 256.  Scratch: part_o float [n_tokens, 2 * heads, n_splits,
+// value_dim rounded up to 64, 128 or 256], part_ml float [n_tokens, 2 * heads, n_splits, 2]; the rest as above.
+ESP_API int esp_attn_decode_diff(const void* q, const void* k_cache, const void* v_cache, void* out, float* part_o,
+                                 float* part_ml, int* counters, const int* tok_seq, const int* tok_pos, const int* seq_past,
+                                 const int* block_table, int table_stride, int n_pages, int page, int n_tokens, int heads,
+                                 int nkv, int key_dim, int value_dim, int window, int split, int n_splits, float score_scale,
+                                 int chunk, float softcap, float lambda, float eps, float out_scale, const float* gate,
+                                 long long ldg, int* status, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (nkv <= 0 || heads % nkv != 0 || n_splits <= 0 || n_splits > 65535 || heads > 32767 || split < PAGE_KEYS ||
+        split % PAGE_KEYS != 0 || page != PAGE_KEYS || key_dim <= 0 || key_dim % 8 != 0 || key_dim > 128 || value_dim <= 0 ||
+        value_dim % 8 != 0 || value_dim > 256 || !(score_scale > 0.f))
+        return (int)cudaErrorInvalidValue;
+    const DiffParams df{key_dim, value_dim, softcap, lambda, eps, out_scale, gate, ldg};
+#define ESP_DIFF(HDK, HDV)                                                                                                  \
+    return launch_split_mma<HDK, HDV, 2>(split, (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache, (bf16*)out, part_o, \
+                                         part_ml, counters, tok_seq, tok_pos, seq_past, block_table, table_stride, n_pages, page, \
+                                         n_tokens, 2 * heads, nkv, window, n_splits, score_scale, 0, nullptr, chunk, status,     \
+                                         stream, df)
+#define ESP_DIFF_V(HDK)                          \
+    do {                                         \
+        if (value_dim <= 64) ESP_DIFF(HDK, 64);   \
+        if (value_dim <= 128) ESP_DIFF(HDK, 128); \
+        ESP_DIFF(HDK, 256);                       \
+    } while (0)
+    if (key_dim <= 32) ESP_DIFF_V(64);
+    if (key_dim <= 64) ESP_DIFF_V(128);
+    ESP_DIFF_V(256);
+#undef ESP_DIFF_V
+#undef ESP_DIFF
 }
 
 // ---------------------------------------------------------------------------------------------------

@@ -6,7 +6,10 @@
 // a - j < window), or, with ``chunk`` > 0, iff j <= a and both lie in the same block of ``chunk`` positions.  score = dot(q, k_j) / sqrt(hd) (divided after the product), or dot(q, k_j) * scale when a scale is
 // given.  Values may have another size than keys (vd).  With ``sink`` the denominator holds one more term, exp(0 - max):
 // a key of score zero that carries no value; with ``sink_vals`` the term is exp(sink_vals[head] - max), a number per head
-// that is not scaled.
+// that is not scaled.  With ``softcap`` > 0 the scaled score s becomes softcap * tanh(s / softcap).  ``maps`` > 1: a key
+// head's row in the cache holds that many keys side by side (hd numbers each) over one value; the query heads of a key
+// head come map by map within each head, so query head h reads the key h % maps of key head h / (nh / nkv).  The result
+// may be kept in float whatever the cache's type (TO), for a caller that goes on computing with it.
 // Keys are walked in chunks of CHUNK positions aligned to absolute multiples of
 // CHUNK with a running maximum and sum, so the order of every addition depends
 // on the query's position alone: not on how the sequence was cut into steps,
@@ -18,20 +21,20 @@ constexpr int CHUNK = 256;
 constexpr int THREADS = 128;
 constexpr int MAX_HD = 256;
 
-template <typename T>
+template <typename T, typename TO>
 __global__ void __launch_bounds__(THREADS)
 attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
-                 T* __restrict__ out, const int* __restrict__ tok_seq, const int* __restrict__ tok_pos,
+                 TO* __restrict__ out, const int* __restrict__ tok_seq, const int* __restrict__ tok_pos,
                  const int* __restrict__ block_table, int table_stride, int n_pages, int page, int nh, int nkv, int hd,
                  int vd, float scale, int sink, const float* __restrict__ sink_vals, int window, int chunk,
-                 int* __restrict__ status) {
+                 float softcap, int maps, int* __restrict__ status) {
     __shared__ float qs[MAX_HD];
     __shared__ float ps[CHUNK];
     __shared__ int pages[CHUNK];      // page id of each key of the chunk (or -1)
     __shared__ float scratch[33];
     const int n = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
     const int seq = tok_seq[n], pos = tok_pos[n];
-    const int kvh = h / (nh / nkv);
+    const int kvh = h / (nh / nkv), map = h % maps;
     const int lo = first_visible_key(pos, window, chunk);
     const T* qrow = q + ((size_t)n * nh + h) * hd;
     for (int d = tid; d < hd; d += THREADS) qs[d] = to_f32(qrow[d]);
@@ -58,10 +61,11 @@ attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T
             pages[t] = pg;
             float s = -INFINITY;
             if (pg >= 0) {
-                const T* krow = k_cache + (((size_t)pg * nkv + kvh) * page + j % page) * hd;
+                const T* krow = k_cache + ((((size_t)pg * nkv + kvh) * page + j % page) * maps + map) * hd;
                 float dot = 0.f;
                 for (int d = 0; d < hd; d++) dot = fmaf(qs[d], to_f32(krow[d]), dot);
                 s = scale > 0.f ? dot * scale : dot / root;
+                if (softcap > 0.f) s = softcap * tanhf(s / softcap);
             }
             ps[t] = s;
             local_max = fmaxf(local_max, s);
@@ -95,31 +99,33 @@ attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T
         }
         __syncthreads();
     }
-    T* orow = out + ((size_t)n * nh + h) * vd;
+    TO* orow = out + ((size_t)n * nh + h) * vd;
 #pragma unroll
     for (int i = 0; i < MAX_HD / THREADS; i++) {
         const int d = tid + i * THREADS;
-        if (d < vd) orow[d] = from_f32<T>(l_run > 0.f ? acc[i] / l_run : 0.f);
+        if (d < vd) orow[d] = from_f32<TO>(l_run > 0.f ? acc[i] / l_run : 0.f);
     }
 }
 }  // namespace
 
-ESP_API int esp_attn_simt(const void* q, const void* k_cache, const void* v_cache, void* out, int is_bf16,
+ESP_API int esp_attn_simt(const void* q, const void* k_cache, const void* v_cache, void* out, int is_bf16, int out_is_bf16,
                           const int* tok_seq, const int* tok_pos, const int* block_table, int table_stride, int n_pages,
                           int page, int n_tokens, int nh, int nkv, int hd, int vd, float scale, int sink,
-                          const float* sink_vals, int window, int chunk, int* status, cudaStream_t stream) {
+                          const float* sink_vals, int window, int chunk, float softcap, int maps, int* status,
+                          cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (vd <= 0) vd = hd;
-    if (vd > MAX_HD || hd > MAX_HD || hd <= 0 || nkv <= 0 || nh % nkv != 0 || nh > 65535) return (int)cudaErrorInvalidValue;
+    if (vd > MAX_HD || hd > MAX_HD || hd <= 0 || nkv <= 0 || nh % nkv != 0 || nh > 65535 || maps <= 0 || (nh / nkv) % maps != 0)
+        return (int)cudaErrorInvalidValue;
     dim3 grid(n_tokens, nh);
-    if (is_bf16)
-        attn_simt_kernel<bf16><<<grid, THREADS, 0, stream>>>((const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache,
-                                                            (bf16*)out, tok_seq, tok_pos, block_table, table_stride,
-                                                            n_pages, page, nh, nkv, hd, vd, scale, sink, sink_vals, window, chunk, status);
-    else
-        attn_simt_kernel<float><<<grid, THREADS, 0, stream>>>((const float*)q, (const float*)k_cache,
-                                                             (const float*)v_cache, (float*)out, tok_seq, tok_pos,
-                                                             block_table, table_stride, n_pages, page, nh, nkv, hd,
-                                                             vd, scale, sink, sink_vals, window, chunk, status);
+#define ESP_SIMT(T, TO)                                                                                                    \
+    attn_simt_kernel<T, TO><<<grid, THREADS, 0, stream>>>((const T*)q, (const T*)k_cache, (const T*)v_cache, (TO*)out, tok_seq, \
+                                                          tok_pos, block_table, table_stride, n_pages, page, nh, nkv, hd, vd, \
+                                                          scale, sink, sink_vals, window, chunk, softcap, maps, status)
+    if (is_bf16 && out_is_bf16) ESP_SIMT(bf16, bf16);
+    else if (is_bf16) ESP_SIMT(bf16, float);
+    else if (!out_is_bf16) ESP_SIMT(float, float);
+    else return (int)cudaErrorInvalidValue;
+#undef ESP_SIMT
     return esp_launch_status();
 }

@@ -474,7 +474,8 @@ ESP_API int esp_embed_sum(const void* table, const void* bigram, int table_is_bf
 // ---------------------------------------------------------------- norm of a sublayer's result + add + the next norm
 // Row r works on source row s = rows ? rows[r] : r.
 //   d = y[s] / sqrt(mean(y[s]^2) + eps_y) * gamma_y;  v = x[s] + d;  if (write_x) x[s] = v;
-//   h[r] = v / sqrt(mean(v^2) + eps) * gamma     (h null: only the first two lines)
+//   h[r] = v / sqrt(mean(v^2) + eps) * gamma     (h null: only the first two lines; gamma null: h[r] = v, for a layer
+//                                                  whose sublayers read the residual stream as it is)
 // All in 32-bit; sums of squares per thread in index order, combined by a fixed tree.  With ``x`` null the kernel
 // writes d itself to ``h32`` (the normed result alone).
 template <typename TH>
@@ -502,12 +503,12 @@ __global__ void norm_add_rmsnorm_kernel(float* __restrict__ x, const float* __re
         ss = fmaf(v, v, ss);
     }
     if (!h) return;
-    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)width + eps);
+    const float inv = gamma ? 1.0f / sqrtf(block_sum(ss, scratch) / (float)width + eps) : 1.0f;
     TH* hr = h + (size_t)r * width;
     float* h32r = h32 ? h32 + (size_t)r * width : nullptr;
     for (int i = threadIdx.x; i < width; i += blockDim.x) {
         const float v = write_x ? xr[i] : xr[i] + yr[i] * inv_y * gamma_y[i];
-        const float o = v * inv * gamma[i];
+        const float o = gamma ? v * inv * gamma[i] : v;
         hr[i] = from_f32<TH>(o);
         if (h32r) h32r[i] = o;
     }
@@ -560,6 +561,14 @@ norm_add_rmsnorm_rows_kernel(float* __restrict__ x, const float* __restrict__ y,
         }
     }
     if (!h) return;
+    if (!gamma) {                                        // no norm ahead of the next sublayer: x itself, in its dtype
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            const int q = threadIdx.x + i * blockDim.x;
+            if (q < pieces) Vec4<TH>::store(h + (size_t)r * width + 4 * q, v[i].x, v[i].y, v[i].z, v[i].w);
+        }
+        return;
+    }
     const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)width + eps);
 #pragma unroll
     for (int i = 0; i < 4; i++) {
@@ -577,7 +586,7 @@ ESP_API int esp_norm_add_rmsnorm(float* x, const float* y, const float* gamma_y,
                                  const int* rows, void* h, int h_is_bf16, float* h32, int n_rows, int width, float eps,
                                  int write_x, cudaStream_t stream) {
     if (n_rows <= 0) return 0;
-    if (!y || !gamma_y || (!x && !h32) || (h && !gamma)) return (int)cudaErrorInvalidValue;
+    if (!y || !gamma_y || (!x && !h32) || (h && !gamma && h32)) return (int)cudaErrorInvalidValue;
     if (x && width % 4 == 0 && width <= 16384) {
         // one piece per thread while a block can hold them (the thread count depends on the width alone in the 32-bit
         // path, so a row's sums have one order whatever else is in the step); many rows rounded to bfloat16: four
@@ -986,5 +995,46 @@ ESP_API int esp_cast_cols(const float* src, long long ld, void* dst, int dst_is_
         esp_launch_pdl(ESP_PDL_SMALL, cast_cols_kernel<bf16>, dim3((int)blocks), dim3(256), 0, stream, src, ld, (bf16*)dst, rows, width);
     else
         esp_launch_pdl(ESP_PDL_SMALL, cast_cols_kernel<float>, dim3((int)blocks), dim3(256), 0, stream, src, ld, (float*)dst, rows, width);
+    return esp_launch_status();
+}
+
+// ---------------------------------------------------------------- difference of two attention maps
+// a: float [rows, 2 * H, V], the outputs of maps one and two of every head side by side.  Per row and head:
+//   o = a_1 - lambda a_2;  o <- o / sqrt(mean(o^2) + eps) * out_scale * sigmoid(gate[row * ldg + head])
+// (gate null: no such factor), stored as y [rows, H, V].  One warp per row and head, everything in 32-bit.
+template <typename T>
+__global__ void __launch_bounds__(256)
+diff_combine_kernel(const float* __restrict__ a, float lambda, float eps, float out_scale, const float* __restrict__ gate,
+                    long long ldg, T* __restrict__ y, long long pairs, int H, int V) {
+    pdl_trigger();
+    pdl_wait();
+    const int lane = threadIdx.x & 31;
+    const long long pair = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    if (pair >= pairs) return;
+    const float* a1 = a + pair * 2 * V;
+    const float* a2 = a1 + V;
+    float ss = 0.f;
+    for (int d = lane; d < V; d += 32) {
+        const float o = a1[d] - lambda * a2[d];
+        ss = fmaf(o, o, ss);
+    }
+    ss = warp_sum(ss);
+    float f = out_scale / sqrtf(ss / (float)V + eps);
+    if (gate) f *= 1.0f / (1.0f + expf(-gate[pair / H * ldg + pair % H]));
+    for (int d = lane; d < V; d += 32) y[pair * V + d] = from_f32<T>((a1[d] - lambda * a2[d]) * f);
+}
+
+ESP_API int esp_diff_combine(const float* a, float lambda, float eps, float out_scale, const float* gate, long long ldg, void* y,
+                             int y_is_bf16, int n_rows, int H, int V, cudaStream_t stream) {
+    if (n_rows <= 0) return 0;
+    if (H <= 0 || V <= 0) return (int)cudaErrorInvalidValue;
+    const long long pairs = (long long)n_rows * H;
+    const unsigned blocks = (unsigned)((pairs + 7) / 8);
+    if (y_is_bf16)
+        esp_launch_pdl(ESP_PDL_SMALL, diff_combine_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, a, lambda, eps, out_scale,
+                       gate, ldg, (bf16*)y, pairs, H, V);
+    else
+        esp_launch_pdl(ESP_PDL_SMALL, diff_combine_kernel<float>, dim3(blocks), dim3(256), 0, stream, a, lambda, eps, out_scale,
+                       gate, ldg, (float*)y, pairs, H, V);
     return esp_launch_status();
 }

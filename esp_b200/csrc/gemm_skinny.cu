@@ -1,6 +1,7 @@
 // Weight-streaming matrix product for a handful of rows (decode):
 //   C[m, n] = scale[m] * sum_k A[row(m), k] * W[g][n, k]          (PLAIN)
-//   act[m, j] = silu(A W_gate[j]) * (A W_up[j])                   (SWIGLU; W = [gate rows; up rows])
+//   act[m, j] = silu(A W_gate[j]) * (A W_up[j])                   (SWIGLU; W = [gate rows; up rows]), or the unit with
+//                                                                  clamped branches of the same two products (glu_act)
 //   q / k / v of a decode step: the packed q/k/v projection whose epilogue adds the bias, rotates queries and
 //   keys by the token's position (split-half pairs (i, i + hd/2)) and writes the keys and values into the
 //   paged cache                                                  (ROPE; a tile holds 8 pairs)
@@ -37,6 +38,7 @@ struct SkinnyParams {
     const int* group_offsets;
     const float* row_scale;
     const float* act_pq;            // plain form only: null, or the two raw numbers of an xIELU applied to every output
+    float glu_limit, glu_alpha, glu_shift;   // SWIGLU form only, glu_limit > 0: the unit with clamped branches instead (glu_act)
     int act_relu2;                  // plain form only: every output (after its row's scale) becomes max(v, 0)^2
     void* C;
     long long ldc;
@@ -64,6 +66,16 @@ enum : int { MODE_PLAIN = 0, MODE_SWIGLU = 1, MODE_ROPE = 2 };
 __device__ __forceinline__ float skinny_softplus(float z) { return z > 20.f ? z : log1pf(expf(z)); }
 __device__ __forceinline__ float skinny_xielu(float v, float ap, float an) {
     return v > 0.f ? fmaf(ap * v, v, 0.5f * v) : fmaf(an, expm1f(v) - v, 0.5f * v);
+}
+
+// What the SWIGLU form makes of a feature's gate and up: silu(gate) * up, or (limit > 0) with g = min(gate, limit) and
+// u = clamp(up, -limit, limit) the value g sigmoid(alpha g) (u + shift), as the stand-alone kernel in elementwise.cu.
+__device__ __forceinline__ float glu_act(float gate, float up, float limit, float alpha, float shift) {
+    if (limit > 0.f) {
+        const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+        return g / (1.0f + expf(-alpha * g)) * (u + shift);
+    }
+    return gate / (1.0f + expf(-gate)) * up;
 }
 
 // One pair (x[i], x[i + hd/2]) of head ``head`` of token row m: bias, rotation in float with the same
@@ -273,7 +285,7 @@ gemm_skinny_kernel(SkinnyParams p) {
                         if (j < p.N) {
                             const float gate = acc[nb][i], up = acc[nb][2 + i];
                             reinterpret_cast<TC*>(p.C)[(size_t)(m0 + tok) * p.ldc + j] =
-                                from_f32<TC>(gate / (1.0f + expf(-gate)) * up);
+                                from_f32<TC>(glu_act(gate, up, p.glu_limit, p.glu_alpha, p.glu_shift));
                         }
                     } else {
                         const float scale = p.row_scale ? p.row_scale[m0 + tok] : 1.0f;
@@ -315,7 +327,7 @@ gemm_skinny_kernel(SkinnyParams p) {
                     if (ROPE) {
                         emit_rope_pair(p, m0 + tok, j, gate, up);
                     } else {
-                        const float v = gate / (1.0f + expf(-gate)) * up;
+                        const float v = glu_act(gate, up, p.glu_limit, p.glu_alpha, p.glu_shift);
                         reinterpret_cast<TC*>(p.C)[(size_t)(m0 + tok) * p.ldc + j] = from_f32<TC>(v);
                     }
                 }
@@ -401,7 +413,7 @@ int launch(const SkinnyParams& p, int groups, cudaStream_t stream) {
 ESP_API int esp_gemm_skinny(const void* A, long long lda, const int* a_rows, const void* W, long long w_group_stride,
                             const float* row_scale, void* C, int c_dtype, long long ldc, const int* group_offsets,
                             int groups, int M, int N, int K, int max_rows, int swiglu, int offsets_ready, const float* act_pq,
-                            cudaStream_t stream) {
+                            float glu_limit, float glu_alpha, float glu_shift, cudaStream_t stream) {
     if (M <= 0 || N <= 0) return 0;
     const int relu2 = swiglu == 2 ? 1 : 0;
     if (relu2) swiglu = 0;
@@ -409,6 +421,7 @@ ESP_API int esp_gemm_skinny(const void* A, long long lda, const int* a_rows, con
     SkinnyParams p{};
     p.act_pq = act_pq;
     p.act_relu2 = relu2;
+    p.glu_limit = glu_limit; p.glu_alpha = glu_alpha; p.glu_shift = glu_shift;
     p.offsets_ready = group_offsets && offsets_ready ? 1 : 0;
     p.W = (const bf16*)W; p.w_group_stride = w_group_stride; p.A = (const bf16*)A; p.lda = lda; p.a_rows = a_rows;
     p.group_offsets = group_offsets; p.row_scale = row_scale; p.C = C; p.ldc = ldc; p.M = M; p.N = N; p.K = K;

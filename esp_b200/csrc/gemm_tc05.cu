@@ -51,6 +51,8 @@ struct Tc05Params {
     long long ldc;
     int M, N, K;                  // N: output columns (SWIGLU: the intermediate size)
     int* status;
+    // SWIGLU, glu_limit > 0: with g = min(gate, limit), u = clamp(up, -limit, limit) the output is g sigmoid(alpha g) (u + shift)
+    float glu_limit, glu_alpha, glu_shift;
 };
 
 // Instruction descriptor: bfloat16 x bfloat16 -> float, both operands K-major, M = 128, N = n.
@@ -460,6 +462,10 @@ gemm_tc05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
                 const int f = t.f0 + pair * 32 + lane;
                 const bool f_ok = f < p.N;
                 bf16* out = reinterpret_cast<bf16*>(p.C);
+                // the plain form is the clamped one without limits, slope one and shift zero
+                const bool clamped = p.glu_limit > 0.f;
+                const float g_max = clamped ? p.glu_limit : INFINITY, g_alpha = clamped ? p.glu_alpha : 1.f;
+                const float u_shift = clamped ? p.glu_shift : 0.f;
                 int flip = 0;
                 for (int c0 = half * 32; c0 < t.n_tok; c0 += 64, flip ^= 1) {
                     float acc[32];
@@ -474,10 +480,12 @@ gemm_tc05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
                     for (int i = 0; i < 16; i++) {
                         const float other = theirs[i * 32 + lane];
                         const float own = is_up ? acc[16 + i] : acc[i];
-                        const float g = is_up ? other : own, u = is_up ? own : other;
+                        float g = is_up ? other : own, u = is_up ? own : other;
+                        g = fminf(g, g_max);
+                        u = fminf(fmaxf(u, -g_max), g_max) + u_shift;
                         const int row = c0 + keep + i;
                         if (f_ok && row < t.n_rows)
-                            out[(size_t)(t.row0 + row) * p.ldc + f] = __float2bfloat16_rn(__fdividef(g, 1.0f + __expf(-g)) * u);
+                            out[(size_t)(t.row0 + row) * p.ldc + f] = __float2bfloat16_rn(__fdividef(g, 1.0f + __expf(-g_alpha * g)) * u);
                     }
                 }
             } else {
@@ -556,7 +564,7 @@ int make_map(CUtensorMap* map, const void* base, unsigned long long d0, unsigned
 ESP_API int esp_gemm_tc05(const void* A, long long rows_total, const void* W, int groups, int w_rows,
                           const float* row_scale, void* C, long long ldc, const int* tile_group, const int* tile_row0,
                           const int* tile_rows, const int* n_tiles, int max_tiles, int tile_max, int M, int N, int K, int swiglu,
-                          int pair, int max_ctas, int* status, cudaStream_t stream) {
+                          int pair, int max_ctas, float glu_limit, float glu_alpha, float glu_shift, int* status, cudaStream_t stream) {
     if (N <= 0 || K <= 0 || rows_total <= 0) return 0;
     if (max_ctas < 0 || (pair && max_ctas == 1)) return (int)cudaErrorInvalidValue;
     if (K % 8 != 0 || ((uintptr_t)A & 15) || ((uintptr_t)W & 15)) return (int)cudaErrorInvalidValue;
@@ -570,7 +578,7 @@ ESP_API int esp_gemm_tc05(const void* A, long long rows_total, const void* W, in
     // the weights always use a 3-D map so that the kernel has one code path; a dense product is one group
     rc = make_map(&map_w, W, (unsigned long long)K, (unsigned long long)w_rows, (unsigned long long)groups, swiglu ? BF / 2 : BF, 3);
     if (rc) return rc;
-    Tc05Params p{tile_group, tile_row0, tile_rows, n_tiles, row_scale, C, ldc, M, N, K, status};
+    Tc05Params p{tile_group, tile_row0, tile_rows, n_tiles, row_scale, C, ldc, M, N, K, status, glu_limit, glu_alpha, glu_shift};
     // ``tile_max``: the most rows a tile of the list has, 128 or 256 (with 256 an expert's weights pass once
     // for up to 256 of its rows); dense products cut tiles of 256 rows (MMAs of N = 256 run at the full rate)
     if (tile_group && tile_max != 128 && tile_max != 256) return (int)cudaErrorInvalidValue;

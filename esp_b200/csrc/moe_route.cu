@@ -13,26 +13,28 @@ constexpr int ROUTE_SMALL_MAX = 64;          // tokens of a step that the two-la
 enum : int {
     ROUTE_RENORM = 1,     // the chosen experts' scores are divided by their sum
     ROUTE_SIGMOID = 2,    // scores are sigmoid(logit), each expert by itself, instead of a softmax over all experts
+    ROUTE_CHOSEN = 4,     // scores are the logits themselves; the weights are a softmax over the chosen experts' logits alone
 };
 
-// A token's scores from its logits, by one warp: ps[e] = softmax(lg)[e], or sigmoid(lg[e]).  lg and ps may be the same
-// array.  ``probs`` (may be null) receives a copy.
-__device__ __forceinline__ void scores_from_logits(const float* lg, float* ps, int n_experts, int lane, int sigmoid,
-                                                   float* probs) {
-    if (sigmoid) {
+// A token's scores from its logits, by one warp: with z = lg + bias (null: no bias) ps[e] = softmax(z)[e], sigmoid(z[e])
+// or z[e] itself (``flags``).  lg and ps may be the same array.  ``probs`` (may be null) receives a copy.
+__device__ __forceinline__ void scores_from_logits(const float* lg, float* ps, int n_experts, int lane, int flags,
+                                                   const float* bias, float* probs) {
+    if (flags & (ROUTE_SIGMOID | ROUTE_CHOSEN)) {
         for (int e = lane; e < n_experts; e += 32) {
-            const float p = 1.0f / (1.0f + expf(-lg[e]));
+            const float z = lg[e] + (bias ? bias[e] : 0.f);
+            const float p = (flags & ROUTE_CHOSEN) ? z : 1.0f / (1.0f + expf(-z));
             ps[e] = p;
             if (probs) probs[e] = p;
         }
         return;
     }
     float mx = -INFINITY;
-    for (int e = lane; e < n_experts; e += 32) mx = fmaxf(mx, lg[e]);
+    for (int e = lane; e < n_experts; e += 32) mx = fmaxf(mx, lg[e] + (bias ? bias[e] : 0.f));
     mx = warp_max(mx);
     float sum = 0.f;
     for (int e = lane; e < n_experts; e += 32) {
-        const float p = expf(lg[e] - mx);
+        const float p = expf(lg[e] + (bias ? bias[e] : 0.f) - mx);
         ps[e] = p;
         sum += p;
     }
@@ -52,7 +54,23 @@ struct RouteChoice {
     const float* correction;
     int n_groups;
     int keep;
+    const float* bias;      // a number per expert added to its logit (may be null)
 };
+
+// The routing weight of a lane's chosen expert (rank = lane) from its score and the sum of the chosen scores; ``bad`` is
+// set where there is nothing to divide by.
+__device__ __forceinline__ float routing_weight(float my_p, float mass, int flags, int lane, int top_k, bool& bad) {
+    if (flags & ROUTE_CHOSEN) {
+        const float best = __shfl_sync(0xffffffffu, my_p, 0);             // rank 0 is the largest logit
+        const float e = lane < top_k ? expf(my_p - best) : 0.f;
+        const float sum = warp_sum(e);
+        if (!(sum > 0.f)) bad = true;
+        return e / sum;
+    }
+    const float denom = (flags & ROUTE_RENORM) ? mass : 1.0f;
+    if (!(denom > 0.f)) bad = true;
+    return my_p / denom;
+}
 
 // One token's top-k by one warp.  ps[e]: its scores (left as they are when a correction or groups are given, else
 // the chosen entries are overwritten); cs: n_experts floats of scratch for the corrected scores.  The k experts with
@@ -230,19 +248,19 @@ router_topk_kernel(const TH* __restrict__ h, const TW* __restrict__ w_router, co
     for (int t = warp; t < live; t += nwarp) {
         const int n = n0 + t;
         float* ps = ps_all + t * n_experts;
-        scores_from_logits(ps, ps, n_experts, lane, norm_topk & ROUTE_SIGMOID, probs_out ? probs_out + (size_t)n * n_experts : nullptr);
+        scores_from_logits(ps, ps, n_experts, lane, norm_topk, choice.bias, probs_out ? probs_out + (size_t)n * n_experts : nullptr);
         __syncwarp();
         bool bad = false;
         float my_p = 0.f;
         int my_e = 0;
         const float mass = choose_topk(ps, cs_all + t * n_experts, n_experts, top_k, lane, choice, my_p, my_e, bad);
-        const float denom = (norm_topk & ROUTE_RENORM) ? mass : 1.0f;
-        if (__any_sync(0xffffffffu, bad) || !(denom > 0.f)) {
+        const float wt = routing_weight(my_p, mass, norm_topk, lane, top_k, bad);
+        if (__any_sync(0xffffffffu, bad)) {
             if (lane == 0) atomicOr(status, ESP_STATUS_ROUTER_NONFINITE);
         }
         if (lane < top_k) {
             topk_ids[(size_t)n * top_k + lane] = my_e;
-            topk_w[(size_t)n * top_k + lane] = my_p / denom;
+            topk_w[(size_t)n * top_k + lane] = wt;
         }
     }
 }
@@ -352,20 +370,20 @@ router_select_kernel(const float* __restrict__ logits, int* __restrict__ topk_id
     if (n >= n_tokens) return;
     float* ps = sel_ps + warp * 2 * n_experts;
     const float* lg = logits + (size_t)n * (n_experts + 1);
-    scores_from_logits(lg, ps, n_experts, lane, norm_topk & ROUTE_SIGMOID, probs_out ? probs_out + (size_t)n * n_experts : nullptr);
+    scores_from_logits(lg, ps, n_experts, lane, norm_topk, choice.bias, probs_out ? probs_out + (size_t)n * n_experts : nullptr);
     if (lane == 0 && has_gate) gate[n] = 1.0f / (1.0f + expf(-lg[n_experts]));
     __syncwarp();
     bool bad = false;
     float my_p = 0.f;
     int my_e = 0;
     const float mass = choose_topk(ps, ps + n_experts, n_experts, top_k, lane, choice, my_p, my_e, bad);
-    const float denom = (norm_topk & ROUTE_RENORM) ? mass : 1.0f;
-    if (__any_sync(0xffffffffu, bad) || !(denom > 0.f)) {
+    const float wt = routing_weight(my_p, mass, norm_topk, lane, top_k, bad);
+    if (__any_sync(0xffffffffu, bad)) {
         if (lane == 0) atomicOr(status, ESP_STATUS_ROUTER_NONFINITE);
     }
     if (lane < top_k) {
         topk_ids[(size_t)n * top_k + lane] = my_e;
-        topk_w[(size_t)n * top_k + lane] = my_p / denom;
+        topk_w[(size_t)n * top_k + lane] = wt;
     }
 }
 
@@ -419,19 +437,19 @@ route_small_kernel(const float* __restrict__ logits, int* __restrict__ topk_ids,
     float* ps = ps_all + warp * 2 * n_experts;
     for (int n = warp; n < n_tokens; n += 8) {
         const float* lg = logits + (size_t)n * (n_experts + 1);
-        scores_from_logits(lg, ps, n_experts, lane, norm_topk & ROUTE_SIGMOID, probs_out ? probs_out + (size_t)n * n_experts : nullptr);
+        scores_from_logits(lg, ps, n_experts, lane, norm_topk, choice.bias, probs_out ? probs_out + (size_t)n * n_experts : nullptr);
         if (lane == 0 && has_gate) gate[n] = 1.0f / (1.0f + expf(-lg[n_experts]));
         __syncwarp();
         bool bad = false;
         float my_p = 0.f;
         int my_e = 0;
         const float mass = choose_topk(ps, ps + n_experts, n_experts, top_k, lane, choice, my_p, my_e, bad);
-        const float denom = (norm_topk & ROUTE_RENORM) ? mass : 1.0f;
-        if (__any_sync(0xffffffffu, bad) || !(denom > 0.f)) {
+        const float wt = routing_weight(my_p, mass, norm_topk, lane, top_k, bad);
+        if (__any_sync(0xffffffffu, bad)) {
             if (lane == 0) atomicOr(status, ESP_STATUS_ROUTER_NONFINITE);
         }
         if (lane < top_k) {
-            const float w = my_p / denom;
+            const float w = wt;
             topk_ids[(size_t)n * top_k + lane] = my_e;
             topk_w[(size_t)n * top_k + lane] = w;
             pair_e[n * top_k + lane] = my_e;                      // kept in shared memory for the placement below
@@ -714,7 +732,8 @@ __global__ void moe_combine_kernel(const float* __restrict__ expert_out, const i
 //   y = (sum of the row's expert outputs in ascending expert id) + gate * shared      (as moe_combine_kernel)
 //   v = x[s] + y;  if (write_x) x[s] = v;  h[r] = v * rsqrt(mean(v^2) + eps) * gamma  (as add_rmsnorm)
 // with s = rows ? rows[r] : r.  Same operations in the same order as the two separate kernels, so the
-// results are the same bits.  Width a multiple of 4, at most 16384.
+// results are the same bits.  Width a multiple of 4, at most 16384.  With gamma_y the combined row is normalised before it
+// is added: y <- y / sqrt(mean(y^2) + eps_y) * gamma_y.  gamma null: h[r] = v as it is; h null: the add alone.
 template <typename TH>
 __global__ void __launch_bounds__(1024)
 moe_combine_add_rmsnorm_kernel(const float* __restrict__ expert_out, const int* __restrict__ topk_ids,
@@ -722,7 +741,7 @@ moe_combine_add_rmsnorm_kernel(const float* __restrict__ expert_out, const int* 
                                const float* __restrict__ shared, float* __restrict__ x, const float* __restrict__ gamma,
                                const int* __restrict__ rows, TH* __restrict__ h, float* __restrict__ h32, int width,
                                int top_k, float eps, int write_x, int early, const float* __restrict__ topk_w,
-                               const float* __restrict__ ident, int n_real) {
+                               const float* __restrict__ ident, int n_real, const float* __restrict__ gamma_y, float eps_y) {
     pdl_trigger();
     // The kernel before this one in the stream made the experts' rows or the shared expert's row.  It lets this one
     // be set up only behind its own wait (the grouped product gives its signal when its weights are in), and by then
@@ -759,7 +778,8 @@ moe_combine_add_rmsnorm_kernel(const float* __restrict__ expert_out, const int* 
     }
     __syncthreads();
     pdl_wait();
-    float ss = 0.f;
+    float4 y[4];
+    float ssy = 0.f;
 #pragma unroll
     for (int i = 0; i < 4; i++) {
         const int q = threadIdx.x + i * blockDim.x;
@@ -780,6 +800,22 @@ moe_combine_add_rmsnorm_kernel(const float* __restrict__ expert_out, const int* 
                 const float4 e = reinterpret_cast<const float4*>(shared + t * width)[q];
                 acc.x += g * e.x; acc.y += g * e.y; acc.z += g * e.z; acc.w += g * e.w;
             }
+            y[i] = acc;
+            if (gamma_y) ssy = fmaf(acc.w, acc.w, fmaf(acc.z, acc.z, fmaf(acc.y, acc.y, fmaf(acc.x, acc.x, ssy))));
+        }
+    }
+    const float inv_y = gamma_y ? 1.0f / sqrtf(block_sum(ssy, scratch) / (float)width + eps_y) : 1.0f;
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        const int q = threadIdx.x + i * blockDim.x;
+        if (q < pieces) {
+            float4 acc = y[i];
+            if (gamma_y) {
+                const float4 gy = reinterpret_cast<const float4*>(gamma_y)[q];
+                acc.x = acc.x * inv_y * gy.x; acc.y = acc.y * inv_y * gy.y;
+                acc.z = acc.z * inv_y * gy.z; acc.w = acc.w * inv_y * gy.w;
+            }
             float4 xv = v[i];
             xv.x += acc.x; xv.y += acc.y; xv.z += acc.z; xv.w += acc.w;
             if (write_x) reinterpret_cast<float4*>(x + t * width)[q] = xv;
@@ -789,6 +825,15 @@ moe_combine_add_rmsnorm_kernel(const float* __restrict__ expert_out, const int* 
             ss = fmaf(xv.z, xv.z, ss);
             ss = fmaf(xv.w, xv.w, ss);
         }
+    }
+    if (!h) return;
+    if (!gamma) {
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            const int q = threadIdx.x + i * blockDim.x;
+            if (q < pieces) Vec4<TH>::store(h + (size_t)r * width + 4 * q, v[i].x, v[i].y, v[i].z, v[i].w);
+        }
+        return;
     }
     const float total = block_sum(ss, scratch);
     const float inv = 1.0f / sqrtf(total / (float)width + eps);
@@ -810,14 +855,14 @@ moe_combine_add_rmsnorm_kernel(const float* __restrict__ expert_out, const int* 
 // weights, many tokens and a width that is a multiple of 128, the logits are made on the tensor cores.
 ESP_API int esp_router_topk(const void* h, int h_is_bf16, const void* w_router, const void* w_gate, int w_is_bf16,
                             int* topk_ids, float* topk_w, float* gate, float* probs_out, float* logits, int n_tokens,
-                            int width, int n_experts, int top_k, int norm_topk, const float* correction, int n_groups,
+                            int width, int n_experts, int top_k, int norm_topk, const float* bias, const float* correction, int n_groups,
                             int keep_groups, int* status, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (top_k > MAX_TOPK || top_k <= 0 || top_k > n_experts) return (int)cudaErrorInvalidValue;
     if (n_groups > 32 || (n_groups > 1 && (n_experts % n_groups != 0 || keep_groups < 1 || keep_groups > n_groups ||
                                            keep_groups * (n_experts / n_groups) < top_k)))
         return (int)cudaErrorInvalidValue;
-    const RouteChoice choice{correction, n_groups, keep_groups};
+    const RouteChoice choice{correction, n_groups, keep_groups, bias};
     const int rows = n_experts + (w_gate ? 1 : 0);
     if (logits && !h_is_bf16 && w_is_bf16 && n_tokens >= 64 && width % 128 == 0 && rows <= 72 &&
         (size_t)16 * n_experts * sizeof(float) <= 48 * 1024 && (reinterpret_cast<uintptr_t>(h) & 15) == 0 &&
@@ -874,7 +919,7 @@ ESP_API int esp_route_small(const void* h, int h_is_bf16, const void* w_router, 
                             float* logits, int* topk_ids, float* topk_w, float* gate, float* probs_out, int n_tokens,
                             int width, int n_experts, int top_k, int norm_topk, int* offsets, int* perm_token,
                             float* perm_weight, int* inverse, int* status, unsigned long long* distinct, int* tile_group,
-                            int* tile_row0, int* tile_count, int* n_tiles, int max_tiles, const float* correction,
+                            int* tile_row0, int* tile_count, int* n_tiles, int max_tiles, const float* bias, const float* correction,
                             int n_groups, int keep_groups, int n_real, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (top_k > MAX_TOPK || top_k <= 0 || top_k > n_experts || n_tokens > ROUTE_SMALL_MAX) return (int)cudaErrorInvalidValue;
@@ -882,7 +927,7 @@ ESP_API int esp_route_small(const void* h, int h_is_bf16, const void* w_router, 
         (n_groups > 1 && (n_experts % n_groups != 0 || keep_groups < 1 || keep_groups > n_groups ||
                           keep_groups * (n_experts / n_groups) < top_k)))
         return (int)cudaErrorInvalidValue;
-    const RouteChoice choice{correction, n_groups, keep_groups};
+    const RouteChoice choice{correction, n_groups, keep_groups, bias};
     // the tile list (all four or none): one tile per expert with rows (experts from n_real on have none)
     if (tile_group && (!tile_row0 || !tile_count || !n_tiles || max_tiles < (n_real < n_tokens * top_k ? n_real : n_tokens * top_k)))
         return (int)cudaErrorInvalidValue;
@@ -943,9 +988,10 @@ ESP_API int esp_moe_combine(const float* expert_out, const int* topk_ids, const 
 ESP_API int esp_moe_combine_add_rmsnorm(const float* expert_out, const int* topk_ids, const int* inverse, const float* gate,
                                         const float* shared, float* x, const float* gamma, const int* rows, void* h,
                                         int h_is_bf16, float* h32, int n_rows, int width, int top_k, float eps, int write_x,
-                                        const float* topk_w, const float* ident, int n_real, cudaStream_t stream) {
+                                        const float* topk_w, const float* ident, int n_real, const float* gamma_y,
+                                        float eps_y, cudaStream_t stream) {
     if (n_rows <= 0) return 0;
-    if (top_k > MAX_TOPK || width % 4 != 0 || width > 16384 || (ident && !topk_w)) return (int)cudaErrorInvalidValue;
+    if (top_k > MAX_TOPK || width % 4 != 0 || width > 16384 || (ident && !topk_w) || (h32 && (!h || !gamma))) return (int)cudaErrorInvalidValue;
     int threads = ((width / 4 + 3) / 4 + 31) / 32 * 32;
     // one piece per thread while a block can hold them: a row's sum then has the same order whatever else is in the
     // step (the 32-bit path relies on it).  Many rows rounded to bfloat16: four pieces per thread, smaller blocks,
@@ -954,10 +1000,10 @@ ESP_API int esp_moe_combine_add_rmsnorm(const float* expert_out, const int* topk
     const int early = esp_pdl_enabled(ESP_PDL_GROUPED) ? 0 : 1;
     if (h_is_bf16)
         esp_launch_pdl(ESP_PDL_SMALL, moe_combine_add_rmsnorm_kernel<bf16>, dim3(n_rows), dim3(threads), 0, stream, expert_out, topk_ids, inverse, gate, shared, x, gamma,
-                                                                            rows, (bf16*)h, h32, width, top_k, eps, write_x, early, topk_w, ident, n_real);
+                                                                            rows, (bf16*)h, h32, width, top_k, eps, write_x, early, topk_w, ident, n_real, gamma_y, eps_y);
     else
         esp_launch_pdl(ESP_PDL_SMALL, moe_combine_add_rmsnorm_kernel<float>, dim3(n_rows), dim3(threads), 0, stream, expert_out, topk_ids, inverse, gate, shared, x,
                                                                              gamma, rows, (float*)h, h32, width, top_k, eps,
-                                                                             write_x, early, topk_w, ident, n_real);
+                                                                             write_x, early, topk_w, ident, n_real, gamma_y, eps_y);
     return esp_launch_status();
 }

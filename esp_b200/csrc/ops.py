@@ -46,8 +46,11 @@ _SIGNATURES = {
     "esp_gemm_simt": [P, c_int, P, P, c_int, P, P, P, c_int, P, c_int, c_int, c_int, c_int, c_longlong, c_longlong, P],
     "esp_rope_kvwrite": [P, P, P, P, P, P, c_int, c_int, P, P, P, c_int, P, c_int, c_int, c_int, c_int, c_int, c_int,
                          c_int, c_int, P, P],
-    "esp_attn_simt": [P, P, P, P, c_int, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, P,
-                      c_int, c_int, P, P],
+    "esp_attn_simt": [P, P, P, P, c_int, c_int, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, P,
+                      c_int, c_int, c_float, c_int, P, P],
+    "esp_headnorm_rope_kvwrite": [P, c_longlong, P, P, c_float, P, c_int, P, P, P, P, P, c_int, P, c_int, c_int, c_int, c_int,
+                                  c_int, c_int, c_int, c_int, c_int, c_int, P, P],
+    "esp_diff_combine": [P, c_float, c_float, c_float, P, c_longlong, P, c_int, c_int, c_int, c_int, P],
     "esp_embed_sum": [P, P, c_int, P, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_longlong, c_longlong, c_float, P, P],
     "esp_norm_add_rmsnorm": [P, P, P, c_float, P, P, P, c_int, P, c_int, c_int, c_float, c_int, P],
     "esp_relu2": [P, P, P, c_int, c_longlong, c_int, P],
@@ -75,19 +78,20 @@ _SIGNATURES = {
     "esp_pair_rope_unitnorm_kvwrite": [P, P, P, c_int, c_float, c_int, P, c_int, P, P, P, P, P, P, c_int, P, c_int, c_int, c_int,
                                        c_int, c_int, c_int, c_int, c_int, c_int, P, P],
     "esp_causal_conv": [P, c_longlong, P, P, P, c_longlong, P, P, P, P, c_int, c_int, c_int, c_int, c_int, P],
-    "esp_router_topk": [P, c_int, P, P, c_int, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, P, c_int, c_int, P, P],
+    "esp_router_topk": [P, c_int, P, P, c_int, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, P, P, c_int, c_int, P, P],
     "esp_moe_permute": [P, P, c_int, c_int, c_int, P, P, P, P, P, P, P, P, c_int, c_int, P, P, c_int, P],
     "esp_gather_rows": [P, P, P, c_int, c_int, P],
     "esp_route_small": [P, c_int, P, P, c_int, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, P, P, P, P, P, P, P, P, P, P,
-                        c_int, P, c_int, c_int, c_int, P],
+                        c_int, P, P, c_int, c_int, c_int, P],
     "esp_gemm_tc05": [P, c_longlong, P, c_int, c_int, P, P, c_longlong, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int,
-                      c_int, c_int, P, P],
+                      c_int, c_int, c_float, c_float, c_float, P, P],
     "esp_wait_probe": [c_int, P, P],
     "esp_moe_combine": [P, P, P, P, P, P, c_int, c_int, c_int, P, P, c_int, P],
     "esp_pick_tokens": [P, c_int, c_int, P, P, P, P, P, P],
-    "esp_moe_combine_add_rmsnorm": [P, P, P, P, P, P, P, P, P, c_int, P, c_int, c_int, c_int, c_float, c_int, P, P, c_int, P],
+    "esp_moe_combine_add_rmsnorm": [P, P, P, P, P, P, P, P, P, c_int, P, c_int, c_int, c_int, c_float, c_int, P, P, c_int, P, c_float,
+                                    P],
     "esp_gemm_skinny": [P, c_longlong, P, P, c_longlong, P, P, c_int, c_longlong, P, c_int, c_int, c_int, c_int, c_int,
-                        c_int, c_int, P, P],
+                        c_int, c_int, P, c_float, c_float, c_float, P],
     "esp_qkv_rope_skinny": [P, c_longlong, P, P, P, P, P, P, c_int, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int,
                             c_int, c_int, c_int, P, P],
     "esp_attn_prefill": [P, P, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int,
@@ -96,6 +100,8 @@ _SIGNATURES = {
                               c_int, P, c_int, c_int, P, P],
     "esp_attn_decode": [P, P, P, P, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                         c_int, c_float, c_int, P, c_int, P, P],
+    "esp_attn_decode_diff": [P, P, P, P, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                             c_int, c_int, c_float, c_int, c_float, c_float, c_float, c_float, P, c_longlong, P, P],
 }
 
 _bound: dict = {}
@@ -359,8 +365,10 @@ def _sink_args(sink, nh):
 
 
 def attn_simt(q, k_cache, v_cache, out, tok_seq, tok_pos, block_table, page, nh, nkv, hd, window, status, vd=None,
-              scale=0.0, sink=False, chunk=None):
-    """Attention of every token over its sequence's cached keys (32-bit arithmetic).  ``vd``: size of a value head
+              scale=0.0, sink=False, chunk=None, softcap=None, maps=1):
+    """Attention of every token over its sequence's cached keys (32-bit arithmetic).  ``out`` may be float32 whatever the
+    cache's dtype.  ``softcap``: scaled scores s become softcap * tanh(s / softcap).  ``maps``: keys that lie side by side
+    in a key head's row of the cache; query head h reads the key h % maps of its key head.  ``vd``: size of a value head
     (default: the key size); ``scale`` > 0 multiplies the scores instead of the division by sqrt(hd); ``sink``: the
     softmax's denominator holds one more term exp(0), or exp(sink[head]) when a tensor is given; ``chunk``: a query
     sees the keys of its own block of that many positions only."""
@@ -370,9 +378,9 @@ def attn_simt(q, k_cache, v_cache, out, tok_seq, tok_pos, block_table, page, nh,
         raise Backend(f"attention: head sizes {hd} / {vd} are beyond the 256 this kernel takes")
     _check(_fn("core", "esp_attn_simt")(
         _ptr(q, FLOATS, "q"), _ptr(k_cache, FLOATS), _ptr(v_cache, FLOATS), _ptr(out, FLOATS), _is_bf16(q),
-        _ptr(tok_seq, torch.int32), _ptr(tok_pos, torch.int32), _ptr(block_table, torch.int32), block_table.shape[1],
+        _is_bf16(out), _ptr(tok_seq, torch.int32), _ptr(tok_pos, torch.int32), _ptr(block_table, torch.int32), block_table.shape[1],
         k_cache.shape[0], page, q.shape[0], nh, nkv, hd, vd, float(scale), sink_flag, sink_ptr, int(window or 0),
-        int(chunk or 0), _ptr(status, torch.int32), _stream()), "attn_simt")
+        int(chunk or 0), float(softcap or 0.0), int(maps), _ptr(status, torch.int32), _stream()), "attn_simt")
 
 
 def _choice_args(choice, n_experts):
@@ -388,8 +396,9 @@ def _choice_args(choice, n_experts):
 
 
 def router_topk(h, w_router, w_gate, topk_ids, topk_w, gate, top_k, norm_topk, status, probs_out=None, logits=None,
-                sigmoid=False, choice=None):
-    """``choice``: None, or (correction, groups, keep): a number per expert added to its score for the choice only, and
+                sigmoid=False, choice=None, bias=None, chosen_softmax=False):
+    """``bias``: float32, a number per expert added to its logit.  ``chosen_softmax``: the experts with the largest logits,
+    weighted by a softmax over those logits alone.  ``choice``: None, or (correction, groups, keep): a number per expert added to its score for the choice only, and
     a limit of the choice to the best ``keep`` of ``groups`` equal groups of neighbouring experts.  ``logits``: optional float32 scratch [n, experts + 1]; with it, 32-bit activations and bfloat16 weights
     the logits of a step of many tokens are made on the tensor cores (three bfloat16 parts of every
     activation: products exact, sums in float)."""
@@ -404,11 +413,14 @@ def router_topk(h, w_router, w_gate, topk_ids, topk_w, gate, top_k, norm_topk, s
         raise Backend("router: router and shared-gate weights must share a dtype")
     if logits is not None and logits.numel() < n * (n_experts + 1):
         raise Backend("router: the logits scratch is smaller than [tokens, experts + 1]")
+    if bias is not None and bias.shape[0] != n_experts:
+        raise Backend("router: the bias has another length than the router has outputs")
     _check(_fn("core", "esp_router_topk")(
         _ptr(h, FLOATS, "h"), _is_bf16(h), _ptr(w_router, FLOATS), _ptr(w_gate, FLOATS), _is_bf16(w_router),
         _ptr(topk_ids, torch.int32), _ptr(topk_w, torch.float32), _ptr(gate, torch.float32),
         _ptr(probs_out, torch.float32), _ptr(logits, torch.float32), n, width, n_experts, top_k,
-        (1 if norm_topk else 0) | (2 if sigmoid else 0), pc, groups, keep, _ptr(status, torch.int32), _stream()), "router_topk")
+        (1 if norm_topk else 0) | (2 if sigmoid else 0) | (4 if chosen_softmax else 0), _ptr(bias, torch.float32, "bias"), pc,
+        groups, keep, _ptr(status, torch.int32), _stream()), "router_topk")
 
 
 ROUTE_SMALL_TOKENS = 64
@@ -421,8 +433,8 @@ def route_small_fits(width: int, n_experts: int) -> bool:
 
 def route_small(h, w_router, w_gate, logits, topk_ids, topk_w, gate, top_k, norm_topk, offsets, perm_token,
                 perm_weight, inverse, status, probs_out=None, distinct=None, tiles=None, sigmoid=False, choice=None,
-                n_real=None):
-    """``choice``: as for router_topk.  ``n_real``: experts from this id on have no rows (their pairs get inverse -1).
+                n_real=None, bias=None, chosen_softmax=False):
+    """``bias``, ``chosen_softmax``: as for router_topk.  ``choice``: as for router_topk.  ``n_real``: experts from this id on have no rows (their pairs get inverse -1).
     Router and permutation for at most ROUTE_SMALL_TOKENS tokens: logits over many blocks, then one
     block for softmax, top-k and the permutation.  ``logits``: float32 scratch [N, E + 1].  ``distinct``:
     an int64 tensor of one element to which the number of experts with at least one token is added.
@@ -432,15 +444,17 @@ def route_small(h, w_router, w_gate, logits, topk_ids, topk_w, gate, top_k, norm
     if n > ROUTE_SMALL_TOKENS or top_k > 32 or not route_small_fits(width, n_experts):
         raise Backend("route_small: too many tokens or experts for this kernel")
     pc, groups, keep = _choice_args(choice, n_experts)
+    if bias is not None and bias.shape[0] != n_experts:
+        raise Backend("route_small: the bias has another length than the router has outputs")
     _check(_fn("core", "esp_route_small")(
         _ptr(h, FLOATS, "h"), _is_bf16(h), _ptr(w_router, FLOATS), _ptr(w_gate, FLOATS), _is_bf16(w_router),
         _ptr(logits, torch.float32), _ptr(topk_ids, torch.int32), _ptr(topk_w, torch.float32),
         _ptr(gate, torch.float32), _ptr(probs_out, torch.float32), n, width, n_experts, top_k,
-        (1 if norm_topk else 0) | (2 if sigmoid else 0), _ptr(offsets, torch.int32), _ptr(perm_token, torch.int32), _ptr(perm_weight, torch.float32),
+        (1 if norm_topk else 0) | (2 if sigmoid else 0) | (4 if chosen_softmax else 0), _ptr(offsets, torch.int32), _ptr(perm_token, torch.int32), _ptr(perm_weight, torch.float32),
         _ptr(inverse, torch.int32), _ptr(status, torch.int32), _ptr(distinct, torch.int64),
         _ptr(tiles[0], torch.int32) if tiles else None, _ptr(tiles[1], torch.int32) if tiles else None,
         _ptr(tiles[2], torch.int32) if tiles else None, _ptr(tiles[3], torch.int32) if tiles else None,
-        tiles[0].shape[0] if tiles else 0, pc, groups, keep, int(n_real if n_real is not None else n_experts), _stream()),
+        tiles[0].shape[0] if tiles else 0, _ptr(bias, torch.float32, "bias"), pc, groups, keep, int(n_real if n_real is not None else n_experts), _stream()),
         "route_small")
 
 
@@ -472,18 +486,21 @@ def moe_combine(expert_out, topk_ids, inverse, gate, shared, y, passing=None):
 
 
 def moe_combine_add_rmsnorm(expert_out, topk_ids, inverse, gate, shared, x, gamma, h, eps, rows=None, write_x=True,
-                            h32=None, passing=None):
+                            h32=None, passing=None, gamma_y=None, eps_y=0.0):
     """moe_combine followed by add_rmsnorm in one kernel (same operations in the same order): x (+)= combined
-    expert outputs, h = rmsnorm(x) * gamma.  Width a multiple of 4, at most 16384.  ``passing``: as for moe_combine."""
-    n_rows, width = h.shape
+    expert outputs, h = rmsnorm(x) * gamma.  Width a multiple of 4, at most 16384.  ``passing``: as for moe_combine.
+    ``gamma_y`` (with ``eps_y``): the combined row is normalised, rmsnorm(y) * gamma_y, before it is added.  ``gamma``
+    None: h = x in h's dtype; ``h`` None: the add alone."""
+    n_rows, width = h.shape if h is not None else x.shape
     pw, pi, pn = (_ptr(passing[0], torch.float32), _ptr(passing[1], torch.float32, "ident"), int(passing[2])) if passing else (None, None, 0)
     if width % 4 != 0 or width > 16384:
         raise Backend(f"moe_combine_add_rmsnorm: width {width} not taken")
     _check(_fn("core", "esp_moe_combine_add_rmsnorm")(
         _ptr(expert_out, torch.float32), _ptr(topk_ids, torch.int32), _ptr(inverse, torch.int32),
         _ptr(gate, torch.float32), _ptr(shared, torch.float32), _ptr(x, torch.float32), _ptr(gamma, torch.float32),
-        _ptr(rows, torch.int32), _ptr(h, FLOATS, "h"), _is_bf16(h), _ptr(h32, torch.float32), n_rows, width,
-        topk_ids.shape[1], float(eps), 1 if write_x else 0, pw, pi, pn, _stream()), "moe_combine_add_rmsnorm")
+        _ptr(rows, torch.int32), _ptr(h, FLOATS, "h"), _is_bf16(h) if h is not None else 0, _ptr(h32, torch.float32), n_rows,
+        width, topk_ids.shape[1], float(eps), 1 if write_x else 0, pw, pi, pn, _ptr(gamma_y, torch.float32, "gamma_y"),
+        float(eps_y), _stream()), "moe_combine_add_rmsnorm")
 
 
 def pick_tokens(logits, temperature, top_p, rng_state, row_slot, tokens):
@@ -507,9 +524,18 @@ def skinny_fits(k: int) -> bool:
     return k % 8 == 0 and 8 * (k + 32) * 2 + 8 * 512 <= SKINNY_MAX_SMEM
 
 
+def _glu_args(glu, swiglu):
+    if glu is None:
+        return 0.0, 0.0, 0.0
+    if not swiglu or not glu[0] > 0:
+        raise Backend("a unit with clamped branches is a form of the fused gate/up product and has a positive limit")
+    return tuple(float(v) for v in glu)
+
+
 def gemm_skinny(a, w, c, swiglu=False, row_scale=None, a_rows=None, group_offsets=None, rows=None, max_rows=None,
-                offsets_ready=False, xielu_pq=None, relu2=False):
-    """Weight-streaming product for few rows; bfloat16 a and w.  Plain: c[m] =
+                offsets_ready=False, xielu_pq=None, relu2=False, glu=None):
+    """``glu`` = (limit, alpha, shift), with swiglu: c[m, j] = g sigmoid(alpha g) (u + shift) instead, g = min(gate_j,
+    limit), u = clamp(up_j, -limit, limit).  Weight-streaming product for few rows; bfloat16 a and w.  Plain: c[m] =
     scale[m] * a[row(m)] @ w[g].T with w [N,K] or [G,N,K].  swiglu: w holds
     [gate rows; up rows] ([2I,K] or [G,2I,K]) and c[m, j] = silu(gate_j) * up_j
     ([rows, I]).  ``max_rows``: upper bound of the rows of one group.  ``offsets_ready``: the group offsets (and
@@ -539,7 +565,7 @@ def gemm_skinny(a, w, c, swiglu=False, row_scale=None, a_rows=None, group_offset
         a.data_ptr(), a.stride(0), _ptr(a_rows, torch.int32, "a_rows"), w.data_ptr(), wn * k,
         _ptr(row_scale, torch.float32, "row_scale"), c.data_ptr(), _is_bf16(c), c.stride(0),
         _ptr(group_offsets, torch.int32, "group_offsets"), groups, m, n, k, max_rows, 2 if relu2 else 1 if swiglu else 0,
-        1 if offsets_ready else 0, _ptr(xielu_pq, torch.float32, "xielu_pq"), _stream())
+        1 if offsets_ready else 0, _ptr(xielu_pq, torch.float32, "xielu_pq"), *_glu_args(glu, swiglu), _stream())
     _check(code, "gemm_skinny")
 
 
@@ -631,6 +657,71 @@ def attn_decode(q, k_cache, v_cache, out, part_o, part_ml, counters, tok_seq, to
         int(chunk or 0), _ptr(status, torch.int32), _stream()), "attn_decode")
 
 
+def attn_decode_diff_fits(key_dim: int, value_dim: int, page: int) -> bool:
+    """Sizes (one map's key, a value) and page size that ``attn_decode_diff`` takes."""
+    return key_dim % 8 == 0 and 0 < key_dim <= 128 and value_dim % 8 == 0 and 0 < value_dim <= 256 and page == 64
+
+
+def attn_diff_tile(dim: int) -> int:
+    """The width that the split-key kernel pads a row of ``dim`` channels to."""
+    return 64 if dim <= 64 else 128 if dim <= 128 else 256
+
+
+def attn_decode_diff(q, k_cache, v_cache, out, part_o, part_ml, counters, tok_seq, tok_pos, block_table, page, heads, nkv,
+                     key_dim, value_dim, scale, split, n_splits, status, lam, eps, out_scale, gate=None, softcap=None,
+                     window=None, chunk=None, seq_past=None):
+    """Differential attention of few token rows (bfloat16), split over the keys as ``attn_decode``, whole: scores times
+    ``scale``, then softcap tanh(s / softcap); softmax per map; per head o = a_1 - lam a_2, rmsnorm(o) * out_scale *
+    sigmoid(gate).  q [N, heads, 2, key_dim]; k_cache [pages, nkv, 64, 2 key_dim], v_cache [pages, nkv, 64, value_dim];
+    out [N, heads, value_dim]; ``gate``: float32 [N, heads], rows may be parts of wider rows.  part_o float32 [N, 2 heads,
+    n_splits, attn_diff_tile(value_dim)], part_ml float32 [N, 2 heads, n_splits, 2]."""
+    n = q.shape[0]
+    if not attn_decode_diff_fits(key_dim, value_dim, page) or not scale > 0:
+        raise Backend(f"attn_decode_diff: sizes {key_dim} / {value_dim} / page {page} not taken")
+    if split < 64 or split % 64:
+        raise Backend(f"attn_decode_diff: split {split} is not a multiple of 64")
+    if counters.numel() < n * 2 * heads or part_o.numel() < n * 2 * heads * n_splits * attn_diff_tile(value_dim) \
+            or part_ml.numel() < n * 2 * heads * n_splits * 2:
+        raise Backend("attn_decode_diff: scratch is too small")
+    gp, ldg = _rows_ld(gate, "gate")
+    _check(_fn("bf16", "esp_attn_decode_diff")(
+        _ptr(q, torch.bfloat16, "q"), _ptr(k_cache, torch.bfloat16), _ptr(v_cache, torch.bfloat16), _ptr(out, torch.bfloat16),
+        _ptr(part_o, torch.float32), _ptr(part_ml, torch.float32), _ptr(counters, torch.int32), _ptr(tok_seq, torch.int32),
+        _ptr(tok_pos, torch.int32), _ptr(seq_past, torch.int32), _ptr(block_table, torch.int32), block_table.shape[1],
+        k_cache.shape[0], page, n, heads, nkv, key_dim, value_dim, int(window or 0), split, n_splits, float(scale),
+        int(chunk or 0), float(softcap or 0.0), float(lam), float(eps), float(out_scale), gp, ldg, _ptr(status, torch.int32),
+        _stream()), "attn_decode_diff")
+
+
+def headnorm_rope_kvwrite(rows, q_w, k_w, eps, inv_freq, rot, tok_seq, tok_pos, q_out, k_cache, v_cache, block_table, page,
+                          nh, nkv, maps, hd, vd, own_kv, status):
+    """RMS norm per head and map (weights q_w, k_w of hd numbers), rotation of the first ``rot`` channels of every run by
+    position * inv_freq, and the write of keys [pages, nkv, page, maps * hd] and values [pages, nkv, page, vd] into the
+    paged cache.  rows float32 [N, >= (nh + nkv) * maps * hd + nkv * vd] (own_kv False: the queries alone, and no cache
+    write); q_out [N, nh * maps * hd]."""
+    n = q_out.shape[0]
+    need = (nh + (nkv if own_kv else 0)) * maps * hd + (nkv * vd if own_kv else 0)
+    if rows.shape[1] < need or q_out.shape[1] != nh * maps * hd:
+        raise Backend("headnorm_rope_kvwrite: the rows' width disagrees with the head counts")
+    p, ld = _rows_ld(rows, "rows")
+    _check(_fn("core", "esp_headnorm_rope_kvwrite")(
+        p, ld, _ptr(q_w, torch.float32), _ptr(k_w, torch.float32), float(eps), _ptr(inv_freq, torch.float32), int(rot),
+        _ptr(tok_seq, torch.int32), _ptr(tok_pos, torch.int32), _ptr(q_out, FLOATS, "q_out"), _ptr(k_cache, q_out.dtype),
+        _ptr(v_cache, q_out.dtype), _is_bf16(q_out), _ptr(block_table, torch.int32), block_table.shape[1], k_cache.shape[0],
+        page, n, nh, nkv, maps, hd, vd, 1 if own_kv else 0, _ptr(status, torch.int32), _stream()), "headnorm_rope_kvwrite")
+
+
+def diff_combine(a, lam, eps, out_scale, gate, y):
+    """y[n, h] = rmsnorm(a[n, 2h] - lam a[n, 2h + 1]) * out_scale * sigmoid(gate[n, h]); a float32 [N, 2H, V], y [N, H, V],
+    gate float32 [N, H] (rows may be parts of wider rows) or None."""
+    n, heads, vd = y.shape
+    if tuple(a.shape) != (n, 2 * heads, vd):
+        raise Backend("diff_combine: shapes disagree")
+    gp, ldg = _rows_ld(gate, "gate")
+    _check(_fn("core", "esp_diff_combine")(_ptr(a, torch.float32, "a"), float(lam), float(eps), float(out_scale), gp, ldg,
+                                           _ptr(y, FLOATS, "y"), _is_bf16(y), n, heads, vd, _stream()), "diff_combine")
+
+
 def attn_flash_fits(hd, vd=None, page=64) -> bool:
     """Head sizes (keys, values) and page size that ``attn_prefill`` takes."""
     vd = hd if vd is None else vd
@@ -704,8 +795,8 @@ TC05_PAIR_ROWS_PER_GROUP = 32          # grouped products with fewer rows per gr
 
 
 def gemm_tc05(a, w, c, status, swiglu=False, row_scale=None, tiles=None, rows=None, tile_rows=None, pair=None,
-              max_ctas=0):
-    """TMA + tcgen05 product for many rows.  a [rows, K] bfloat16 contiguous; w [N, K] or [G, N, K]
+              max_ctas=0, glu=None):
+    """``glu``: as for gemm_skinny.  TMA + tcgen05 product for many rows.  a [rows, K] bfloat16 contiguous; w [N, K] or [G, N, K]
     bfloat16.  Plain: c float32 [rows, N] = scale * a @ w[g].T.  swiglu: w rows are [gate; up] and c is
     bfloat16 [rows, I].  Grouped: ``tiles`` = (tile_group, tile_row0, tile_count, n_tiles) from moe_permute,
     ``tile_rows`` the most rows a tile has (128 or 256; TC05_TILE_ROWS when not given).  ``max_ctas`` > 0:
@@ -739,7 +830,7 @@ def gemm_tc05(a, w, c, status, swiglu=False, row_scale=None, tiles=None, rows=No
         _ptr(tiles[1], torch.int32) if grouped else None, _ptr(tiles[2], torch.int32) if grouped else None,
         _ptr(tiles[3], torch.int32) if grouped else None, tiles[0].shape[0] if grouped else 0,
         tile_rows if grouped else 0, m, n, k,
-        1 if swiglu else 0, 1 if pair else 0, int(max_ctas), _ptr(status, torch.int32), _stream())
+        1 if swiglu else 0, 1 if pair else 0, int(max_ctas), *_glu_args(glu, swiglu), _ptr(status, torch.int32), _stream())
     _check(code, "gemm_tc05")
 
 
@@ -939,8 +1030,8 @@ def embed_sum(table, bigram, freq, ids, tok_seq, tok_pos, seq_start, seq_slot, p
 
 
 def norm_add_rmsnorm(x, y, gamma_y, eps_y, gamma, h, eps, rows=None, write_x=True, h32=None):
-    """x (+)= rmsnorm(y) * gamma_y, then h = rmsnorm(x) * gamma, in one launch; all float32 but h.  ``h`` None: the
-    add alone.  ``x`` None: h32 = rmsnorm(y) * gamma_y and nothing else."""
+    """x (+)= rmsnorm(y) * gamma_y, then h = rmsnorm(x) * gamma, in one launch; all float32 but h.  ``gamma``
+    None: h = x in h's dtype.  ``h`` None: the add alone.  ``x`` None: h32 = rmsnorm(y) * gamma_y and nothing else."""
     width = y.shape[1]
     if x is None:
         n_rows = h32.shape[0]

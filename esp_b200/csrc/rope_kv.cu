@@ -637,3 +637,145 @@ ESP_API int esp_pair_rope_unitnorm_kvwrite(const float* qkv, const float* bias, 
 #undef ESP_PAIR_ROPE
     return esp_launch_status();
 }
+
+// ---------------------------------------------------------------- norm per head and map, split-half rotation
+// rows: float, one per token, ``ld`` numbers apart: [nh * maps * hd queries | nkv * maps * hd keys | nkv * vd values],
+// without the keys and values when ``own_kv`` is 0 (a layer that reads another's cache); what follows in a row (a
+// gate, padding) is left alone.  A head's channels are ``maps`` runs of hd.  Every run of a query (key) is divided by
+// its root mean square over hd (eps inside the root) and multiplied by q_w (k_w), hd numbers that all heads and maps
+// share (null: no norm for that side); then its first ``rot`` channels are rotated, channel i with channel i + rot/2,
+// by the angle position * inv_freq[i] (a 32-bit product; sine and cosine in 32-bit).  Queries go to q_out
+// [n_tokens, nh, maps * hd], keys [pages, nkv, PAGE, maps * hd] and values [pages, nkv, PAGE, vd] to the token's place
+// in the paged cache.  One block per token; a row's queries and keys are staged in shared memory.
+// VEC 4: sizes are whole pieces of four channels and the buffers aligned to them; VEC 1: any sizes.  Which form runs
+// depends on the sizes and the alignment alone.  Dynamic shared memory: (staged channels + rotated runs + rot) floats.
+template <typename T, int VEC>
+__global__ void __launch_bounds__(256)
+headnorm_rope_kvwrite_kernel(const float* __restrict__ rows, long long ld, const float* __restrict__ q_w,
+                             const float* __restrict__ k_w, float eps, const float* __restrict__ inv_freq, int rot,
+                             const int* __restrict__ tok_seq, const int* __restrict__ tok_pos, T* __restrict__ q_out,
+                             T* __restrict__ k_cache, T* __restrict__ v_cache, const int* __restrict__ block_table,
+                             int table_stride, int n_pages, int page, int nh, int nkv, int maps, int hd, int vd, int own_kv,
+                             int* __restrict__ status) {
+    pdl_trigger();
+    extern __shared__ __align__(16) float head_smem[];
+    const int n = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nwarp = blockDim.x >> 5;
+    const int q_runs = nh * maps, runs = q_runs + (own_kv ? nkv * maps : 0), chans = runs * hd, half = rot / 2;
+    float* row = head_smem;                 // [chans]
+    float* inv = row + chans;               // [runs] reciprocal root mean squares
+    float* cs = inv + runs;                 // [half] cosines, then [half] sines of this row's angles
+    pdl_wait();
+    const int pos = tok_pos[n], seq = tok_seq[n];
+    const float p = (float)pos;
+    for (int c = tid; c < half; c += blockDim.x) sincosf(p * inv_freq[c], &cs[half + c], &cs[c]);
+    int page_id = -1;
+    if (own_kv) {
+        page_id = block_table[(size_t)seq * table_stride + pos / page];
+        if (page_id < 0 || page_id >= n_pages) {
+            if (tid == 0) atomicOr(status, ESP_STATUS_BAD_INDEX);
+            page_id = -1;
+        }
+    }
+    const int in_page = pos % page;
+    const float* src = rows + (size_t)n * ld;
+    for (int e = VEC * tid; e < chans; e += VEC * blockDim.x) {
+        if (VEC == 4) *reinterpret_cast<float4*>(row + e) = *reinterpret_cast<const float4*>(src + e);
+        else row[e] = src[e];
+    }
+    __syncthreads();
+    for (int r = warp; r < runs; r += nwarp) {
+        float ss = 0.f;
+        for (int c = lane; c < hd; c += 32) ss = fmaf(row[r * hd + c], row[r * hd + c], ss);
+        ss = warp_sum(ss);
+        if (lane == 0) inv[r] = (r < q_runs ? q_w : k_w) ? 1.0f / sqrtf(ss / (float)hd + eps) : 1.0f;
+    }
+    __syncthreads();
+    for (int e = VEC * tid; e < chans; e += VEC * blockDim.x) {
+        const int r = e / hd, c = e - r * hd;
+        if (c >= half && c < rot) continue;                 // the second channel of a pair is written with the first
+        const bool is_q = r < q_runs;
+        const float* w = is_q ? q_w : k_w;
+        T* dst;
+        if (is_q) {
+            dst = q_out + ((size_t)n * q_runs + r) * hd;
+        } else if (page_id >= 0) {
+            const int kr = r - q_runs, head = kr / maps, m = kr - head * maps;
+            dst = k_cache + (((size_t)page_id * nkv + head) * page + in_page) * (maps * hd) + m * hd;
+        } else {
+            continue;
+        }
+        const float f = inv[r];
+        float a[VEC], b[VEC];
+#pragma unroll
+        for (int i = 0; i < VEC; i++) a[i] = w ? row[e + i] * f * w[c + i] : row[e + i];
+        if (c < half) {
+            float lo[VEC], hi[VEC];
+#pragma unroll
+            for (int i = 0; i < VEC; i++) {
+                b[i] = w ? row[e + half + i] * f * w[c + half + i] : row[e + half + i];
+                const float co = cs[c + i], si = cs[half + c + i];
+                lo[i] = a[i] * co - b[i] * si;
+                hi[i] = b[i] * co + a[i] * si;
+            }
+            if constexpr (VEC == 4) {
+                Vec4<T>::store(dst + c, lo[0], lo[1], lo[2], lo[3]);
+                Vec4<T>::store(dst + c + half, hi[0], hi[1], hi[2], hi[3]);
+            } else {
+                dst[c] = from_f32<T>(lo[0]);
+                dst[c + half] = from_f32<T>(hi[0]);
+            }
+        } else {
+            if constexpr (VEC == 4) Vec4<T>::store(dst + c, a[0], a[1], a[2], a[3]);
+            else dst[c] = from_f32<T>(a[0]);
+        }
+    }
+    if (page_id >= 0) {
+        for (int e = VEC * tid; e < nkv * vd; e += VEC * blockDim.x) {
+            const int head = e / vd, c = e - head * vd;
+            T* dst = v_cache + (((size_t)page_id * nkv + head) * page + in_page) * vd + c;
+            if constexpr (VEC == 4) {
+                const float4 v = *reinterpret_cast<const float4*>(src + chans + e);
+                Vec4<T>::store(dst, v.x, v.y, v.z, v.w);
+            } else {
+                *dst = from_f32<T>(src[chans + e]);
+            }
+        }
+    }
+}
+
+ESP_API int esp_headnorm_rope_kvwrite(const float* rows, long long ld, const float* q_w, const float* k_w, float eps,
+                                      const float* inv_freq, int rot, const int* tok_seq, const int* tok_pos, void* q_out,
+                                      void* k_cache, void* v_cache, int is_bf16, const int* block_table, int table_stride,
+                                      int n_pages, int page, int n_tokens, int nh, int nkv, int maps, int hd, int vd,
+                                      int own_kv, int* status, cudaStream_t stream) {
+    if (n_tokens <= 0) return 0;
+    if (hd <= 0 || vd <= 0 || nkv <= 0 || nh <= 0 || maps <= 0 || page <= 0 || rot < 0 || rot > hd || rot % 2 != 0 ||
+        (rot > 0 && !inv_freq))
+        return (int)cudaErrorInvalidValue;
+    const long long runs = (long long)(nh + (own_kv ? nkv : 0)) * maps;
+    const size_t smem = (size_t)(runs * hd + runs + rot) * sizeof(float);
+    if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
+    const size_t ptrs = (size_t)rows | (size_t)q_w | (size_t)k_w | (size_t)q_out | (size_t)k_cache | (size_t)v_cache;
+    const bool vec = hd % 4 == 0 && vd % 4 == 0 && rot % 8 == 0 && ld % 4 == 0 && (ptrs & 15) == 0;
+    const int threads = runs * hd >= 1024 ? 256 : 128;
+#define ESP_HEADNORM(T, VEC)                                                                                              \
+    do {                                                                                                                  \
+        if (smem > 48 * 1024) {                                                                                           \
+            cudaError_t e = cudaFuncSetAttribute(headnorm_rope_kvwrite_kernel<T, VEC>,                                     \
+                                                 cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);                  \
+            if (e != cudaSuccess) return (int)e;                                                                          \
+        }                                                                                                                 \
+        esp_launch_pdl(ESP_PDL_SMALL, headnorm_rope_kvwrite_kernel<T, VEC>, dim3(n_tokens), dim3(threads), smem, stream,    \
+                       rows, ld, q_w, k_w, eps, inv_freq, rot, tok_seq, tok_pos, (T*)q_out, (T*)k_cache, (T*)v_cache,       \
+                       block_table, table_stride, n_pages, page, nh, nkv, maps, hd, vd, own_kv, status);                   \
+    } while (0)
+    if (is_bf16) {
+        if (vec) ESP_HEADNORM(bf16, 4);
+        else ESP_HEADNORM(bf16, 1);
+    } else {
+        if (vec) ESP_HEADNORM(float, 4);
+        else ESP_HEADNORM(float, 1);
+    }
+#undef ESP_HEADNORM
+    return esp_launch_status();
+}

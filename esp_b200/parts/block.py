@@ -159,6 +159,55 @@ class SandwichBlock(Part):
         return pending
 
 
+class OutputNormBlock(Part):
+    """x += norm1(mixer(x)); x += norm2(ffn(x)): the sublayers read the residual stream as it is (rounded to the
+    activation dtype; a part with ``wants_f32_input`` gets x itself besides) and only their results are normalised.  A
+    result travels as a ``DeferredPostNorm`` until its reader adds it: this block or the next one, which take x in the
+    activation dtype in the same launch, or the model's last norm."""
+
+    graph_safe = True
+
+    def __init__(self, spec, rt):
+        self.spec, self.rt = spec, rt
+        self.mixer = build("mixer", spec.mixer, rt)
+        self.mixer_post = build("norm", spec.mixer_post_norm, rt)
+        self.ffn = build("ffn", spec.ffn, rt)
+        self.ffn_post = build("norm", spec.ffn_post_norm, rt)
+
+    def children(self):
+        return [p for p in (self.mixer, self.mixer_post, self.ffn, self.ffn_post) if p is not None]
+
+    def _read(self, x, pending):
+        """x with ``pending`` added, in the activation dtype (x itself in the 32-bit engine: a sublayer has read its
+        input by the time its own result is added)."""
+        rt = self.rt
+        h = x if rt.dtype == torch.float32 else rt.ws.get("block_h", tuple(x.shape), rt.dtype)
+        if isinstance(pending, DeferredPostNorm):
+            pending.add_to(x, None if h is x else h)
+            return h
+        pending = plain_delta(None, pending)
+        if pending is not None:
+            x.add_(pending)
+        if h is not x:
+            ops.cast_cols(x, h)
+        return h
+
+    def forward(self, x, pending, ctx, layer):
+        rt = self.rt
+        h = self._read(x, pending)
+        pending = DeferredPostNorm(rt, self.mixer.forward(h, ctx, layer), self.mixer_post)
+        if self.ffn is not None:
+            h = self._read(x, pending)
+            h32 = x if getattr(self.ffn, "wants_f32_input", False) and h is not x else None
+            pending = DeferredPostNorm(rt, self.ffn.forward(h, ctx, h32=h32), self.ffn_post)
+        if "residual_trace" in ctx.aux:
+            # debugging aid (see ScaledDepthMixBlock._trace): the add is done here so that x is the layer's result
+            pending.add_to(x)
+            ctx.aux["residual_trace"].append(x.clone())
+            return None
+        return pending
+
+
 class DeferredStreamWrite:
     """The write of a sublayer into the copies of the residual stream, on its way to whoever reads them next: the
     next layer's first read, or the model's last norm (which then sees the sum of the copies).  Either does the
@@ -266,4 +315,5 @@ class HyperConnectionBlock(Part):
 register("block", "prenorm_residual", PreNormResidualBlock)
 register("block", "hyper_connections", HyperConnectionBlock)
 register("block", "sandwich_residual", SandwichBlock)
+register("block", "output_norm_residual", OutputNormBlock)
 register("block", "prenorm_scaled_depthmix", ScaledDepthMixBlock)

@@ -25,9 +25,11 @@ class DeferredMoeCombine:
         ops.moe_combine(self.expert_out, self.ids, self.inverse, self.gate, self.shared, y, passing=self.passing)
         return y
 
-    def fused_add_rmsnorm(self, x, gamma, h, eps, rows, write_x, h32):
+    def fused_add_rmsnorm(self, x, gamma, h, eps, rows, write_x, h32, post=None):
+        """``post`` = (weight, eps): the combined rows are normalised before they are added."""
         ops.moe_combine_add_rmsnorm(self.expert_out, self.ids, self.inverse, self.gate, self.shared, x, gamma, h, eps,
-                                    rows=rows, write_x=write_x, h32=h32, passing=self.passing)
+                                    rows=rows, write_x=write_x, h32=h32, passing=self.passing,
+                                    gamma_y=post[0] if post else None, eps_y=post[1] if post else 0.0)
 
 
 # Steps with at least AHEAD_ROWS rows start the shared expert's first product on a second stream before the
@@ -41,12 +43,12 @@ ROUTING_SMS = 8
 SIDE_STREAM_ROWS = 64      # steps with at most this many rows run the shared expert on a second stream
 
 
-def _swiglu_mlp(rt, h, w_gate_up, w_down, out, tag):
-    """out = down(silu(gate h) * (up h)); w_gate_up is [2I, H], gate rows first."""
+def _swiglu_mlp(rt, h, w_gate_up, w_down, out, tag, glu=None):
+    """out = down(silu(gate h) * (up h)); w_gate_up is [2I, H], gate rows first.  ``glu``: see ``swiglu_linear``."""
     n = h.shape[0]
     inter = w_gate_up.shape[0] // 2
     act = rt.ws.get(tag + "_act", (n, inter), rt.dtype)
-    swiglu_linear(rt, h, w_gate_up, act, tag)
+    swiglu_linear(rt, h, w_gate_up, act, tag, glu=glu)
     linear(rt, act, w_down, out)
     return out
 
@@ -176,7 +178,8 @@ class MoeSwiGluShared(Part):
     SwiGLU expert scaled by sigmoid(h . w_shared_gate)
     (crates/esp/src/infer/decoder/moe.rs:135-256).  Options of the spec: router outputs without an expert behind
     them (a chosen one returns the block's input times its weight), a correction per output that counts for the
-    choice only, a choice limited to the best groups of neighbouring outputs, no shared expert."""
+    choice only, a choice limited to the best groups of neighbouring outputs, a bias on the logits, weights that are a
+    softmax over the chosen logits alone, gated units with clamped branches, no shared expert or one without a gate."""
 
     graph_safe = True
 
@@ -190,7 +193,7 @@ class MoeSwiGluShared(Part):
                                                    f"outputs; the groups are equal and at most 32")
             if spec.keep_groups * (self.n_outputs // spec.groups) < spec.top_k:
                 raise Unsupported("router.groups", "the kept groups hold fewer experts than are chosen")
-        self.correction = None
+        self.correction = self.router_bias = None
         self.w_router = self.w_shared_gate = None
         self.w_gate_up = self.w_down = None            # [E, 2Im, H], [E, H, Im]
         self.w_shared_gate_up = self.w_shared_down = None
@@ -201,7 +204,7 @@ class MoeSwiGluShared(Part):
         """(router, shared gate, shared (gate, up, down), [per expert (gate, up, down)])"""
         s, p, n = self.spec, self.spec.prefix, self.spec.names
         mlp = lambda q: (q + n.mlp.gate, q + n.mlp.up, q + n.mlp.down)
-        return (p + n.router, p + n.shared_gate, mlp(p + n.shared),
+        return (p + n.router, p + n.shared_gate if n.shared_gate is not None else None, mlp(p + n.shared),
                 [mlp(p + n.expert.format(e=e)) for e in range(s.num_experts)])
 
     def param_specs(self):
@@ -209,10 +212,13 @@ class MoeSwiGluShared(Part):
         router, shared_gate, shared, experts = self._names()
         specs = [ParamSpec(router, (self.n_outputs, s.hidden), "matrix")]
         if s.shared_intermediate is not None:
-            specs += [ParamSpec(shared_gate, (1, s.hidden), "matrix"),
-                      ParamSpec(shared[0], (s.shared_intermediate, s.hidden), "matrix"),
+            if shared_gate is not None:
+                specs.append(ParamSpec(shared_gate, (1, s.hidden), "matrix"))
+            specs += [ParamSpec(shared[0], (s.shared_intermediate, s.hidden), "matrix"),
                       ParamSpec(shared[1], (s.shared_intermediate, s.hidden), "matrix"),
                       ParamSpec(shared[2], (s.hidden, s.shared_intermediate), "matrix")]
+        if s.router_bias is not None:
+            specs.append(ParamSpec(s.prefix + s.router_bias, (self.n_outputs,), "router_bias", init=(0.0, 0.1)))
         if s.correction is not None:
             specs.append(ParamSpec(s.prefix + s.correction, (self.n_outputs,), "router_correction", init=(0.0, 0.02)))
         for gate, up, down in experts:
@@ -227,22 +233,27 @@ class MoeSwiGluShared(Part):
         E, Im, Is, H = s.num_experts, s.expert_intermediate, s.shared_intermediate, s.hidden
         router, shared_gate, shared, experts = self._names()
         has_shared = Is is not None
-        rdt = rt.matrix_dtype([stored[router]] + ([stored[shared_gate]] if has_shared else []))
+        rdt = rt.matrix_dtype([stored[router]] + ([stored[shared_gate]] if has_shared and shared_gate is not None else []))
         self.w_router = torch.empty((self.n_outputs, H), dtype=rdt, device=dev)
         gu_dt = rt.matrix_dtype([stored[n] for g, u, _d in experts for n in (g, u)])
         self.w_gate_up = torch.empty((E, 2 * Im, H), dtype=gu_dt, device=dev)
         self.w_down = torch.empty((E, H, Im), dtype=rt.matrix_dtype([stored[d] for _g, _u, d in experts]), device=dev)
         views = {router: self.w_router}
         if has_shared:
-            self.w_shared_gate = torch.empty((1, H), dtype=rdt, device=dev)
+            if shared_gate is not None:
+                self.w_shared_gate = torch.empty((1, H), dtype=rdt, device=dev)
+                views[shared_gate] = self.w_shared_gate
             sdt = rt.matrix_dtype([stored[shared[0]], stored[shared[1]]])
             self.w_shared_gate_up = torch.empty((2 * Is, H), dtype=sdt, device=dev)
             self.w_shared_down = torch.empty((H, Is), dtype=rt.matrix_dtype([stored[shared[2]]]), device=dev)
-            views.update({shared_gate: self.w_shared_gate, shared[0]: self.w_shared_gate_up[:Is],
-                          shared[1]: self.w_shared_gate_up[Is:], shared[2]: self.w_shared_down})
+            views.update({shared[0]: self.w_shared_gate_up[:Is], shared[1]: self.w_shared_gate_up[Is:],
+                          shared[2]: self.w_shared_down})
         if s.correction is not None:
             self.correction = torch.empty(self.n_outputs, dtype=torch.float32, device=dev)
             views[s.prefix + s.correction] = self.correction
+        if s.router_bias is not None:
+            self.router_bias = torch.empty(self.n_outputs, dtype=torch.float32, device=dev)
+            views[s.prefix + s.router_bias] = self.router_bias
         for e, (gate, up, down) in enumerate(experts):
             views[gate] = self.w_gate_up[e, :Im]
             views[up] = self.w_gate_up[e, Im:]
@@ -273,7 +284,7 @@ class MoeSwiGluShared(Part):
         ws = rt.ws
         ids = ws.get("moe_ids", (n, k), torch.int32)
         wts = ws.get("moe_w", (n, k), torch.float32)
-        gate = ws.get("moe_gate", (n,), torch.float32) if has_shared else None
+        gate = ws.get("moe_gate", (n,), torch.float32) if self.w_shared_gate is not None else None
         probs = None
         if rt.record_routing:
             probs = torch.empty((n, R), dtype=torch.float32, device=rt.device)
@@ -298,14 +309,15 @@ class MoeSwiGluShared(Part):
             rt.side_stream.wait_stream(main)
             act_s = ws.get("moe_shared_act", (n, s.shared_intermediate), rt.dtype)
             with torch.cuda.stream(rt.side_stream):
-                swiglu_linear(rt, h, self.w_shared_gate_up, act_s, "moe_shared", max_ctas=max(2, rt.sm_count - ROUTING_SMS))
+                swiglu_linear(rt, h, self.w_shared_gate_up, act_s, "moe_shared", max_ctas=max(2, rt.sm_count - ROUTING_SMS),
+                              glu=s.shared_glu)
         if beside:
             # few rows: the shared expert depends neither on the router nor on the routing, so it runs beside
             # them and the routed experts on a second stream (in a captured step: a parallel branch of the graph)
             main = torch.cuda.current_stream()
             rt.side_stream.wait_stream(main)
             with torch.cuda.stream(rt.side_stream):
-                _swiglu_mlp(rt, h, self.w_shared_gate_up, self.w_shared_down, shared, "moe_shared")
+                _swiglu_mlp(rt, h, self.w_shared_gate_up, self.w_shared_down, shared, "moe_shared", glu=s.shared_glu)
         uses_tc05 = grouped_uses_tc05(h, self.w_gate_up, n * k, n) and Im % 8 == 0
         if uses_tc05 and R > E:
             perm_token.zero_()                   # the gather reads n * k rows; those behind the last expert's are never placed
@@ -320,10 +332,11 @@ class MoeSwiGluShared(Part):
             logits = ws.get("moe_logits", (n, R + 1), torch.float32)
             ops.route_small(router_in, self.w_router, self.w_shared_gate, logits, ids, wts, gate, k, s.norm_topk,
                             offsets, perm_token, perm_weight, inverse, rt.status, probs, distinct=self.expert_reads,
-                            tiles=tiles, choice=choice, n_real=E)
+                            tiles=tiles, choice=choice, n_real=E, bias=self.router_bias, chosen_softmax=s.chosen_softmax)
         else:
             ops.router_topk(router_in, self.w_router, self.w_shared_gate, ids, wts, gate, k, s.norm_topk, rt.status,
-                            probs, logits=ws.get("moe_logits", (n, R + 1), torch.float32), choice=choice)
+                            probs, logits=ws.get("moe_logits", (n, R + 1), torch.float32), choice=choice, bias=self.router_bias,
+                            chosen_softmax=s.chosen_softmax)
             ops.moe_permute(ids, wts, E, offsets, perm_token, perm_weight, inverse, rt.status, tiles=tiles,
                             distinct=self.expert_reads, n_ids=R)
         if rt.record_routing:
@@ -336,7 +349,7 @@ class MoeSwiGluShared(Part):
         elif ahead:
             linear(rt, act_s, self.w_shared_down, shared)
         elif has_shared:
-            _swiglu_mlp(rt, h, self.w_shared_gate_up, self.w_shared_down, shared, "moe_shared")
+            _swiglu_mlp(rt, h, self.w_shared_gate_up, self.w_shared_down, shared, "moe_shared", glu=s.shared_glu)
         if y is None:
             return DeferredMoeCombine(rt, expert_out, ids, inverse, gate, shared, H, passing)
         ops.moe_combine(expert_out, ids, inverse, gate, shared, y, passing=passing)
@@ -348,7 +361,7 @@ class MoeSwiGluShared(Part):
         ``max_rows``: no expert has more rows than this (a token names an expert once)."""
         s, rt = self.spec, self.rt
         act = rt.ws.get("moe_act", (rows, s.expert_intermediate), rt.dtype)
-        grouped_swiglu_linear(rt, h, self.w_gate_up, act, offsets, perm_token, rows, max_rows, "moe", tiles)
+        grouped_swiglu_linear(rt, h, self.w_gate_up, act, offsets, perm_token, rows, max_rows, "moe", tiles, glu=s.glu)
         out = rt.ws.get("moe_expert_out", (rows, s.hidden), torch.float32)
         # the routing was complete before the first product started: the second may look its groups up and ask for
         # its weights while the first still runs.  Only for few rows, where the first product is one wave of
@@ -483,7 +496,7 @@ class ScaledInputMoe(Part):
             main = torch.cuda.current_stream()
             rt.side_stream.wait_stream(main)
             with torch.cuda.stream(rt.side_stream):
-                _relu2_mlp(rt, h, self.w_shared_up, self.w_shared_down, shared, "moe_shared")
+                _relu2_mlp(rt, h, self.w_shared_up, self.w_shared_down, shared, "moe_shared", glu=s.shared_glu)
         if n <= ops.ROUTE_SMALL_TOKENS and ops.route_small_fits(H, E):
             logits = ws.get("moe_logits", (n, E + 1), torch.float32)
             ops.route_small(router_in, self.w_router, None, logits, ids, wts, None, k, False, offsets, perm_token, perm_weight,
@@ -520,7 +533,7 @@ class ScaledInputMoe(Part):
                 main.wait_stream(rt.side_stream)
             else:
                 shared = ws.get("moe_shared_out", (n, H), torch.float32)
-                _relu2_mlp(rt, h, self.w_shared_up, self.w_shared_down, shared, "moe_shared")
+                _relu2_mlp(rt, h, self.w_shared_up, self.w_shared_down, shared, "moe_shared", glu=s.shared_glu)
         ops.moe_combine(out, ids, inverse, None, shared, y)
         return y
 

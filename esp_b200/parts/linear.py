@@ -47,21 +47,29 @@ def linear(rt, a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Ten
     return out
 
 
-def swiglu_linear(rt, a, w_gate_up, act, tag, max_ctas=0):
+def _gated_unit(gu, act, glu):
+    if glu is None:
+        ops.swiglu(gu, act)
+    else:
+        ops.glu_clamped(gu, act, *glu)
+
+
+def swiglu_linear(rt, a, w_gate_up, act, tag, max_ctas=0, glu=None):
     """act = silu(a @ w_gate.T) * (a @ w_up.T) in the activation dtype; w_gate_up
-    is [2I, K] with the gate rows first.  ``max_ctas`` > 0 bounds the SMs that the
+    is [2I, K] with the gate rows first.  ``glu`` = (limit, alpha, shift): the unit with clamped branches instead,
+    g sigmoid(alpha g) (u + shift) with g = min(gate, limit) and u = clamp(up, -limit, limit).  ``max_ctas`` > 0 bounds the SMs that the
     many-row kernel takes."""
     n = a.shape[0]
     inter = w_gate_up.shape[0] // 2
     if _both_bf16(a, w_gate_up) and n <= SKINNY_ROWS and ops.skinny_fits(a.shape[1]):
-        ops.gemm_skinny(a, w_gate_up, act, swiglu=True)
+        ops.gemm_skinny(a, w_gate_up, act, swiglu=True, glu=glu)
         return act
     if _both_bf16(a, w_gate_up) and DENSE_GEMM in ("own", "mixed") and a.shape[1] % 8 == 0 and a.is_contiguous() and act.is_contiguous():
-        ops.gemm_tc05(a, w_gate_up, act, rt.status, swiglu=True, max_ctas=max_ctas)
+        ops.gemm_tc05(a, w_gate_up, act, rt.status, swiglu=True, max_ctas=max_ctas, glu=glu)
         return act
     gu = rt.ws.get(tag + "_gu", (n, 2 * inter), torch.float32)
     linear(rt, a, w_gate_up, gu)
-    ops.swiglu(gu, act)
+    _gated_unit(gu, act, glu)
     return act
 
 
@@ -99,7 +107,7 @@ def grouped_uses_tc05(a, w, rows, max_rows=None) -> bool:
     return _both_bf16(a, w) and many and a.shape[1] % 8 == 0 and w.shape[1] % 16 == 0
 
 
-def grouped_swiglu_linear(rt, a, w_gate_up, act, group_offsets, a_rows, rows, max_rows, tag, tiles=None):
+def grouped_swiglu_linear(rt, a, w_gate_up, act, group_offsets, a_rows, rows, max_rows, tag, tiles=None, glu=None):
     """Grouped form of swiglu_linear: permuted row r reads a[a_rows[r]] and the
     weights of the group whose range holds r (w_gate_up [G, 2I, K]).  With
     ``tiles`` (the row-tile list of the permutation) the rows are gathered
@@ -107,16 +115,16 @@ def grouped_swiglu_linear(rt, a, w_gate_up, act, group_offsets, a_rows, rows, ma
     if tiles is not None:
         gathered = rt.ws.get(tag + "_gathered", (rows, a.shape[1]), torch.bfloat16)
         ops.gather_rows(a, a_rows, gathered)
-        ops.gemm_tc05(gathered, w_gate_up, act, rt.status, swiglu=True, tiles=tiles)
+        ops.gemm_tc05(gathered, w_gate_up, act, rt.status, swiglu=True, tiles=tiles, glu=glu)
         return act
     if _both_bf16(a, w_gate_up) and ops.skinny_fits(a.shape[1]):
         ops.gemm_skinny(a, w_gate_up, act, swiglu=True, a_rows=a_rows, group_offsets=group_offsets, rows=rows,
-                        max_rows=max_rows)
+                        max_rows=max_rows, glu=glu)
         return act
     inter = w_gate_up.shape[1] // 2
     gu = rt.ws.get(tag + "_gu", (rows, 2 * inter), torch.float32)
     ops.gemm_simt(a, w_gate_up, gu, a_rows=a_rows, group_offsets=group_offsets, rows=rows)
-    ops.swiglu(gu, act)
+    _gated_unit(gu, act, glu)
     return act
 
 

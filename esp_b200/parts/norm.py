@@ -78,20 +78,31 @@ class DeferredPostNorm:
     normed rows from ``materialize()``."""
 
     def __init__(self, rt, y, norm):
+        """``y``: float32 rows, or a deferred output that can fold the norm into its own last step."""
         self.rt, self.y, self.norm = rt, y, norm
 
+    def _plain(self):
+        if hasattr(self.y, "materialize"):
+            self.y = self.y.materialize()
+        return self.y
+
     def materialize(self):
-        out = self.rt.ws.get("post_normed", tuple(self.y.shape), torch.float32)
-        ops.norm_add_rmsnorm(None, self.y, self.norm.weight, self.norm.spec.eps, None, None, 0.0, h32=out)
+        y = self._plain()
+        out = self.rt.ws.get("post_normed", tuple(y.shape), torch.float32)
+        ops.norm_add_rmsnorm(None, y, self.norm.weight, self.norm.spec.eps, None, None, 0.0, h32=out)
         return out
 
     def fused_add_rmsnorm(self, x, gamma, h, eps, rows, write_x, h32):
+        """x (+)= norm(y), then h = rmsnorm(x) * gamma (``gamma`` None: h = x in h's dtype; ``h`` None: the add alone)."""
+        if hasattr(self.y, "materialize"):
+            self.y.fused_add_rmsnorm(x, gamma, h, eps, rows, write_x, h32, post=(self.norm.weight, self.norm.spec.eps))
+            return
         ops.norm_add_rmsnorm(x, self.y, self.norm.weight, self.norm.spec.eps, gamma, h, eps, rows=rows, write_x=write_x,
                              h32=h32)
 
-    def add_to(self, x):
-        """x += norm(y), nothing else."""
-        ops.norm_add_rmsnorm(x, self.y, self.norm.weight, self.norm.spec.eps, None, None, 0.0)
+    def add_to(self, x, h=None):
+        """x += norm(y); ``h`` (optional) receives x in its dtype."""
+        self.fused_add_rmsnorm(x, None, h, 0.0, None, True, None)
 
 
 register("norm", "rmsnorm", RmsNorm)
