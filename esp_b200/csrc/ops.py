@@ -100,6 +100,8 @@ _SIGNATURES = {
                               c_int, P, c_int, c_int, P, P],
     "esp_attn_decode": [P, P, P, P, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                         c_int, c_float, c_int, P, c_int, P, P],
+    "esp_attn_diff_tc05": [P, c_longlong, P, P, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
+                           c_float, c_int, c_float, c_float, c_float, P, c_longlong, P, P],
     "esp_attn_decode_diff": [P, P, P, P, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
                              c_int, c_int, c_float, c_int, c_float, c_float, c_float, c_float, P, c_longlong, P, P],
 }
@@ -691,6 +693,35 @@ def attn_decode_diff(q, k_cache, v_cache, out, part_o, part_ml, counters, tok_se
         k_cache.shape[0], page, n, heads, nkv, key_dim, value_dim, int(window or 0), split, n_splits, float(scale),
         int(chunk or 0), float(softcap or 0.0), float(lam), float(eps), float(out_scale), gp, ldg, _ptr(status, torch.int32),
         _stream()), "attn_decode_diff")
+
+
+def attn_diff_tc05_fits(key_dim: int, value_dim: int, page: int) -> bool:
+    """Sizes (one map's key, a value) and page size that ``attn_diff_tc05`` takes."""
+    return key_dim % 8 == 0 and 0 < key_dim <= 128 and value_dim % 8 == 0 and 0 < value_dim <= 256 and page == 64
+
+
+ATTN_DIFF_FUSED_VALUES = 128       # values of up to this many channels: attn_diff_tc05 makes the difference, norm and gate itself
+
+
+def attn_diff_tc05(q, k_cache, v_cache, out, maps_out, tile_seq, tile_first, seq_start, seq_past, block_table, page, heads, nkv,
+                   key_dim, value_dim, scale, status, lam, eps, out_scale, gate=None, softcap=None, chunk=None):
+    """Differential attention of runs of new tokens on tcgen05 (bfloat16); the arguments of ``attn_decode_diff`` with the
+    tiles of ``attn_prefill_tc05``.  Values of more than ATTN_DIFF_FUSED_VALUES channels: the maps' outputs are left in
+    ``maps_out`` (float32 [N, 2 heads, value_dim]) for ``diff_combine``, and ``out`` is not written."""
+    if not attn_diff_tc05_fits(key_dim, value_dim, page) or not scale > 0:
+        raise Backend(f"attn_diff_tc05: sizes {key_dim} / {value_dim} / page {page} not taken")
+    n = q.shape[0]
+    if q.numel() != n * heads * 2 * key_dim:
+        raise Backend("attn_diff_tc05 takes queries [tokens, heads, 2, key_dim]")
+    if value_dim > ATTN_DIFF_FUSED_VALUES and (maps_out is None or maps_out.numel() < n * 2 * heads * value_dim):
+        raise Backend("attn_diff_tc05: values this wide need room for the maps' outputs")
+    gp, ldg = _rows_ld(gate, "gate")
+    _check(_fn("tc05", "esp_attn_diff_tc05")(
+        _ptr(q, torch.bfloat16, "q"), n, _ptr(k_cache, torch.bfloat16), _ptr(v_cache, torch.bfloat16), _ptr(out, torch.bfloat16),
+        _ptr(maps_out, torch.float32), _ptr(tile_seq, torch.int32), _ptr(tile_first, torch.int32), _ptr(seq_start, torch.int32),
+        _ptr(seq_past, torch.int32), _ptr(block_table, torch.int32), block_table.shape[1], k_cache.shape[0], page,
+        tile_seq.shape[0], heads, nkv, key_dim, value_dim, float(scale), float(softcap or 0.0), int(chunk or 0), float(lam),
+        float(eps), float(out_scale), gp, ldg, _ptr(status, torch.int32), _stream()), "attn_diff_tc05")
 
 
 def headnorm_rope_kvwrite(rows, q_w, k_w, eps, inv_freq, rot, tok_seq, tok_pos, q_out, k_cache, v_cache, block_table, page,

@@ -117,6 +117,8 @@ class DifferentialAttention(Part):
         if self.rt.dtype == torch.bfloat16:
             if n <= DECODE_ROWS and ops.attn_decode_diff_fits(s.key_dim, s.value_dim, page):
                 return "split"         # few rows: the keys are split over blocks
+            if ops.attn_diff_tc05_fits(s.key_dim, s.value_dim, page):
+                return "tc05"          # many rows: both maps' scores and weighted values in tensor memory
         return "plain"
 
     def step_arrays_key(self):
@@ -168,10 +170,22 @@ class DifferentialAttention(Part):
                                  rt.status, self.lam, s.eps, out_scale, gate=gate, softcap=s.softcap, chunk=s.chunk,
                                  seq_past=ctx.seq_past if layer.writes else None)
             return
-        maps = rt.ws.get("diff_maps", (n, 2 * s.num_heads, s.value_dim), torch.float32)
-        ops.attn_simt(q, layer.k, layer.v, maps, ctx.tok_seq, ctx.tok_pos, table, layer.page, 2 * s.num_heads, s.num_kv_heads,
-                      s.key_dim, None, rt.status, vd=s.value_dim, scale=s.scale,
-                      chunk=s.chunk, softcap=s.softcap, maps=2)
+        tile_seq = None
+        if kind == "tc05":
+            rows = ops.ATTN_TC05_TILE_ROWS
+            tile_seq, tile_first = ctx.arrays.get(f"attention.tiles{rows}.seq"), ctx.arrays.get(f"attention.tiles{rows}.first")
+        fused = tile_seq is not None and s.value_dim <= ops.ATTN_DIFF_FUSED_VALUES
+        maps = None if fused else rt.ws.get("diff_maps", (n, 2 * s.num_heads, s.value_dim), torch.float32)
+        if tile_seq is not None:
+            ops.attn_diff_tc05(q, layer.k, layer.v, o if fused else None, maps, tile_seq, tile_first, ctx.seq_start, ctx.seq_past,
+                               table, layer.page, s.num_heads, s.num_kv_heads, s.key_dim, s.value_dim, s.scale, rt.status,
+                               self.lam, s.eps, out_scale, gate=gate, softcap=s.softcap, chunk=s.chunk)
+            if fused:
+                return
+        else:                              # (a step made without this part's lists takes the plain kernel as well)
+            ops.attn_simt(q, layer.k, layer.v, maps, ctx.tok_seq, ctx.tok_pos, table, layer.page, 2 * s.num_heads,
+                          s.num_kv_heads, s.key_dim, None, rt.status, vd=s.value_dim, scale=s.scale, chunk=s.chunk,
+                          softcap=s.softcap, maps=2)
         ops.diff_combine(maps, self.lam, s.eps, out_scale, gate, o.view(n, s.num_heads, s.value_dim))
 
 

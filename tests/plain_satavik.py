@@ -193,7 +193,7 @@ def random_weights(cfg, seed, gain=1.0):
         elif leaf == "norm":
             t = 1 + 0.3 * rn(*shape)
         elif leaf in ("lq1", "lk1", "lq2", "lk2"):
-            t = rn(*shape) * (0.6 / shape[0] ** 0.25)
+            t = rn(*shape) * (0.4 / shape[0] ** 0.25)
         elif leaf == "b":
             t = rn(*shape) * 0.5
         elif len(shape) == 2:
