@@ -496,7 +496,7 @@ class ScaledInputMoe(Part):
             main = torch.cuda.current_stream()
             rt.side_stream.wait_stream(main)
             with torch.cuda.stream(rt.side_stream):
-                _relu2_mlp(rt, h, self.w_shared_up, self.w_shared_down, shared, "moe_shared", glu=s.shared_glu)
+                _relu2_mlp(rt, h, self.w_shared_up, self.w_shared_down, shared, "moe_shared")
         if n <= ops.ROUTE_SMALL_TOKENS and ops.route_small_fits(H, E):
             logits = ws.get("moe_logits", (n, E + 1), torch.float32)
             ops.route_small(router_in, self.w_router, None, logits, ids, wts, None, k, False, offsets, perm_token, perm_weight,
@@ -533,7 +533,7 @@ class ScaledInputMoe(Part):
                 main.wait_stream(rt.side_stream)
             else:
                 shared = ws.get("moe_shared_out", (n, H), torch.float32)
-                _relu2_mlp(rt, h, self.w_shared_up, self.w_shared_down, shared, "moe_shared", glu=s.shared_glu)
+                _relu2_mlp(rt, h, self.w_shared_up, self.w_shared_down, shared, "moe_shared")
         ops.moe_combine(out, ids, inverse, None, shared, y)
         return y
 
