@@ -540,6 +540,22 @@ def sebevik_config(width, ff, layers, vocab, window):
     return {"architecture": "Sebevik", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "layers": out}
 
 
+# --design satavik: the decoder with differential attention (two maps of 64 channels a head over values of 128, so a head
+# is as wide as the other's; every second layer reads the keys and values of the one before it) and routed experts with
+# clamped gated units in every layer, beside the Qwen2 MoE decoder of the same width, depth, heads and expert sizes with
+# experts in every layer (the closest model this library has: grouped attention, a router over gated experts, a shared
+# expert).  The mask's blocks are longer than the prompts, so that both models' queries see the same keys.
+def satavik_config(width, ff, layers, vocab, chunk):
+    heads = width // 128
+    mix = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 64, "vdim": 128, "scale": 64 ** -0.5, "softcap": 30.0, "diff": 0.4,
+           "rot": {"dims": 64, "base": 1e6}, "mask": {"size": chunk}}
+    moe = {"kind": "moe", "router": {"experts": VUMEDRA_EXPERTS, "top": VUMEDRA_TOP}, "expert": {"ff": ff // 4, "limit": 7.0},
+           "shared": {"ff": ff // 2, "limit": 7.0}}
+    out = [{"type": "attention", "mixer": dict(mix, kv_from=i - 1) if i % 2 else dict(mix), "mlp": dict(moe)} for i in range(layers)]
+    return {"architecture": "Satavik", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": 16.0},
+            "layers": out}
+
+
 def measure_design(torch, raw, prefill_tokens, batches, context, steps, warmup, clocks):
     """Prefill of one prompt and decode steps of a model with random weights: tokens per second, and device time
     by kind of kernel for one eager prefill and one eager decode step (library products count with the kernel
@@ -596,8 +612,9 @@ def bench_design(torch, a, pk):
     sizes = {"w1024": (1024, 2816, 8), "w2048": (2048, 5632, 8), "w4096": (4096, 11008, 8)}
     picked = [s for s in a.design_sizes.split(",") if s]
     vocab, window = 32768, 4096
-    vumedra, migosun, sebevik = a.design == "vumedra", a.design == "migosun", a.design == "sebevik"
+    vumedra, migosun, sebevik, satavik = (a.design == d for d in ("vumedra", "migosun", "sebevik", "satavik"))
     beside = ("Qwen2 MoE decoder of equal width, depth, heads, dense and expert sizes" if vumedra or sebevik else
+              "Qwen2 MoE decoder of equal width, depth, heads and expert sizes, experts in every layer" if satavik else
               "Zusepel decoder of equal width, depth and feed-forward width" if migosun else
               "dense Qwen2 decoder of equal width, depth and feed-forward width")
     result = {"design": a.design, "beside": beside, "dtype": "bf16",
@@ -613,10 +630,13 @@ def bench_design(torch, a, pk):
             mine, other = vumedra_config(width, ff, layers, vocab), sparse_qwen2_config(width, ff, layers, vocab)
         elif sebevik:
             mine, other = sebevik_config(width, ff, layers, vocab, window), sparse_qwen2_config(width, ff, layers, vocab)
+        elif satavik:
+            mine = satavik_config(width, ff, layers, vocab, window)
+            other = dict(sparse_qwen2_config(width, ff, layers, vocab), mlp_only_layers=[])
         else:
             mine, other = zusepel_config(width, ff, layers, vocab, window), dense_qwen2_config(width, ff, layers, vocab)
         entry[a.design] = measure_design(torch, mine, a.prefill_tokens, (1, 8), a.context, a.steps, a.warmup, clocks)
-        entry["zusepel" if migosun else "qwen2_moe" if vumedra or sebevik else "qwen2_dense"] = measure_design(
+        entry["zusepel" if migosun else "qwen2_moe" if vumedra or sebevik or satavik else "qwen2_dense"] = measure_design(
             torch, other, a.prefill_tokens, (1, 8), a.context, a.steps, a.warmup, clocks)
         result["sizes"][name] = entry
     result["clocks"] = clocks.summary()
@@ -626,10 +646,10 @@ def bench_design(torch, a, pk):
 
 def main() -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--design", default=None, choices=["zusepel", "vumedra", "migosun", "sebevik"],
+    ap.add_argument("--design", default=None, choices=["zusepel", "vumedra", "migosun", "sebevik", "satavik"],
                     help="instead of the default workload: prefill and decode of this design at a few layer sizes, beside "
                          "the closest other decoder of equal size (the dense Qwen2 for zusepel, the Qwen2 with routed "
-                         "experts for vumedra and sebevik, zusepel for migosun)")
+                         "experts for vumedra, sebevik and satavik, zusepel for migosun)")
     ap.add_argument("--design-sizes", default="w1024,w2048", help="with --design: which of w1024, w2048, w4096")
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=32)
