@@ -98,9 +98,10 @@ struct DiffParams {
     long long ldg;
 };
 
-// cap * tanh(s / cap) by tanh(x) = 1 - 2 / (1 + e^(2x)): the absolute error is a few units of 2^-24 times cap
-__device__ __forceinline__ float softcap_score(float s, float cap) {
-    return cap - __fdividef(2.0f * cap, 1.0f + __expf(2.0f * s / cap));
+// cap * tanh(s * unit), unit = scale / cap, by tanh(x) = 1 - 2 / (1 + e^(2x)): the absolute error is a few units of 2^-24
+// times cap
+__device__ __forceinline__ float softcap_score(float s, float unit, float cap) {
+    return cap - __fdividef(2.0f * cap, 1.0f + __expf(s * (2.0f * unit)));
 }
 
 template <int HDK, int HDV, int MAPS>
@@ -210,7 +211,7 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
         for (; issued < min(RING, n_items); issued++) issue(issued);
     }
 
-    const float root = sqrtf((float)HDK);
+    const float root = sqrtf((float)HDK), cap_unit = MAPS == 2 && df.softcap > 0.f ? score_scale / df.softcap : 0.f;
     float o[NBW][4];
 #pragma unroll
     for (int i = 0; i < NBW; i++)
@@ -243,8 +244,9 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
             for (int j = 0; j < 4; j++) {
                 const int t = warp * 16 + nb * 8 + tg * 2 + (j & 1), key = key0 + t;
                 const bool live = page_ok && key >= j0 && key <= j1;
-                float sv = score_scale > 0.f ? sc[nb][j] * score_scale : sc[nb][j] / root;
-                if (MAPS == 2 && df.softcap > 0.f) sv = softcap_score(sv, df.softcap);
+                float sv;
+                if (MAPS == 2) sv = df.softcap > 0.f ? softcap_score(sc[nb][j], cap_unit, df.softcap) : sc[nb][j] * score_scale;
+                else sv = score_scale > 0.f ? sc[nb][j] * score_scale : sc[nb][j] / root;
                 if (g8 + (j >> 1) * 8 < heads) s_s[g8 + (j >> 1) * 8][t] = live ? sv : -INFINITY;
             }
         __syncthreads();                           // scores are written; the key buffer is free

@@ -986,11 +986,33 @@ __global__ void cast_cols_kernel(const float* __restrict__ src, long long ld, TO
     }
 }
 
+// The same for widths and strides of whole pieces of four numbers on aligned buffers.
+template <typename TO>
+__global__ void cast_cols_vec_kernel(const float* __restrict__ src, long long ld, TO* __restrict__ dst, long long rows, int width) {
+    pdl_trigger();
+    pdl_wait();
+    const int pieces = width / 4;
+    const long long total = rows * pieces;
+    for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
+        const long long r = i / pieces;
+        const float4 v = *reinterpret_cast<const float4*>(src + r * ld + 4 * (i - r * pieces));
+        Vec4<TO>::store(dst + 4 * i, v.x, v.y, v.z, v.w);
+    }
+}
+
 ESP_API int esp_cast_cols(const float* src, long long ld, void* dst, int dst_is_bf16, long long rows, int width,
                           cudaStream_t stream) {
     if (rows <= 0 || width <= 0) return 0;
-    long long blocks = (rows * width + 255) / 256;
+    const bool vec = width % 4 == 0 && ld % 4 == 0 && (((size_t)src | (size_t)dst) & 15) == 0;
+    long long blocks = (rows * (vec ? width / 4 : width) + 255) / 256;
     if (blocks > 148 * 16) blocks = 148 * 16;
+    if (vec) {
+        if (dst_is_bf16)
+            esp_launch_pdl(ESP_PDL_SMALL, cast_cols_vec_kernel<bf16>, dim3((int)blocks), dim3(256), 0, stream, src, ld, (bf16*)dst, rows, width);
+        else
+            esp_launch_pdl(ESP_PDL_SMALL, cast_cols_vec_kernel<float>, dim3((int)blocks), dim3(256), 0, stream, src, ld, (float*)dst, rows, width);
+        return esp_launch_status();
+    }
     if (dst_is_bf16)
         esp_launch_pdl(ESP_PDL_SMALL, cast_cols_kernel<bf16>, dim3((int)blocks), dim3(256), 0, stream, src, ld, (bf16*)dst, rows, width);
     else

@@ -743,6 +743,90 @@ headnorm_rope_kvwrite_kernel(const float* __restrict__ rows, long long ld, const
     }
 }
 
+// The same for runs of up to 128 channels in whole pieces of four, half a rotation in whole pieces and aligned buffers:
+// LPR lanes hold a run, four channels each, so its sum of squares and the partners of its rotation come by shuffle, and a
+// warp keeps its angles and the norms' weights in registers over the runs it takes.  Grid: (tokens, shares of the runs).
+// Positions and page tables were written before the step's first kernel: what hangs on them precedes the wait.
+template <typename T, int LPR>
+__global__ void __launch_bounds__(128)
+headnorm_rope_kvwrite_lanes_kernel(const float* __restrict__ rows, long long ld, const float* __restrict__ q_w,
+                                   const float* __restrict__ k_w, float eps, const float* __restrict__ inv_freq, int rot,
+                                   const int* __restrict__ tok_seq, const int* __restrict__ tok_pos, T* __restrict__ q_out,
+                                   T* __restrict__ k_cache, T* __restrict__ v_cache, const int* __restrict__ block_table,
+                                   int table_stride, int n_pages, int page, int nh, int nkv, int maps, int hd, int vd,
+                                   int own_kv, int* __restrict__ status) {
+    pdl_trigger();
+    constexpr int RPW = 32 / LPR;                           // runs that a warp holds at a time
+    const int n = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nwarp = blockDim.x >> 5;
+    const int sub = lane / LPR, c = 4 * (lane % LPR), half = rot / 2;
+    const int q_runs = nh * maps, runs = q_runs + (own_kv ? nkv * maps : 0), chans = runs * hd;
+    const bool in_run = c < hd;
+    const int pos = tok_pos[n], seq = tok_seq[n];
+    int page_id = -1;
+    if (own_kv) {
+        page_id = block_table[(size_t)seq * table_stride + pos / page];
+        if (page_id < 0 || page_id >= n_pages) {
+            if (tid == 0 && blockIdx.y == 0) atomicOr(status, ESP_STATUS_BAD_INDEX);
+            page_id = -1;
+        }
+    }
+    const int in_page = pos % page;
+    float co[4], si[4];
+    const bool first = c < half, turns = c < rot;           // this lane's four channels are the first / a rotated half
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        co[i] = 1.f, si[i] = 0.f;
+        if (turns) sincosf((float)pos * inv_freq[(first ? c : c - half) + i], &si[i], &co[i]);
+        if (first) si[i] = -si[i];
+    }
+    const int partner = turns ? (first ? lane + half / 4 : lane - half / 4) : lane;
+    float4 wq = make_float4(1.f, 1.f, 1.f, 1.f), wk = wq;
+    if (in_run && q_w) wq = *reinterpret_cast<const float4*>(q_w + c);
+    if (in_run && k_w) wk = *reinterpret_cast<const float4*>(k_w + c);
+    pdl_wait();
+    const float* src = rows + (size_t)n * ld;
+    const int step = gridDim.y * nwarp * RPW;
+    int r = (blockIdx.y * nwarp + warp) * RPW + sub;
+    const float4 none = make_float4(0.f, 0.f, 0.f, 0.f);
+    float4 next = in_run && r < runs ? *reinterpret_cast<const float4*>(src + (size_t)r * hd + c) : none;
+    for (int r0 = r - sub; r0 < runs; r0 += step, r += step) {        // the warp's lanes leave together
+        const float4 x = next;
+        if (in_run && r + step < runs) next = *reinterpret_cast<const float4*>(src + (size_t)(r + step) * hd + c);
+        float ss = fmaf(x.w, x.w, fmaf(x.z, x.z, fmaf(x.y, x.y, x.x * x.x)));
+#pragma unroll
+        for (int o = LPR / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+        const bool is_q = r < q_runs;
+        const bool normed = is_q ? q_w != nullptr : k_w != nullptr;
+        const float f = normed ? 1.0f / sqrtf(ss / (float)hd + eps) : 1.0f;
+        const float4 w = is_q ? wq : wk;
+        const float a[4] = {x.x * f * w.x, x.y * f * w.y, x.z * f * w.z, x.w * f * w.w};
+        float y[4];
+#pragma unroll
+        for (int i = 0; i < 4; i++) {
+            const float b = __shfl_sync(0xffffffffu, a[i], partner);
+            y[i] = turns ? a[i] * co[i] + b * si[i] : a[i];
+        }
+        if (!in_run || r >= runs) continue;
+        T* dst;
+        if (is_q) {
+            dst = q_out + ((size_t)n * q_runs + r) * hd;
+        } else if (page_id >= 0) {
+            const int kr = r - q_runs, head = kr / maps, m = kr - head * maps;
+            dst = k_cache + (((size_t)page_id * nkv + head) * page + in_page) * (maps * hd) + m * hd;
+        } else {
+            continue;
+        }
+        Vec4<T>::store(dst + c, y[0], y[1], y[2], y[3]);
+    }
+    if (page_id >= 0) {
+        for (int e = 4 * (blockIdx.y * blockDim.x + tid); e < nkv * vd; e += 4 * gridDim.y * blockDim.x) {
+            const int head = e / vd, d = e - head * vd;
+            const float4 v = *reinterpret_cast<const float4*>(src + chans + e);
+            Vec4<T>::store(v_cache + (((size_t)page_id * nkv + head) * page + in_page) * vd + d, v.x, v.y, v.z, v.w);
+        }
+    }
+}
+
 ESP_API int esp_headnorm_rope_kvwrite(const float* rows, long long ld, const float* q_w, const float* k_w, float eps,
                                       const float* inv_freq, int rot, const int* tok_seq, const int* tok_pos, void* q_out,
                                       void* k_cache, void* v_cache, int is_bf16, const int* block_table, int table_stride,
@@ -757,6 +841,26 @@ ESP_API int esp_headnorm_rope_kvwrite(const float* rows, long long ld, const flo
     if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
     const size_t ptrs = (size_t)rows | (size_t)q_w | (size_t)k_w | (size_t)q_out | (size_t)k_cache | (size_t)v_cache;
     const bool vec = hd % 4 == 0 && vd % 4 == 0 && rot % 8 == 0 && ld % 4 == 0 && (ptrs & 15) == 0;
+    if (vec && hd <= 128) {
+        const int lanes = hd <= 32 ? 8 : hd <= 64 ? 16 : 32, per_block = 4 * (32 / lanes);
+        // few tokens: a block takes a warp's worth of runs per warp and the token is spread over several
+        const dim3 grid(n_tokens, n_tokens <= 64 ? (unsigned)((runs + per_block - 1) / per_block) : 1u);
+#define ESP_HEADNORM_LANES(T, LPR)                                                                                           \
+    esp_launch_pdl(ESP_PDL_SMALL, headnorm_rope_kvwrite_lanes_kernel<T, LPR>, grid, dim3(128), 0, stream, rows, ld, q_w, k_w, eps, \
+                   inv_freq, rot, tok_seq, tok_pos, (T*)q_out, (T*)k_cache, (T*)v_cache, block_table, table_stride, n_pages, page, \
+                   nh, nkv, maps, hd, vd, own_kv, status)
+#define ESP_HEADNORM_LANES_T(T)                       \
+    do {                                              \
+        if (lanes == 8) ESP_HEADNORM_LANES(T, 8);     \
+        else if (lanes == 16) ESP_HEADNORM_LANES(T, 16); \
+        else ESP_HEADNORM_LANES(T, 32);               \
+    } while (0)
+        if (is_bf16) ESP_HEADNORM_LANES_T(bf16);
+        else ESP_HEADNORM_LANES_T(float);
+#undef ESP_HEADNORM_LANES_T
+#undef ESP_HEADNORM_LANES
+        return esp_launch_status();
+    }
     const int threads = runs * hd >= 1024 ? 256 : 128;
 #define ESP_HEADNORM(T, VEC)                                                                                              \
     do {                                                                                                                  \
