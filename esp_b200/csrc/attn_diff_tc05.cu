@@ -15,9 +15,10 @@
 // sigmoid(gate), all in 32-bit, on its way out.  Two groups of row threads take a map each, so the two maps are what
 // keeps the tensor core busy while the other's scores are turned into weights.
 //
-// Soft cap: a scaled score s becomes cap tanh(s / cap).  For |s / cap| <= 3/4 it is an odd polynomial (interpolated at
-// Chebyshev points; relative error below 1e-7), evaluated for two scores at a time on the multiply-add units; a warp
-// that holds a larger one in a run of 32 keys takes tanh(x) = 1 - 2 / (1 + e^(2x)) for that run.
+// Soft cap: a scaled score s becomes cap tanh(s / cap).  For |s / cap| <= 5/8 it is an odd polynomial (interpolated at
+// Chebyshev points; relative error 1.2e-7), evaluated for two scores at a time on the multiply-add units, with the scale
+// and the cap in its coefficients; a warp that holds a larger one in a run of 32 keys takes tanh(x) = 1 - 2 / (1 + e^(2x))
+// for that run.
 //
 // FIXED: with a cap of at most 60 no score leaves +-60 log2(e) < 87 in powers of two, so the weights are taken as they
 // are (reference 0): float and bfloat16 have the range, and there is no maximum to find and nothing to rescale.  Else
@@ -37,10 +38,10 @@ namespace {
 using namespace tc05;
 constexpr int BM = 128, BN = 128, PAGE = 64, MAPS = 2, ROWT = 2;
 constexpr int ATOM_BYTES = 128 * 128;           // 128 rows of 128 bytes: one 64-wide slice of a 128-row operand
-constexpr int POLY = 6;
-// tanh(x) / x as a polynomial in x^2 on |x| <= 3/4
-constexpr float TANH_POLY[POLY] = {1.0f, -0.33332952857f, 0.13325339556f, -0.05334111676f, 0.01957621612f, -0.00471152226f};
-constexpr float TANH_POLY_MAX = 0.75f;
+constexpr int POLY = 5;
+// tanh(x) / x as a polynomial in x^2 on |x| <= 5/8
+constexpr double TANH_POLY[POLY] = {0.99999988079, -0.33331942558, 0.13304379582, -0.051815912127, 0.015043356456};
+constexpr float TANH_POLY_MAX = 0.625f;
 constexpr float LOG2E = 1.4426950408889634f;
 constexpr float FIXED_CAP_MAX = 60.f;
 
@@ -59,7 +60,8 @@ struct DiffAttnParams {
     float to_unit;            // scores to the argument of tanh (scale / cap); without a cap to powers of two (scale log2 e)
     float cap2;               // cap log2(e), or 0: no cap
     float lambda, eps, out_scale;
-    unsigned long long poly[POLY];   // TANH_POLY times cap2, each twice
+    float raw_max;            // raw scores up to here take the polynomial
+    unsigned long long poly[POLY];   // TANH_POLY[k] cap2 to_unit^(2k + 1), each twice: a polynomial in the raw score's square
 };
 
 __device__ __forceinline__ unsigned idesc_attn(int n, bool b_mn_major) {
@@ -100,6 +102,17 @@ __device__ __forceinline__ unsigned long long fma2(unsigned long long a, unsigne
 __device__ __forceinline__ unsigned long long mul2(unsigned long long a, unsigned long long b) {
     unsigned long long d;
     asm("mul.rn.f32x2 %0, %1, %2;\n" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+__device__ __forceinline__ unsigned long long add2(unsigned long long a, unsigned long long b) {
+    unsigned long long d;
+    asm("add.rn.f32x2 %0, %1, %2;\n" : "=l"(d) : "l"(a), "l"(b));
+    return d;
+}
+// the largest magnitude of three
+__device__ __forceinline__ float max_abs3(float a, float b, float c) {
+    float d;
+    asm("max.abs.f32 %0, %1, %2, %3;\n" : "=f"(d) : "f"(a), "f"(b), "f"(c));
     return d;
 }
 // the ``count`` threads that meet at named barrier ``id`` learn whether all of them are well
@@ -359,7 +372,6 @@ attn_diff_tc05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
         const unsigned s_addr = tm_s + grp * BN + lane_sel + side * CW;
         const bool capped = FIXED || p.cap2 > 0.f;
         const float unit = p.to_unit, cap2 = p.cap2;
-        const float raw_max = TANH_POLY_MAX / unit;                       // raw scores up to here take the polynomial
         bool ok = true;
         int n_b = 0;                                                      // key blocks so far
         for (int round = 0; ok; round++) {
@@ -425,7 +437,7 @@ attn_diff_tc05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                 }
                 const float m_use = FIXED || m_ref == -INFINITY ? 0.f : m_ref;
                 const unsigned long long neg_m = pack2(-m_use, -m_use), unit2 = pack2(unit, unit);
-                float l_add = 0.f;
+                unsigned long long l_add = 0;                              // two sums: of the even and of the odd keys
                 // the weights of keys 2c and 2c + 1 of this thread's run go to column c of its columns of S
 #pragma unroll
                 for (int c = 0; c < CW / 32; c++) {
@@ -434,17 +446,19 @@ attn_diff_tc05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                     tc_ld32(s_addr + c * 32, sv);
                     bool small = false;
                     if (capped) {
-                        float am = fabsf(sv[0]);
+                        float am = max_abs3(sv[0], sv[1], sv[2]), bm = max_abs3(sv[3], sv[4], sv[5]);
 #pragma unroll
-                        for (int i = 1; i < 32; i++) am = fmaxf(am, fabsf(sv[i]));
-                        small = __all_sync(0xffffffffu, am <= raw_max);
+                        for (int i = 6; i < 30; i += 4) {
+                            am = max_abs3(am, sv[i], sv[i + 1]);
+                            bm = max_abs3(bm, sv[i + 2], sv[i + 3]);
+                        }
+                        small = __all_sync(0xffffffffu, fmaxf(max_abs3(am, sv[30], sv[31]), bm) <= p.raw_max);
                     }
                     if (small) {
 #pragma unroll
                         for (int i = 0; i < 32; i += 2) {
-                            const unsigned long long x = mul2(pack2(sv[i], sv[i + 1]), unit2), y = mul2(x, x);
-                            unsigned long long f = fma2(p.poly[5], y, p.poly[4]);
-                            f = fma2(f, y, p.poly[3]);
+                            const unsigned long long x = pack2(sv[i], sv[i + 1]), y = mul2(x, x);
+                            unsigned long long f = fma2(p.poly[4], y, p.poly[3]);
                             f = fma2(f, y, p.poly[2]);
                             f = fma2(f, y, p.poly[1]);
                             f = fma2(f, y, p.poly[0]);
@@ -466,14 +480,16 @@ attn_diff_tc05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
 #pragma unroll
                     for (int i = 0; i < 32; i += 2) {                     // a masked score is -inf: its weight is 0
                         const float p0 = fast_exp2(sv[i]), p1 = fast_exp2(sv[i + 1]);
-                        l_add += p0 + p1;
+                        l_add = add2(l_add, pack2(p0, p1));
                         __nv_bfloat162 b2 = __floats2bfloat162_rn(p0, p1);
                         packed[i >> 1] = *reinterpret_cast<unsigned*>(&b2);
                     }
                     tc_st16(s_addr + c * 16, packed);
                 }
                 tc_wait_st();
-                l_run += l_add;
+                float l_even, l_odd;
+                unpack2(l_add, l_even, l_odd);
+                l_run += l_even + l_odd;
                 tc_fence_before();                                        // S has been read, P and O written
                 __syncwarp();
                 if (lane == 0) mbar_arrive(&p_ready[grp]);
@@ -652,8 +668,11 @@ ESP_API int esp_attn_diff_tc05(const void* q, long long n_tokens, const void* k_
     p.kv_rows = (int)kv_rows; p.n_tiles = n_tiles; p.status = status; p.lambda = lambda; p.eps = eps; p.out_scale = out_scale;
     p.cap2 = softcap * LOG2E;
     p.to_unit = softcap > 0.f ? scale / softcap : scale * LOG2E;
-    for (int i = 0; i < POLY; i++) {
-        const float c = TANH_POLY[i] * p.cap2;
+    p.raw_max = TANH_POLY_MAX / p.to_unit;
+    double power = (double)p.cap2 * p.to_unit;
+    for (int i = 0; i < POLY; i++, power *= (double)p.to_unit * p.to_unit) {
+        const float c = (float)(TANH_POLY[i] * power);
+        if (softcap > 0.f && !(c < -1e-36f || c > 1e-36f)) p.raw_max = -1.f;      // too small for float: the other form throughout
         unsigned bits;
         memcpy(&bits, &c, 4);
         p.poly[i] = ((unsigned long long)bits << 32) | bits;
