@@ -115,7 +115,8 @@ class DifferentialAttention(Part):
     def kernel_for(self, n: int, page: int = PAGE) -> str:
         s = self.spec
         if self.rt.dtype == torch.bfloat16:
-            if n <= DECODE_ROWS and ops.attn_decode_diff_fits(s.key_dim, s.value_dim, page):
+            if (n <= DECODE_ROWS and ops.attn_decode_diff_fits(s.key_dim, s.value_dim, page)
+                    and n * 2 * s.num_heads <= ops.ATTN_DECODE_COUNTERS):
                 return "split"         # few rows: the keys are split over blocks
             if ops.attn_diff_tc05_fits(s.key_dim, s.value_dim, page):
                 return "tc05"          # many rows: both maps' scores and weighted values in tensor memory
