@@ -176,12 +176,13 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
         for (; issued < min(RING, n_items); issued++) issue(issued);
     }
     pdl_wait();
+    const bf16* q_now = behind_wait(q);            // the kernel before this one wrote the queries
     // the query fragments of the block's heads (rows beyond ``heads`` are zero)
     unsigned qa[HDK / 16][4];
     if constexpr (MAPS == 2) {
         // a row's channels lie where its map's keys lie in a key row (h0 is even: rows g8 and g8 + 8 belong to map g8 % 2)
         const int kd = df.key_dim, off = (g8 & 1) * kd;
-        const bf16* q0 = q + ((size_t)n * nh + h0 + g8) * kd - off;
+        const bf16* q0 = q_now + ((size_t)n * nh + h0 + g8) * kd - off;
         const bf16* q1 = q0 + (size_t)8 * kd;
         auto piece = [&](const bf16* row, int c, bool live) {
             return live && c >= off && c < off + kd ? *reinterpret_cast<const unsigned*>(row + c) : 0u;
@@ -195,8 +196,8 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
             qa[kk][3] = piece(q1, c + 8, g8 + 8 < heads);
         }
     } else {
-        const bf16* q0 = q + ((size_t)n * nh + h0 + g8) * HDK;
-        const bf16* q1 = q + ((size_t)n * nh + h0 + g8 + 8) * HDK;
+        const bf16* q0 = q_now + ((size_t)n * nh + h0 + g8) * HDK;
+        const bf16* q1 = q_now + ((size_t)n * nh + h0 + g8 + 8) * HDK;
 #pragma unroll
         for (int kk = 0; kk < HDK / 16; kk++) {
             const int c = kk * 16 + tg * 2;

@@ -110,6 +110,13 @@ static inline int esp_launch_status() { return (int)cudaGetLastError(); }
 __device__ __forceinline__ void pdl_wait() { asm volatile("griddepcontrol.wait;\n" ::: "memory"); }
 __device__ __forceinline__ void pdl_trigger() { asm volatile("griddepcontrol.launch_dependents;\n" ::: "memory"); }
 
+// A pointer for use behind pdl_wait().  Loads through a ``const __restrict__`` pointer may be taken for loads of constant
+// memory, which nothing keeps behind the wait; the compiler does not know this pointer's value before the wait.
+template <typename T> __device__ __forceinline__ T* behind_wait(T* p) {
+    asm volatile("" : "+l"(p)::"memory");
+    return p;
+}
+
 #define ESP_PDL_DEFAULT_MASK 61
 // classes of kernels, so that the attribute can be tried class by class: ESP_B200_PDL is a bit mask.  GROUPED: every
 // grouped product (off: it holds SM room while it waits for the routing); GROUPED_AFTER: a second grouped product

@@ -484,6 +484,7 @@ __global__ void norm_add_rmsnorm_kernel(float* __restrict__ x, const float* __re
                                         TH* __restrict__ h, float* __restrict__ h32, int width, float eps, int write_x) {
     pdl_trigger();
     pdl_wait();
+    y = behind_wait(y);
     __shared__ float scratch[33];
     const int r = blockIdx.x;
     const size_t s = rows ? (size_t)rows[r] : (size_t)r;
@@ -524,6 +525,7 @@ norm_add_rmsnorm_rows_kernel(float* __restrict__ x, const float* __restrict__ y,
                              TH* __restrict__ h, float* __restrict__ h32, int width, float eps, int write_x) {
     pdl_trigger();
     pdl_wait();
+    y = behind_wait(y);
     __shared__ float scratch[33];
     const int r = blockIdx.x;
     const size_t s = rows ? (size_t)rows[r] : (size_t)r;
@@ -991,6 +993,7 @@ template <typename TO>
 __global__ void cast_cols_vec_kernel(const float* __restrict__ src, long long ld, TO* __restrict__ dst, long long rows, int width) {
     pdl_trigger();
     pdl_wait();
+    src = behind_wait(src);
     const int pieces = width / 4;
     const long long total = rows * pieces;
     for (long long i = blockIdx.x * (long long)blockDim.x + threadIdx.x; i < total; i += (long long)gridDim.x * blockDim.x) {
@@ -1033,7 +1036,7 @@ diff_combine_kernel(const float* __restrict__ a, float lambda, float eps, float 
     const int lane = threadIdx.x & 31;
     const long long pair = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (pair >= pairs) return;
-    const float* a1 = a + pair * 2 * V;
+    const float* a1 = behind_wait(a) + pair * 2 * V;
     const float* a2 = a1 + V;
     float ss = 0.f;
     for (int d = lane; d < V; d += 32) {

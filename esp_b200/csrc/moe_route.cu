@@ -405,6 +405,7 @@ router_logits_kernel(const TH* __restrict__ h, const TW* __restrict__ w_router, 
         for (int b = lane * 128; b < width * (int)sizeof(TW); b += 32 * 128)
             asm volatile("prefetch.global.L2 [%0];\n" ::"l"(reinterpret_cast<const char*>(wr) + b));
     pdl_wait();
+    h = behind_wait(h);
     for (int i = tid; i < width; i += 256) hs[i] = to_f32(h[(size_t)n * width + i]);
     __syncthreads();
     if (e >= rows) return;
@@ -425,6 +426,7 @@ route_small_kernel(const float* __restrict__ logits, int* __restrict__ topk_ids,
                    int* __restrict__ tile_count, int* __restrict__ n_tiles) {
     pdl_trigger();
     pdl_wait();
+    logits = behind_wait(logits);
     extern __shared__ float sm_f[];
     float* ps_all = sm_f;                                      // [8 warps][2 * n_experts]: scores, corrected scores
     int* counts = reinterpret_cast<int*>(sm_f + 16 * n_experts); // [n_experts]
@@ -674,6 +676,8 @@ __global__ void moe_combine_kernel(const float* __restrict__ expert_out, const i
                                    const float* __restrict__ topk_w, const float* __restrict__ ident, int n_real) {
     pdl_trigger();
     pdl_wait();
+    expert_out = behind_wait(expert_out);
+    shared = behind_wait(shared);
     __shared__ int order[MAX_TOPK];
     __shared__ float pass_w[MAX_TOPK];
     const int t = blockIdx.x;
@@ -778,6 +782,8 @@ moe_combine_add_rmsnorm_kernel(const float* __restrict__ expert_out, const int* 
     }
     __syncthreads();
     pdl_wait();
+    expert_out = behind_wait(expert_out);
+    shared = behind_wait(shared);
     float4 y[4];
     float ssy = 0.f;
 #pragma unroll

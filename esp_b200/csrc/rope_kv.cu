@@ -677,7 +677,7 @@ headnorm_rope_kvwrite_kernel(const float* __restrict__ rows, long long ld, const
         }
     }
     const int in_page = pos % page;
-    const float* src = rows + (size_t)n * ld;
+    const float* src = behind_wait(rows) + (size_t)n * ld;
     for (int e = VEC * tid; e < chans; e += VEC * blockDim.x) {
         if (VEC == 4) *reinterpret_cast<float4*>(row + e) = *reinterpret_cast<const float4*>(src + e);
         else row[e] = src[e];
@@ -784,7 +784,7 @@ headnorm_rope_kvwrite_lanes_kernel(const float* __restrict__ rows, long long ld,
     if (in_run && q_w) wq = *reinterpret_cast<const float4*>(q_w + c);
     if (in_run && k_w) wk = *reinterpret_cast<const float4*>(k_w + c);
     pdl_wait();
-    const float* src = rows + (size_t)n * ld;
+    const float* src = behind_wait(rows) + (size_t)n * ld;
     const int step = gridDim.y * nwarp * RPW;
     int r = (blockIdx.y * nwarp + warp) * RPW + sub;
     const float4 none = make_float4(0.f, 0.f, 0.f, 0.f);

@@ -253,6 +253,26 @@ def test_cuttings_agree_bit_for_bit_in_float32(folders, name):
             assert np.array_equal(first, other.logits_of(rid, at))
 
 
+@pytest.mark.parametrize("name", ["B", "+blocks", "+cap", "+no_cap", "+all_keys"])
+def test_captured_decode_steps_in_bfloat16(folders, name):
+    """Decode steps replayed from captured graphs, where a kernel is set up while the one before it still runs: what it
+    reads of that one before it has waited shows as the last step's values.  Models in which no expert's choice can flip;
+    each request three times over, alone and as one batch."""
+    reqs = requests_for(name, (60, 75, 45), seed=17)
+    eng = engine_for(folders[name], "bfloat16", record=False)
+    ids = list(reqs)
+    for steps in [steps_tail(reqs, tail=30)] * 3 + [steps_batches(reqs, [ids], {rid: len(t) - 25 for rid, t in reqs.items()})] * 2:
+        before = eng.graph_replays
+        rec = Rec(model(name)[0]["vocab"])
+        run_steps(eng, steps, rec)
+        assert eng.graph_replays > before
+        raw, w = model(name)
+        for rid, toks in reqs.items():
+            ref = plain.forward(raw, w, toks).numpy()
+            err = relative_error(rec.logits_of(rid, list(range(len(toks)))), ref)
+            assert (err <= allowed(raw, w, toks, None, "bfloat16", ref, err)).all(), (rid, int(err.argmax()), float(err.max()))
+
+
 def test_long_decoding_in_a_small_cache(folders):
     """300 single tokens after a prompt of 3 in a cache of 6 pages: layers whose blocks end give their old pages back and
     get them again (the cache that two layers read under blocks of different sizes keeps what the longer one sees)."""
