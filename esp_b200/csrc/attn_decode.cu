@@ -259,9 +259,12 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
             const float m_new = fmaxf(m_old, warp_max(fmaxf(a, b)));
             const float m_use = m_new == -INFINITY ? 0.f : m_new;
             const float pa = a == -INFINITY ? 0.f : expf(a - m_use), pb = b == -INFINITY ? 0.f : expf(b - m_use);
-            const float sum = warp_sum(pa + pb);
-            p_s[h][lane] = __float2bfloat16_rn(pa);
-            p_s[h][lane + 32] = __float2bfloat16_rn(pb);
+            const bf16 ra = __float2bfloat16_rn(pa), rb = __float2bfloat16_rn(pb);
+            // the differential form sums the weights as the product will see them: what is left of two maps that nearly
+            // cancel must not be their rounding
+            const float sum = warp_sum(MAPS == 2 ? __bfloat162float(ra) + __bfloat162float(rb) : pa + pb);
+            p_s[h][lane] = ra;
+            p_s[h][lane + 32] = rb;
             if (lane == 0) {
                 const float scale = expf(m_old - m_use);
                 scale_s[h] = scale;

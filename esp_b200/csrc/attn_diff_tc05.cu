@@ -479,10 +479,12 @@ attn_diff_tc05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_co
                     }
 #pragma unroll
                     for (int i = 0; i < 32; i += 2) {                     // a masked score is -inf: its weight is 0
-                        const float p0 = fast_exp2(sv[i]), p1 = fast_exp2(sv[i + 1]);
-                        l_add = add2(l_add, pack2(p0, p1));
-                        __nv_bfloat162 b2 = __floats2bfloat162_rn(p0, p1);
-                        packed[i >> 1] = *reinterpret_cast<unsigned*>(&b2);
+                        __nv_bfloat162 b2 = __floats2bfloat162_rn(fast_exp2(sv[i]), fast_exp2(sv[i + 1]));
+                        // the sum is of the weights as the product will see them: a row with one key then returns its value
+                        // exactly in either map, whatever the weight (the maps' difference may be all that is left of it)
+                        const unsigned w2 = *reinterpret_cast<unsigned*>(&b2);
+                        l_add = add2(l_add, pack2(__uint_as_float(w2 << 16), __uint_as_float(w2 & 0xffff0000u)));
+                        packed[i >> 1] = w2;
                     }
                     tc_st16(s_addr + c * 16, packed);
                 }

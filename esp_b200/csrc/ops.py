@@ -48,7 +48,7 @@ _SIGNATURES = {
                          c_int, c_int, P, P],
     "esp_attn_simt": [P, P, P, P, c_int, c_int, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, P,
                       c_int, c_int, c_float, c_int, P, P],
-    "esp_headnorm_rope_kvwrite": [P, c_longlong, P, P, c_float, P, c_int, P, P, P, P, P, c_int, P, c_int, c_int, c_int, c_int,
+    "esp_headnorm_rope_kvwrite": [P, c_longlong, P, P, c_float, P, P, c_int, P, P, P, P, P, c_int, P, c_int, c_int, c_int, c_int,
                                   c_int, c_int, c_int, c_int, c_int, c_int, P, P],
     "esp_diff_combine": [P, c_float, c_float, c_float, P, c_longlong, P, c_int, c_int, c_int, c_int, P],
     "esp_embed_sum": [P, P, c_int, P, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_longlong, c_longlong, c_float, P, P],
@@ -724,10 +724,10 @@ def attn_diff_tc05(q, k_cache, v_cache, out, maps_out, tile_seq, tile_first, seq
         float(eps), float(out_scale), gp, ldg, _ptr(status, torch.int32), _stream()), "attn_diff_tc05")
 
 
-def headnorm_rope_kvwrite(rows, q_w, k_w, eps, inv_freq, rot, tok_seq, tok_pos, q_out, k_cache, v_cache, block_table, page,
+def headnorm_rope_kvwrite(rows, q_w, k_w, eps, inv_freq, inv_freq_lo, rot, tok_seq, tok_pos, q_out, k_cache, v_cache, block_table, page,
                           nh, nkv, maps, hd, vd, own_kv, status):
     """RMS norm per head and map (weights q_w, k_w of hd numbers), rotation of the first ``rot`` channels of every run by
-    position * inv_freq, and the write of keys [pages, nkv, page, maps * hd] and values [pages, nkv, page, vd] into the
+    position * (inv_freq + inv_freq_lo), and the write of keys [pages, nkv, page, maps * hd] and values [pages, nkv, page, vd] into the
     paged cache.  rows float32 [N, >= (nh + nkv) * maps * hd + nkv * vd] (own_kv False: the queries alone, and no cache
     write); q_out [N, nh * maps * hd]."""
     n = q_out.shape[0]
@@ -736,8 +736,9 @@ def headnorm_rope_kvwrite(rows, q_w, k_w, eps, inv_freq, rot, tok_seq, tok_pos, 
         raise Backend("headnorm_rope_kvwrite: the rows' width disagrees with the head counts")
     p, ld = _rows_ld(rows, "rows")
     _check(_fn("core", "esp_headnorm_rope_kvwrite")(
-        p, ld, _ptr(q_w, torch.float32), _ptr(k_w, torch.float32), float(eps), _ptr(inv_freq, torch.float32), int(rot),
-        _ptr(tok_seq, torch.int32), _ptr(tok_pos, torch.int32), _ptr(q_out, FLOATS, "q_out"), _ptr(k_cache, q_out.dtype),
+        p, ld, _ptr(q_w, torch.float32), _ptr(k_w, torch.float32), float(eps), _ptr(inv_freq, torch.float32),
+        _ptr(inv_freq_lo, torch.float32), int(rot), _ptr(tok_seq, torch.int32), _ptr(tok_pos, torch.int32),
+        _ptr(q_out, FLOATS, "q_out"), _ptr(k_cache, q_out.dtype),
         _ptr(v_cache, q_out.dtype), _is_bf16(q_out), _ptr(block_table, torch.int32), block_table.shape[1], k_cache.shape[0],
         page, n, nh, nkv, maps, hd, vd, 1 if own_kv else 0, _ptr(status, torch.int32), _stream()), "headnorm_rope_kvwrite")
 

@@ -644,15 +644,28 @@ ESP_API int esp_pair_rope_unitnorm_kvwrite(const float* qkv, const float* bias, 
 // gate, padding) is left alone.  A head's channels are ``maps`` runs of hd.  Every run of a query (key) is divided by
 // its root mean square over hd (eps inside the root) and multiplied by q_w (k_w), hd numbers that all heads and maps
 // share (null: no norm for that side); then its first ``rot`` channels are rotated, channel i with channel i + rot/2,
-// by the angle position * inv_freq[i] (a 32-bit product; sine and cosine in 32-bit).  Queries go to q_out
+// by the angle position * frequency (angle_sincos).  Queries go to q_out
 // [n_tokens, nh, maps * hd], keys [pages, nkv, PAGE, maps * hd] and values [pages, nkv, PAGE, vd] to the token's place
 // in the paged cache.  One block per token; a row's queries and keys are staged in shared memory.
 // VEC 4: sizes are whole pieces of four channels and the buffers aligned to them; VEC 1: any sizes.  Which form runs
 // depends on the sizes and the alignment alone.  Dynamic shared memory: (staged channels + rotated runs + rot) floats.
+
+// Sine and cosine of position * frequency in 32-bit, the frequency given as the sum of two floats: what the product's
+// rounding and the frequency's own leave out (p times 2^-24 of a turn's radians, more than a score's other errors from a
+// few hundred positions on) is put back to first order.
+__device__ __forceinline__ void angle_sincos(float p, float f, float f_lo, float& sn, float& cs) {
+    const float a = __fmul_rn(p, f), e = fmaf(p, f_lo, fmaf(p, f, -a));
+    float s0, c0;
+    sincosf(a, &s0, &c0);
+    sn = fmaf(e, c0, s0);
+    cs = fmaf(-e, s0, c0);
+}
+
 template <typename T, int VEC>
 __global__ void __launch_bounds__(256)
 headnorm_rope_kvwrite_kernel(const float* __restrict__ rows, long long ld, const float* __restrict__ q_w,
-                             const float* __restrict__ k_w, float eps, const float* __restrict__ inv_freq, int rot,
+                             const float* __restrict__ k_w, float eps, const float* __restrict__ inv_freq,
+                             const float* __restrict__ inv_freq_lo, int rot,
                              const int* __restrict__ tok_seq, const int* __restrict__ tok_pos, T* __restrict__ q_out,
                              T* __restrict__ k_cache, T* __restrict__ v_cache, const int* __restrict__ block_table,
                              int table_stride, int n_pages, int page, int nh, int nkv, int maps, int hd, int vd, int own_kv,
@@ -667,7 +680,7 @@ headnorm_rope_kvwrite_kernel(const float* __restrict__ rows, long long ld, const
     pdl_wait();
     const int pos = tok_pos[n], seq = tok_seq[n];
     const float p = (float)pos;
-    for (int c = tid; c < half; c += blockDim.x) sincosf(p * inv_freq[c], &cs[half + c], &cs[c]);
+    for (int c = tid; c < half; c += blockDim.x) angle_sincos(p, inv_freq[c], inv_freq_lo[c], cs[half + c], cs[c]);
     int page_id = -1;
     if (own_kv) {
         page_id = block_table[(size_t)seq * table_stride + pos / page];
@@ -750,7 +763,8 @@ headnorm_rope_kvwrite_kernel(const float* __restrict__ rows, long long ld, const
 template <typename T, int LPR>
 __global__ void __launch_bounds__(128)
 headnorm_rope_kvwrite_lanes_kernel(const float* __restrict__ rows, long long ld, const float* __restrict__ q_w,
-                                   const float* __restrict__ k_w, float eps, const float* __restrict__ inv_freq, int rot,
+                                   const float* __restrict__ k_w, float eps, const float* __restrict__ inv_freq,
+                             const float* __restrict__ inv_freq_lo, int rot,
                                    const int* __restrict__ tok_seq, const int* __restrict__ tok_pos, T* __restrict__ q_out,
                                    T* __restrict__ k_cache, T* __restrict__ v_cache, const int* __restrict__ block_table,
                                    int table_stride, int n_pages, int page, int nh, int nkv, int maps, int hd, int vd,
@@ -776,7 +790,8 @@ headnorm_rope_kvwrite_lanes_kernel(const float* __restrict__ rows, long long ld,
 #pragma unroll
     for (int i = 0; i < 4; i++) {
         co[i] = 1.f, si[i] = 0.f;
-        if (turns) sincosf((float)pos * inv_freq[(first ? c : c - half) + i], &si[i], &co[i]);
+        const int k = (first ? c : c - half) + i;
+        if (turns) angle_sincos((float)pos, inv_freq[k], inv_freq_lo[k], si[i], co[i]);
         if (first) si[i] = -si[i];
     }
     const int partner = turns ? (first ? lane + half / 4 : lane - half / 4) : lane;
@@ -828,13 +843,14 @@ headnorm_rope_kvwrite_lanes_kernel(const float* __restrict__ rows, long long ld,
 }
 
 ESP_API int esp_headnorm_rope_kvwrite(const float* rows, long long ld, const float* q_w, const float* k_w, float eps,
-                                      const float* inv_freq, int rot, const int* tok_seq, const int* tok_pos, void* q_out,
+                                      const float* inv_freq, const float* inv_freq_lo, int rot, const int* tok_seq,
+                                      const int* tok_pos, void* q_out,
                                       void* k_cache, void* v_cache, int is_bf16, const int* block_table, int table_stride,
                                       int n_pages, int page, int n_tokens, int nh, int nkv, int maps, int hd, int vd,
                                       int own_kv, int* status, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (hd <= 0 || vd <= 0 || nkv <= 0 || nh <= 0 || maps <= 0 || page <= 0 || rot < 0 || rot > hd || rot % 2 != 0 ||
-        (rot > 0 && !inv_freq))
+        (rot > 0 && (!inv_freq || !inv_freq_lo)))
         return (int)cudaErrorInvalidValue;
     const long long runs = (long long)(nh + (own_kv ? nkv : 0)) * maps;
     const size_t smem = (size_t)(runs * hd + runs + rot) * sizeof(float);
@@ -847,7 +863,7 @@ ESP_API int esp_headnorm_rope_kvwrite(const float* rows, long long ld, const flo
         const dim3 grid(n_tokens, n_tokens <= 64 ? (unsigned)((runs + per_block - 1) / per_block) : 1u);
 #define ESP_HEADNORM_LANES(T, LPR)                                                                                           \
     esp_launch_pdl(ESP_PDL_SMALL, headnorm_rope_kvwrite_lanes_kernel<T, LPR>, grid, dim3(128), 0, stream, rows, ld, q_w, k_w, eps, \
-                   inv_freq, rot, tok_seq, tok_pos, (T*)q_out, (T*)k_cache, (T*)v_cache, block_table, table_stride, n_pages, page, \
+                   inv_freq, inv_freq_lo, rot, tok_seq, tok_pos, (T*)q_out, (T*)k_cache, (T*)v_cache, block_table, table_stride, n_pages, page, \
                    nh, nkv, maps, hd, vd, own_kv, status)
 #define ESP_HEADNORM_LANES_T(T)                       \
     do {                                              \
@@ -870,7 +886,7 @@ ESP_API int esp_headnorm_rope_kvwrite(const float* rows, long long ld, const flo
             if (e != cudaSuccess) return (int)e;                                                                          \
         }                                                                                                                 \
         esp_launch_pdl(ESP_PDL_SMALL, headnorm_rope_kvwrite_kernel<T, VEC>, dim3(n_tokens), dim3(threads), smem, stream,    \
-                       rows, ld, q_w, k_w, eps, inv_freq, rot, tok_seq, tok_pos, (T*)q_out, (T*)k_cache, (T*)v_cache,       \
+                       rows, ld, q_w, k_w, eps, inv_freq, inv_freq_lo, rot, tok_seq, tok_pos, (T*)q_out, (T*)k_cache, (T*)v_cache,       \
                        block_table, table_stride, n_pages, page, nh, nkv, maps, hd, vd, own_kv, status);                   \
     } while (0)
     if (is_bf16) {

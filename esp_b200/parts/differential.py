@@ -138,8 +138,8 @@ class DifferentialAttention(Part):
         linear(rt, h, self.w_in, rows)
         q = rt.ws.get("attn_q", (n, self.q_width), rt.dtype)
         pos = self.position
-        ops.headnorm_rope_kvwrite(rows, self.q_norm, self.k_norm, s.eps, pos.inv_freq if pos is not None else None,
-                                  pos.spec.rotary_dim if pos is not None else 0, ctx.tok_seq, ctx.tok_pos, q, layer.k, layer.v,
+        freq = (pos.inv_freq, pos.inv_freq_lo, pos.spec.rotary_dim) if pos is not None else (None, None, 0)
+        ops.headnorm_rope_kvwrite(rows, self.q_norm, self.k_norm, s.eps, *freq, ctx.tok_seq, ctx.tok_pos, q, layer.k, layer.v,
                                   table, layer.page, s.num_heads, s.num_kv_heads, 2, s.key_dim, s.value_dim, s.own_kv, rt.status)
         o = rt.ws.get("attn_o", (n, self.o_width), rt.dtype)
         gate = rows[:, self.gate_at:self.gate_at + s.num_heads] if s.head_gate else None

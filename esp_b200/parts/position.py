@@ -75,11 +75,16 @@ class RopeScaled(Part):
 
     def __init__(self, spec, rt):
         self.spec, self.rt = spec, rt
-        self.inv_freq = None
+        self.inv_freq = self.inv_freq_lo = None
         self.magnitude = 1.0
 
     def frequencies(self):
         """(float32 [rotary_dim / 2], magnitude), on the host."""
+        f, mag = self.exact_frequencies()
+        return f.astype(np.float32), mag
+
+    def exact_frequencies(self):
+        """The same in float64."""
         sp = self.spec
         i = np.arange(sp.rotary_dim // 2, dtype=np.float64)
         f = np.power(float(sp.theta), -2.0 * i / sp.rotary_dim)
@@ -92,12 +97,15 @@ class RopeScaled(Part):
             ramp = np.clip((i - lo) / max(hi - lo, 0.001), 0.0, 1.0)
             f = f / sp.factor * ramp + f * (1.0 - ramp)
             mag = 0.1 * float(np.log(sp.factor)) + 1.0
-        return f.astype(np.float32), float(mag)
+        return f, float(mag)
 
     def finalize(self):
         if self.inv_freq is None:
-            f, self.magnitude = self.frequencies()
-            self.inv_freq = torch.from_numpy(f).to(self.rt.device).contiguous()
+            f, self.magnitude = self.exact_frequencies()
+            hi = f.astype(np.float32)
+            self.inv_freq = torch.from_numpy(hi).to(self.rt.device).contiguous()
+            # what 32-bit leaves out of the frequencies, for kernels that take them as the sum of two
+            self.inv_freq_lo = torch.from_numpy((f - hi).astype(np.float32)).to(self.rt.device).contiguous()
 
 
 register("position", "rope_split_half", RopeSplitHalf)
