@@ -462,10 +462,7 @@ gemm_tc05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
                 const int f = t.f0 + pair * 32 + lane;
                 const bool f_ok = f < p.N;
                 bf16* out = reinterpret_cast<bf16*>(p.C);
-                // the plain form is the clamped one without limits, slope one and shift zero
                 const bool clamped = p.glu_limit > 0.f;
-                const float g_max = clamped ? p.glu_limit : INFINITY, g_alpha = clamped ? p.glu_alpha : 1.f;
-                const float u_shift = clamped ? p.glu_shift : 0.f;
                 int flip = 0;
                 for (int c0 = half * 32; c0 < t.n_tok; c0 += 64, flip ^= 1) {
                     float acc[32];
@@ -476,17 +473,24 @@ gemm_tc05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constan
 #pragma unroll
                     for (int i = 0; i < 16; i++) mine[i * 32 + lane] = is_up ? acc[i] : acc[16 + i];
                     asm volatile("bar.sync %0, 64;\n" ::"r"(1 + half * 2 + pair) : "memory");
+                    auto finish = [&](auto unit) {
 #pragma unroll
-                    for (int i = 0; i < 16; i++) {
-                        const float other = theirs[i * 32 + lane];
-                        const float own = is_up ? acc[16 + i] : acc[i];
-                        float g = is_up ? other : own, u = is_up ? own : other;
-                        g = fminf(g, g_max);
-                        u = fminf(fmaxf(u, -g_max), g_max) + u_shift;
-                        const int row = c0 + keep + i;
-                        if (f_ok && row < t.n_rows)
-                            out[(size_t)(t.row0 + row) * p.ldc + f] = __float2bfloat16_rn(__fdividef(g, 1.0f + __expf(-g_alpha * g)) * u);
-                    }
+                        for (int i = 0; i < 16; i++) {
+                            const float other = theirs[i * 32 + lane];
+                            const float own = is_up ? acc[16 + i] : acc[i];
+                            const float g = is_up ? other : own, u = is_up ? own : other;
+                            const int row = c0 + keep + i;
+                            if (f_ok && row < t.n_rows) out[(size_t)(t.row0 + row) * p.ldc + f] = __float2bfloat16_rn(unit(g, u));
+                        }
+                    };
+                    if (clamped)
+                        finish([&](float g, float u) {
+                            g = fminf(g, p.glu_limit);
+                            u = fminf(fmaxf(u, -p.glu_limit), p.glu_limit) + p.glu_shift;
+                            return __fdividef(g, 1.0f + __expf(-p.glu_alpha * g)) * u;
+                        });
+                    else
+                        finish([&](float g, float u) { return __fdividef(g, 1.0f + __expf(-g)) * u; });
                 }
             } else {
                 const int f = t.f0 + quad * 32 + lane;                    // this thread's output feature

@@ -405,8 +405,8 @@ router_logits_kernel(const TH* __restrict__ h, const TW* __restrict__ w_router, 
         for (int b = lane * 128; b < width * (int)sizeof(TW); b += 32 * 128)
             asm volatile("prefetch.global.L2 [%0];\n" ::"l"(reinterpret_cast<const char*>(wr) + b));
     pdl_wait();
-    h = behind_wait(h);
-    for (int i = tid; i < width; i += 256) hs[i] = to_f32(h[(size_t)n * width + i]);
+    const TH* h_now = behind_wait(h);
+    for (int i = tid; i < width; i += 256) hs[i] = to_f32(__ldg(h_now + (size_t)n * width + i));
     __syncthreads();
     if (e >= rows) return;
     float s[1];
@@ -705,7 +705,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ expert_out, const i
             for (int r = 0; r < top_k; r++) {
                 const int row = order[r];
                 if (row >= 0) {
-                    const float4 v = *reinterpret_cast<const float4*>(expert_out + (size_t)row * width + i);
+                    const float4 v = __ldg(reinterpret_cast<const float4*>(expert_out + (size_t)row * width + i));
                     acc.x += v.x; acc.y += v.y; acc.z += v.z; acc.w += v.w;
                 } else if (pass_w[r] != 0.f) {
                     const float4 v = *reinterpret_cast<const float4*>(ident + (size_t)t * width + i);
@@ -714,7 +714,7 @@ __global__ void moe_combine_kernel(const float* __restrict__ expert_out, const i
                 }
             }
             if (shared) {
-                const float4 v = *reinterpret_cast<const float4*>(shared + (size_t)t * width + i);
+                const float4 v = __ldg(reinterpret_cast<const float4*>(shared + (size_t)t * width + i));
                 acc.x += g * v.x; acc.y += g * v.y; acc.z += g * v.z; acc.w += g * v.w;
             }
             *reinterpret_cast<float4*>(y + (size_t)t * width + i) = acc;
@@ -737,8 +737,8 @@ __global__ void moe_combine_kernel(const float* __restrict__ expert_out, const i
 //   v = x[s] + y;  if (write_x) x[s] = v;  h[r] = v * rsqrt(mean(v^2) + eps) * gamma  (as add_rmsnorm)
 // with s = rows ? rows[r] : r.  Same operations in the same order as the two separate kernels, so the
 // results are the same bits.  Width a multiple of 4, at most 16384.  With gamma_y the combined row is normalised before it
-// is added: y <- y / sqrt(mean(y^2) + eps_y) * gamma_y.  gamma null: h[r] = v as it is; h null: the add alone.
-template <typename TH>
+// is added: y <- y / sqrt(mean(y^2) + eps_y) * gamma_y (POST), and then gamma null: h[r] = v as it is; h null: the add alone.
+template <typename TH, bool POST>
 __global__ void __launch_bounds__(1024)
 moe_combine_add_rmsnorm_kernel(const float* __restrict__ expert_out, const int* __restrict__ topk_ids,
                                const int* __restrict__ inverse, const float* __restrict__ gate,
@@ -794,7 +794,7 @@ moe_combine_add_rmsnorm_kernel(const float* __restrict__ expert_out, const int* 
             for (int j = 0; j < top_k; j++) {
                 const int row = order[j];
                 if (row >= 0) {
-                    const float4 e = reinterpret_cast<const float4*>(expert_out + (size_t)row * width)[q];
+                    const float4 e = __ldg(reinterpret_cast<const float4*>(expert_out + (size_t)row * width) + q);
                     acc.x += e.x; acc.y += e.y; acc.z += e.z; acc.w += e.w;
                 } else if (pass_w[j] != 0.f) {
                     const float4 e = reinterpret_cast<const float4*>(ident + t * width)[q];
@@ -803,21 +803,21 @@ moe_combine_add_rmsnorm_kernel(const float* __restrict__ expert_out, const int* 
                 }
             }
             if (shared) {
-                const float4 e = reinterpret_cast<const float4*>(shared + t * width)[q];
+                const float4 e = __ldg(reinterpret_cast<const float4*>(shared + t * width) + q);
                 acc.x += g * e.x; acc.y += g * e.y; acc.z += g * e.z; acc.w += g * e.w;
             }
             y[i] = acc;
-            if (gamma_y) ssy = fmaf(acc.w, acc.w, fmaf(acc.z, acc.z, fmaf(acc.y, acc.y, fmaf(acc.x, acc.x, ssy))));
+            if (POST) ssy = fmaf(acc.w, acc.w, fmaf(acc.z, acc.z, fmaf(acc.y, acc.y, fmaf(acc.x, acc.x, ssy))));
         }
     }
-    const float inv_y = gamma_y ? 1.0f / sqrtf(block_sum(ssy, scratch) / (float)width + eps_y) : 1.0f;
+    const float inv_y = POST ? 1.0f / sqrtf(block_sum(ssy, scratch) / (float)width + eps_y) : 1.0f;
     float ss = 0.f;
 #pragma unroll
     for (int i = 0; i < 4; i++) {
         const int q = threadIdx.x + i * blockDim.x;
         if (q < pieces) {
             float4 acc = y[i];
-            if (gamma_y) {
+            if (POST) {
                 const float4 gy = reinterpret_cast<const float4*>(gamma_y)[q];
                 acc.x = acc.x * inv_y * gy.x; acc.y = acc.y * inv_y * gy.y;
                 acc.z = acc.z * inv_y * gy.z; acc.w = acc.w * inv_y * gy.w;
@@ -832,8 +832,8 @@ moe_combine_add_rmsnorm_kernel(const float* __restrict__ expert_out, const int* 
             ss = fmaf(xv.w, xv.w, ss);
         }
     }
-    if (!h) return;
-    if (!gamma) {
+    if (POST && !h) return;
+    if (POST && !gamma) {
 #pragma unroll
         for (int i = 0; i < 4; i++) {
             const int q = threadIdx.x + i * blockDim.x;
@@ -997,19 +997,25 @@ ESP_API int esp_moe_combine_add_rmsnorm(const float* expert_out, const int* topk
                                         const float* topk_w, const float* ident, int n_real, const float* gamma_y,
                                         float eps_y, cudaStream_t stream) {
     if (n_rows <= 0) return 0;
-    if (top_k > MAX_TOPK || width % 4 != 0 || width > 16384 || (ident && !topk_w) || (h32 && (!h || !gamma))) return (int)cudaErrorInvalidValue;
+    if (top_k > MAX_TOPK || width % 4 != 0 || width > 16384 || (ident && !topk_w) || (h32 && (!h || !gamma)) || (!gamma_y && (!h || !gamma)))
+        return (int)cudaErrorInvalidValue;
     int threads = ((width / 4 + 3) / 4 + 31) / 32 * 32;
     // one piece per thread while a block can hold them: a row's sum then has the same order whatever else is in the
     // step (the 32-bit path relies on it).  Many rows rounded to bfloat16: four pieces per thread, smaller blocks,
     // more rows in flight per SM.
     if (width / 4 <= 1024 && !(h_is_bf16 && n_rows >= 256)) threads = (width / 4 + 31) / 32 * 32;
     const int early = esp_pdl_enabled(ESP_PDL_GROUPED) ? 0 : 1;
-    if (h_is_bf16)
-        esp_launch_pdl(ESP_PDL_SMALL, moe_combine_add_rmsnorm_kernel<bf16>, dim3(n_rows), dim3(threads), 0, stream, expert_out, topk_ids, inverse, gate, shared, x, gamma,
-                                                                            rows, (bf16*)h, h32, width, top_k, eps, write_x, early, topk_w, ident, n_real, gamma_y, eps_y);
-    else
-        esp_launch_pdl(ESP_PDL_SMALL, moe_combine_add_rmsnorm_kernel<float>, dim3(n_rows), dim3(threads), 0, stream, expert_out, topk_ids, inverse, gate, shared, x,
-                                                                             gamma, rows, (float*)h, h32, width, top_k, eps,
-                                                                             write_x, early, topk_w, ident, n_real, gamma_y, eps_y);
+#define ESP_COMBINE(TH, POST)                                                                                                \
+    esp_launch_pdl(ESP_PDL_SMALL, moe_combine_add_rmsnorm_kernel<TH, POST>, dim3(n_rows), dim3(threads), 0, stream, expert_out,  \
+                   topk_ids, inverse, gate, shared, x, gamma, rows, (TH*)h, h32, width, top_k, eps, write_x, early, topk_w,      \
+                   ident, n_real, gamma_y, eps_y)
+    if (h_is_bf16) {
+        if (gamma_y) ESP_COMBINE(bf16, true);
+        else ESP_COMBINE(bf16, false);
+    } else {
+        if (gamma_y) ESP_COMBINE(float, true);
+        else ESP_COMBINE(float, false);
+    }
+#undef ESP_COMBINE
     return esp_launch_status();
 }
