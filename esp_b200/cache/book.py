@@ -5,7 +5,8 @@ Nothing here touches a device.  A *slot* is a sequence's handle for the time it
 lives; a *page* holds PAGE consecutive positions of one sequence (for every
 layer of its group).  Layers with the same needs form a group with a pool of
 its own: a group of full-attention layers keeps every position, a group of
-windowed layers gives pages back once the window has passed them, a group whose
+windowed layers gives pages back once the window has passed them (all but those of
+the first positions, where a layer keeps them in sight), a group whose
 queries see their own block of positions only once the block is complete.
 """
 from __future__ import annotations
@@ -68,6 +69,7 @@ class KvLayout:
     values: bool = True              # False: one pool of rows only (a layer whose values are part of its key rows)
     value_dim: Optional[int] = None  # size of a value head where it differs from a key head's
     chunk: Optional[int] = None      # C: a query sees the keys of its own block of C positions (counted from 0) only
+    keep_first: int = 0              # with a window: the first so many positions are seen (and kept) besides
 
     @property
     def keeps_all(self) -> bool:
@@ -98,6 +100,11 @@ class GroupBook:
             return 0
         return max(0, length - self.layout.window + 1)
 
+    @property
+    def kept_pages(self) -> int:
+        """Pages at a sequence's start that a window with kept first positions never gives back."""
+        return 0 if self.layout.keeps_all else pages_for(self.layout.keep_first)
+
     def missing(self, slot: int, old_len: int, new_len: int) -> list:
         """Page indices that a step taking the slot from old_len to new_len
         needs and does not hold yet."""
@@ -107,7 +114,8 @@ class GroupBook:
             # nothing is ever given back before the slot closes: the table has no gaps
             return list(range(len(table), hi)) if hi > len(table) else []
         lo = self.first_needed(old_len) // PAGE
-        return [i for i in range(lo, hi) if i >= len(table) or table[i] < 0]
+        wanted = [*range(min(self.kept_pages, lo, hi)), *range(lo, hi)]
+        return [i for i in wanted if i >= len(table) or table[i] < 0]
 
     def reserve(self, slot: int, old_len: int, new_len: int) -> tuple:
         """Takes the pages the step needs.  Returns what ``cancel`` needs to undo it."""
@@ -139,10 +147,10 @@ class GroupBook:
         if not table or self.layout.keeps_all:
             return
         keep_from = self.first_needed(length) // PAGE
-        gone = [p for p in table[:keep_from] if p >= 0]
+        gone = [p for p in table[self.kept_pages:keep_from] if p >= 0]
         if gone:
             self.pool.give_back(gone)
-            for i in range(min(keep_from, len(table))):
+            for i in range(self.kept_pages, min(keep_from, len(table))):
                 table[i] = -1
 
     def release(self, slot: int) -> None:

@@ -8,8 +8,10 @@ from .vumedra import VumedraConfig
 from .migosun import MigosunConfig
 from .sebevik import SebevikConfig
 from .satavik import SatavikConfig
+from .galirax import GaliraxConfig
 
 __all__ = ["AttentionSpec", "BlockSpec", "DecayBonusRecurrenceSpec", "DenseFfnSpec", "DepthMixBlockSpec",
            "LatentAttentionSpec", "LowerBoundRecurrenceSpec", "ModelPlan", "MoeFfnSpec", "NormSpec", "PositionSpec",
-           "ScaledRopeSpec", "ScheduleEntry", "XieluFfnSpec", "ZusepelConfig", "VumedraConfig", "MigosunConfig", "SebevikConfig", "SatavikConfig", "config_from_dict", "config_from_json", "register_architecture",
+           "ScaledRopeSpec", "ScheduleEntry", "XieluFfnSpec", "ZusepelConfig", "VumedraConfig", "MigosunConfig", "SebevikConfig", "SatavikConfig", "GaliraxConfig",
+           "config_from_dict", "config_from_json", "register_architecture",
            "supported_architectures", "Qwen2MoeConfig"]

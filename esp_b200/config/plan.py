@@ -19,6 +19,7 @@ class NormSpec:
     width: int
     eps: float
     weight: str          # tensor name of the scale vector
+    bias: Optional[str] = None   # "layernorm": tensor name of the bias vector
 
 
 @dataclass(frozen=True)
@@ -104,7 +105,9 @@ class MoeFfnSpec:
     chosen among them returns its input (times its routing weight).  ``correction``: the name of a tensor with one
     number per router output that is added to the score for the choice only; the weights stay the scores.
     ``groups`` / ``keep_groups``: the router's outputs form that many equal groups of neighbours, a group's score is
-    its largest corrected score, and only experts of the best ``keep_groups`` groups can be chosen.
+    the sum of its ``group_top`` (1 or 2) largest corrected scores, and only experts of the best ``keep_groups`` groups can
+    be chosen.  ``sigmoid_scores``: scores are sigmoids of the logits, each expert by itself (with ``norm_topk`` the chosen
+    ones are divided by their sum plus 1e-20); ``weight_scale`` multiplies the routing weights.
     ``router_bias``: the name of a tensor with one number per router output that is added to the logits.
     ``chosen_softmax``: the experts with the largest logits, their weights a softmax over the chosen logits alone.
     ``glu`` / ``shared_glu``: (limit, alpha, shift) of gated units with clamped branches in place of SwiGLU, see
@@ -126,6 +129,9 @@ class MoeFfnSpec:
     chosen_softmax: bool = False
     glu: Optional[tuple] = None
     shared_glu: Optional[tuple] = None
+    sigmoid_scores: bool = False
+    group_top: int = 1
+    weight_scale: float = 1.0
 
 
 @dataclass(frozen=True)
@@ -424,15 +430,16 @@ class WideNormAttentionNames:
     q_norm: str = "q.norm"
     k_norm: str = "k.norm"
     sink: str = "sink"
+    bias: str = ".b"                 # after q, k or v
 
 
 @dataclass(frozen=True)
 class WideNormAttentionSpec:
     """Causal softmax attention over cached keys and values with grouped query heads, where the RMS norm of the
-    queries (and of the keys) runs over the whole projection, all heads at once, with a weight per channel, before the
-    rotation; the rotation (``position``, split-half pairs) covers the first channels of every head; scores are
+    queries (and of the keys) runs over the whole projection (with ``qkv_bias`` added), all heads at once, with a weight per
+    channel, before the rotation; the rotation (``position``: split-half or neighbour pairs) covers the first channels of every head; scores are
     multiplied by ``scale`` as given; keys and values may have different sizes.  Which keys a query sees: every
-    earlier one, the last ``window``, or (``chunk``) those of its own block of ``chunk`` positions counted from the
+    earlier one, the last ``window`` (and besides, with ``keep_first``, the sequence's first so many), or (``chunk``) those of its own block of ``chunk`` positions counted from the
     sequence's start.  ``learned_sink``: the softmax's denominator holds one more term exp(sink_h), a learned number
     per head that is not scaled and carries no value."""
     hidden: int
@@ -445,10 +452,12 @@ class WideNormAttentionSpec:
     learned_sink: bool
     window: Optional[int]
     chunk: Optional[int]
-    position: Optional[ScaledRopeSpec]
+    position: Optional[Any]          # ScaledRopeSpec or NeighbourRopeSpec
     prefix: str
     kind: str = "attention_widenorm"
     names: WideNormAttentionNames = WideNormAttentionNames()
+    qkv_bias: bool = False
+    keep_first: int = 0
 
 
 @dataclass(frozen=True)
@@ -524,6 +533,32 @@ class ChannelDecayAttentionSpec:
 
 
 @dataclass(frozen=True)
+class FixedDecayAttentionNames:
+    q: str = "q"
+    k: str = "k"
+    v: str = "v"
+    o: str = "o"
+    gate: str = "g"
+    norm: str = "norm"
+
+
+@dataclass(frozen=True)
+class FixedDecayAttentionSpec:
+    """Linear attention with one fixed decay per head: q, k and v are SiLUs of their projections (no other scale),
+    S_t = decay_h S_(t-1) + k_t v_t^T, o_t = S_t^T q_t per head; the heads' concatenation is RMS-normed as one row with a
+    weight per channel, multiplied by sigmoid(W_g h), then W_o."""
+    hidden: int
+    num_heads: int
+    key_dim: int
+    value_dim: int
+    decay: tuple                     # one number per head
+    eps: float
+    prefix: str
+    kind: str = "lightning"
+    names: FixedDecayAttentionNames = FixedDecayAttentionNames()
+
+
+@dataclass(frozen=True)
 class ParallelMixerSpec:
     """Several mixers side by side on the same input; the result is sum_i scales[i] * branches[i](h)."""
     hidden: int
@@ -576,10 +611,15 @@ class HyperConnectionBlockSpec:
 @dataclass(frozen=True)
 class NeighbourRopeSpec:
     """Rotary encoding over neighbouring channels: of the first ``rotary_dim`` channels of a head, channel 2i is
-    rotated with channel 2i + 1 by the angle position * theta^(-2i / rotary_dim)."""
+    rotated with channel 2i + 1 by the angle position * f_i, f_i = theta^(-2i / rotary_dim).  With ``factor`` slow frequencies
+    are slowed further by their wavelength l = 2 pi / f: f stays where l < original / high, is divided by the factor where
+    l > original / low, and in between is (1 - s) f / factor + s f with s = (original / l - low) / (high - low)."""
     rotary_dim: int
     theta: float
-    factor: Optional[float] = None   # no interpolation in this form
+    factor: Optional[float] = None
+    original: Optional[float] = None
+    low: Optional[float] = None
+    high: Optional[float] = None
     kind: str = "rope_neighbour_pairs"
 
 
@@ -704,6 +744,15 @@ class OutputNormBlockSpec:
     mixer_post_norm: NormSpec
     ffn_post_norm: Optional[NormSpec]
     kind: str = "output_norm_residual"
+
+
+@dataclass(frozen=True)
+class ParallelBlockSpec:
+    """x += mixer(h) + ffn(h) with h = norm(x): one norm, and both sublayers read its output.  ``ffn`` None: a mixer only."""
+    mixer: Any
+    ffn: Any
+    norm: NormSpec
+    kind: str = "parallel_residual"
 
 
 @dataclass(frozen=True)

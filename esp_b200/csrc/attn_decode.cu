@@ -9,13 +9,13 @@
 // ascending order.  Which splits a row has depends on its position (and window)
 // alone, so the result does not depend on the batch around it.
 //
-// The query at position a sees key j iff j <= a and (window == 0 or a - j < window);
-// score = dot(q, k) / sqrt(hd).
+// The query at position a sees key j iff j <= a and (window == 0 or a - j < window or j < keep);
+// score = dot(q, k) / sqrt(hd).  Heads narrower than the kernel's tiles are read with zeros behind them.
 //
 // MAPS 2 is the differential form: every head has two attention maps over the same values, and a key head's row in the
 // cache holds the keys of both maps side by side.  A block's 16 rows are then up to eight heads times two maps; a
 // row's query is padded with zeros over the other map's channels, so both maps share the pages and the products of a
-// block, and the combine ends with the difference of the two, its norm and the head's gate (DiffParams).
+// block, and the combine ends with the difference of the two, its norm and the head's gate (HeadParams).
 #include <cuda.h>
 
 #include "common.cuh"
@@ -89,10 +89,10 @@ __device__ __forceinline__ const bf16* tile_at(const bf16* tile, int r, int d) {
     return tile + (d >> 6) * (PAGE_KEYS * 64) + r * 64 + ((((d & 63) >> 3) ^ (r & 7)) << 3);
 }
 
-// The differential form's constants: scores s become softcap tanh(s / softcap) (0: as they are); per head
+// Sizes of a head, both multiples of 8, and the differential form's constants: scores s become softcap tanh(s / softcap) (0: as they are); per head
 // o = a_1 - lambda a_2, then o / sqrt(mean(o^2) + eps) * out_scale * sigmoid(gate[row * ldg + head]) (gate null: no gate).
-struct DiffParams {
-    int key_dim, value_dim;         // channels of one map's key, of a value; both multiples of 8
+struct HeadParams {
+    int key_dim, value_dim;         // channels of (one map's) key, of a value
     float softcap, lambda, eps, out_scale;
     const float* gate;
     long long ldg;
@@ -111,7 +111,7 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
                       int* __restrict__ counters, const int* __restrict__ tok_seq, const int* __restrict__ tok_pos,
                       const int* __restrict__ seq_past, const int* __restrict__ block_table, int table_stride, int n_pages,
                       int page, int nh, int nkv, int window, int split_keys, int n_splits, float score_scale, int sink,
-                      const float* __restrict__ sink_vals, int chunk, int* __restrict__ status, DiffParams df) {
+                      const float* __restrict__ sink_vals, int chunk, int keep, int* __restrict__ status, HeadParams df) {
     pdl_trigger();
     constexpr int ITEM_K = PAGE_KEYS * HDK, ITEM_V = PAGE_KEYS * HDV;
     constexpr int NBW = HDV / 32;                   // 8-column blocks of the head that one warp accumulates
@@ -130,10 +130,16 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
     const int kvh = blockIdx.y / blocks_per_kv, h0 = kvh * group + (blockIdx.y % blocks_per_kv) * MMA_HEADS;
     const int heads = min(MMA_HEADS, (kvh + 1) * group - h0);
     const int pos = tok_pos[n], seq = tok_seq[n];
-    const int lo = first_visible_key(pos, window, chunk);
-    const int j0 = max(lo, split * split_keys), j1 = min(pos, split * split_keys + split_keys - 1);
-    if (j0 > j1) return;
-    const int first_page = j0 / PAGE_KEYS, n_pg = j1 / PAGE_KEYS - first_page + 1, n_items = 2 * n_pg;
+    // the split's keys: kept first positions [a0, a1], then the window's [b0, b1]; either may be empty.  A page that
+    // holds both is read once.
+    const VisibleKeys seen = visible_keys(pos, window, chunk, keep);
+    const int a0 = split * split_keys, a1 = min(seen.kept, a0 + split_keys) - 1;
+    const int b0 = max(seen.lo, a0), b1 = min(pos, a0 + split_keys - 1);
+    if (a0 > a1 && b0 > b1) return;
+    const int first_a = a0 / PAGE_KEYS, n_a = a0 <= a1 ? a1 / PAGE_KEYS - first_a + 1 : 0;
+    const int first_b = max(b0 / PAGE_KEYS, n_a > 0 ? first_a + n_a : 0), n_b = b0 <= b1 ? max(b1 / PAGE_KEYS - first_b + 1, 0) : 0;
+    const int n_pg = n_a + n_b, n_items = 2 * n_pg, j1 = b0 <= b1 ? b1 : a1;
+    auto page_of = [&](int i) { return i < n_a ? first_a + i : first_b + i - n_a; };
 
     if (tid < MMA_HEADS) {
         m_s[tid] = -INFINITY;
@@ -145,7 +151,7 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
     }
     auto issue = [&](int item) {
         const int slot = item % RING;
-        int pg = block_table[(size_t)seq * table_stride + first_page + item / 2];
+        int pg = block_table[(size_t)seq * table_stride + page_of(item / 2)];
         const bool ok = pg >= 0 && pg < n_pages;
         if (!ok) atomicOr(status, ESP_STATUS_BAD_INDEX);
         item_ok[slot] = ok ? 1 : 0;
@@ -196,15 +202,17 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
             qa[kk][3] = piece(q1, c + 8, g8 + 8 < heads);
         }
     } else {
-        const bf16* q0 = q_now + ((size_t)n * nh + h0 + g8) * HDK;
-        const bf16* q1 = q_now + ((size_t)n * nh + h0 + g8 + 8) * HDK;
+        const int kd = df.key_dim;
+        const bf16* q0 = q_now + ((size_t)n * nh + h0 + g8) * kd;
+        const bf16* q1 = q0 + (size_t)8 * kd;
+        auto piece = [&](const bf16* row, int c, bool live) { return live && c < kd ? *reinterpret_cast<const unsigned*>(row + c) : 0u; };
 #pragma unroll
         for (int kk = 0; kk < HDK / 16; kk++) {
             const int c = kk * 16 + tg * 2;
-            qa[kk][0] = g8 < heads ? *reinterpret_cast<const unsigned*>(q0 + c) : 0u;
-            qa[kk][1] = g8 + 8 < heads ? *reinterpret_cast<const unsigned*>(q1 + c) : 0u;
-            qa[kk][2] = g8 < heads ? *reinterpret_cast<const unsigned*>(q0 + c + 8) : 0u;
-            qa[kk][3] = g8 + 8 < heads ? *reinterpret_cast<const unsigned*>(q1 + c + 8) : 0u;
+            qa[kk][0] = piece(q0, c, g8 < heads);
+            qa[kk][1] = piece(q1, c, g8 + 8 < heads);
+            qa[kk][2] = piece(q0, c + 8, g8 < heads);
+            qa[kk][3] = piece(q1, c + 8, g8 + 8 < heads);
         }
     }
     __syncthreads();
@@ -212,7 +220,7 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
         for (; issued < min(RING, n_items); issued++) issue(issued);
     }
 
-    const float root = sqrtf((float)HDK), cap_unit = MAPS == 2 && df.softcap > 0.f ? score_scale / df.softcap : 0.f;
+    const float root = sqrtf((float)df.key_dim), cap_unit = MAPS == 2 && df.softcap > 0.f ? score_scale / df.softcap : 0.f;
     float o[NBW][4];
 #pragma unroll
     for (int i = 0; i < NBW; i++)
@@ -221,7 +229,7 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
     bool failed = false;
 
     for (int pi = 0; pi < n_pg; pi++) {
-        const int key0 = (first_page + pi) * PAGE_KEYS;
+        const int key0 = page_of(pi) * PAGE_KEYS;
         const int item_k = 2 * pi, slot_k = item_k % RING;
         if (__syncthreads_or(!mbar_wait(&full_bar[slot_k], (item_k / RING) & 1))) { failed = true; break; }
         const bf16* kp = ring;
@@ -244,7 +252,7 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
 #pragma unroll
             for (int j = 0; j < 4; j++) {
                 const int t = warp * 16 + nb * 8 + tg * 2 + (j & 1), key = key0 + t;
-                const bool live = page_ok && key >= j0 && key <= j1;
+                const bool live = page_ok && key <= j1 && seen.sees(key);
                 float sv;
                 if (MAPS == 2) sv = df.softcap > 0.f ? softcap_score(sc[nb][j], cap_unit, df.softcap) : sc[nb][j] * score_scale;
                 else sv = score_scale > 0.f ? sc[nb][j] * score_scale : sc[nb][j] / root;
@@ -343,11 +351,15 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
     __shared__ int is_last;
     __threadfence();
     __syncthreads();
-    const int s0 = lo / split_keys, s1 = pos / split_keys;
+    // the row's splits in ascending order: those that hold kept first positions, then those of the window.  The i-th of
+    // them is split i, or i + gap from the window's first on.
+    const int s_kept = (seen.kept + split_keys - 1) / split_keys, gap = max(seen.lo / split_keys - s_kept, 0);
+    const int n_live = pos / split_keys - gap + 1;
+    auto split_at = [&](int i) { return i < s_kept ? i : i + gap; };
     if (tid == 0) {
         int* c = counters + (size_t)n * gridDim.y + blockIdx.y;
         const int done = atomicAdd(c, 1);
-        is_last = done == s1 - s0;
+        is_last = done == n_live - 1;
         if (is_last) *c = 0;
     }
     __syncthreads();
@@ -365,7 +377,7 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
         const float* ml = part_ml + ((size_t)n * nh + h0 + g) * n_splits * 2;
         const float* po = part_o + ((size_t)n * nh + h0 + g) * n_splits * HDV;
         float mx = -INFINITY;
-        for (int sp = s0 + lane; sp <= s1; sp += 32) mx = fmaxf(mx, __ldcg(ml + 2 * sp));
+        for (int i = lane; i < n_live; i += 32) mx = fmaxf(mx, __ldcg(ml + 2 * split_at(i)));
 #pragma unroll
         for (int off = 16; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
         // one more key without a value, of score zero or of the head's own score
@@ -374,23 +386,25 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
         float denom = sink ? expf(sink_score - mx) : 0.f, num[NV][2];
 #pragma unroll
         for (int j = 0; j < NV; j++) num[j][0] = num[j][1] = 0.f;
-        for (int c0 = s0; c0 <= s1; c0 += WCH) {
-            const int cn = min(WCH, s1 + 1 - c0);
+        for (int c0 = 0; c0 < n_live; c0 += WCH) {
+            const int cn = min(WCH, n_live - c0);
             __syncwarp();                                  // the pass (or head) before this one has been read
             for (int i = lane; i < cn; i += 32) {
-                const float m_sp = __ldcg(ml + 2 * (c0 + i));
+                const float* ml_sp = ml + 2 * split_at(c0 + i);
+                const float m_sp = __ldcg(ml_sp);
                 w_w[i] = m_sp == -INFINITY ? 0.f : expf(m_sp - mx);
-                l_w[i] = __ldcg(ml + 2 * (c0 + i) + 1);
+                l_w[i] = __ldcg(ml_sp + 1);
             }
             __syncwarp();
-            const float* pc = po + (size_t)c0 * HDV + lane * 2;
+            const float* pc = po + lane * 2;
 #pragma unroll 8
             for (int i = 0; i < cn; i++) {
                 const float w = w_w[i];
+                const float* pi = pc + (size_t)split_at(c0 + i) * HDV;
                 denom += l_w[i] * w;
 #pragma unroll
                 for (int j = 0; j < NV; j++) {
-                    const float2 v = __ldcg(reinterpret_cast<const float2*>(pc + (size_t)i * HDV + j * 64));
+                    const float2 v = __ldcg(reinterpret_cast<const float2*>(pi + j * 64));
                     num[j][0] += v.x * w;
                     num[j][1] += v.y * w;
                 }
@@ -432,11 +446,14 @@ attn_split_mma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_co
         for (int g = warp; g < heads; g += THREADS / 32) {
             float res[NV][2];
             combine_row(g, res);
-            bf16* orow = out + ((size_t)n * nh + h0 + g) * HDV + lane * 2;
-    #pragma unroll
-            for (int j = 0; j < NV; j++)
-                *reinterpret_cast<__nv_bfloat162*>(orow + j * 64) =
-                    __nv_bfloat162(__float2bfloat16_rn(res[j][0]), __float2bfloat16_rn(res[j][1]));
+            bf16* orow = out + ((size_t)n * nh + h0 + g) * df.value_dim;
+#pragma unroll
+            for (int j = 0; j < NV; j++) {
+                const int d = j * 64 + lane * 2;
+                if (d < df.value_dim)
+                    *reinterpret_cast<__nv_bfloat162*>(orow + d) =
+                        __nv_bfloat162(__float2bfloat16_rn(res[j][0]), __float2bfloat16_rn(res[j][1]));
+            }
         }
     }
 }
@@ -470,14 +487,13 @@ template <int HDK, int HDV, int MAPS>
 int launch_split_mma(int split, const bf16* q, const bf16* k, const bf16* v, bf16* out, float* po, float* pml, int* counters,
                      const int* tok_seq, const int* tok_pos, const int* seq_past, const int* table, int stride, int n_pages, int page,
                      int n_tokens, int nh, int nkv, int window, int n_splits, float score_scale, int sink,
-                     const float* sink_vals, int chunk, int* status,
-                     cudaStream_t stream, const DiffParams& df = DiffParams{}) {
+                     const float* sink_vals, int chunk, int keep, int* status, cudaStream_t stream, const HeadParams& df) {
     CUtensorMap map_k, map_v;
     const unsigned long long rows = (unsigned long long)n_pages * nkv * PAGE_KEYS;
     // heads narrower than the kernel's tiles are read with zeros behind them
-    int rc = make_cache_map(&map_k, k, rows, MAPS == 2 ? 2 * df.key_dim : HDK);
+    int rc = make_cache_map(&map_k, k, rows, MAPS * df.key_dim);
     if (rc) return rc;
-    rc = make_cache_map(&map_v, v, rows, MAPS == 2 ? df.value_dim : HDV);
+    rc = make_cache_map(&map_v, v, rows, df.value_dim);
     if (rc) return rc;
     const size_t dyn = (size_t)PAGE_KEYS * (HDK + HDV) * sizeof(bf16) + 1024;
     static bool raised[64] = {false};              // per device: the attribute belongs to the device's context
@@ -492,7 +508,7 @@ int launch_split_mma(int split, const bf16* q, const bf16* k, const bf16* v, bf1
     dim3 grid(n_tokens, nkv * ((group + MMA_HEADS - 1) / MMA_HEADS), n_splits);
     esp_launch_pdl(ESP_PDL_ATTENTION, attn_split_mma_kernel<HDK, HDV, MAPS>, dim3(grid), dim3(THREADS), dyn, stream, map_k, map_v, q, out, po, pml,
                    counters, tok_seq, tok_pos, seq_past, table, stride, n_pages, page, nh, nkv, window, split, n_splits, score_scale,
-                   sink, sink_vals, chunk, status, df);
+                   sink, sink_vals, chunk, keep, status, df);
     return esp_launch_status();
 }
 }  // namespace
@@ -500,24 +516,30 @@ int launch_split_mma(int split, const bf16* q, const bf16* k, const bf16* v, bf1
 // Scratch: part_o float [n_tokens, nh, n_splits, hd], part_ml float [n_tokens, nh, n_splits, 2];
 // counters int [n_tokens * head groups], all zero when the call starts (the kernel leaves them zero);
 // split: key positions per block, a multiple of 64 (the caller picks: short splits when there are few rows, so
-// that every SM still gets blocks); n_splits >= ceil(longest sequence / split).  Head sizes 64, 128, 192, 256; pages of 64 positions or any
-// size; any head counts with nh % nkv == 0.  ``seq_past`` (may be null): per sequence of the step, the positions
+// that every SM still gets blocks); n_splits >= ceil(longest sequence / split).  Keys of hd and values of vd channels (0: hd),
+// multiples of 8 up to 256, both padded to the larger one's multiple of 64, which is part_o's last size; pages of 64 positions;
+// any head counts with nh % nkv == 0.  ``keep`` (with a window): the first ``keep`` positions of a sequence are seen besides.  ``seq_past`` (may be null): per sequence of the step, the positions
 // that were cached before it; with it, blocks whose keys are all older start their loads without waiting for the
 // kernel before this one.  score_scale > 0 multiplies the scores (else they are divided by sqrt(hd)); ``sink``: the
 // softmax's denominator holds one more term exp(0).
 ESP_API int esp_attn_decode(const void* q, const void* k_cache, const void* v_cache, void* out, float* part_o,
                             float* part_ml, int* counters, const int* tok_seq, const int* tok_pos, const int* seq_past,
                             const int* block_table, int table_stride, int n_pages, int page, int n_tokens, int nh, int nkv,
-                            int hd, int window, int split, int n_splits, float score_scale, int sink, const float* sink_vals,
-                            int chunk, int* status, cudaStream_t stream) {
+                            int hd, int vd, int window, int split, int n_splits, float score_scale, int sink,
+                            const float* sink_vals, int chunk, int keep, int* status, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (nkv <= 0 || nh % nkv != 0 || n_splits <= 0 || n_splits > 65535 || nh > 65535 || split < PAGE_KEYS || split % PAGE_KEYS != 0 ||
-        page != PAGE_KEYS)
+        page != PAGE_KEYS || hd <= 0 || hd % 8 != 0)
         return (int)cudaErrorInvalidValue;
+    if (vd <= 0) vd = hd;
+    if (vd % 8 != 0 || keep < 0) return (int)cudaErrorInvalidValue;
+    HeadParams head{};
+    head.key_dim = hd;
+    head.value_dim = vd;
 #define ESP_HD(HD) return launch_split_mma<HD, HD, 1>(split, (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache, (bf16*)out, part_o, \
                                                part_ml, counters, tok_seq, tok_pos, seq_past, block_table, table_stride, n_pages, \
-                                               page, n_tokens, nh, nkv, window, n_splits, score_scale, sink, sink_vals, chunk, status, stream)
-    switch (hd) {
+                                               page, n_tokens, nh, nkv, window, n_splits, score_scale, sink, sink_vals, chunk, keep, status, stream, head)
+    switch (((hd > vd ? hd : vd) + 63) / 64 * 64) {
         case 64: ESP_HD(64);
         case 128: ESP_HD(128);
         case 192: ESP_HD(192);
@@ -542,11 +564,11 @@ ESP_API int esp_attn_decode_diff(const void* q, const void* k_cache, const void*
         split % PAGE_KEYS != 0 || page != PAGE_KEYS || key_dim <= 0 || key_dim % 8 != 0 || key_dim > 128 || value_dim <= 0 ||
         value_dim % 8 != 0 || value_dim > 256 || !(score_scale > 0.f))
         return (int)cudaErrorInvalidValue;
-    const DiffParams df{key_dim, value_dim, softcap, lambda, eps, out_scale, gate, ldg};
+    const HeadParams df{key_dim, value_dim, softcap, lambda, eps, out_scale, gate, ldg};
 #define ESP_DIFF(HDK, HDV)                                                                                                  \
     return launch_split_mma<HDK, HDV, 2>(split, (const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache, (bf16*)out, part_o, \
                                          part_ml, counters, tok_seq, tok_pos, seq_past, block_table, table_stride, n_pages, page, \
-                                         n_tokens, 2 * heads, nkv, window, n_splits, score_scale, 0, nullptr, chunk, status,     \
+                                         n_tokens, 2 * heads, nkv, window, n_splits, score_scale, 0, nullptr, chunk, 0, status,  \
                                          stream, df)
 #define ESP_DIFF_V(HDK)                          \
     do {                                         \
@@ -607,5 +629,5 @@ extern "C" int esp_attn_decode_noalloc(const void* q, const void* k_cache, const
     float* part_ml = part_o + (size_t)n_tokens * nh * n_splits * hd;
     int* counters = reinterpret_cast<int*>(noalloc_scratch_of_device[device] + esp_attn_decode_noalloc_capacity());
     return esp_attn_decode(q, k_cache, v_cache, out, part_o, part_ml, counters, tok_seq, tok_pos, nullptr, block_table, table_stride,
-                           n_pages, page, n_tokens, nh, nkv, hd, window, split, n_splits, 0.f, 0, nullptr, 0, status, stream);
+                           n_pages, page, n_tokens, nh, nkv, hd, hd, window, split, n_splits, 0.f, 0, nullptr, 0, 0, status, stream);
 }

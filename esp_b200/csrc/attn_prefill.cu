@@ -13,7 +13,8 @@
 // Key heads up to HDK and value heads up to HDV (64 or 128 each; keys and values may differ in size) are padded
 // with zeros to that in shared memory; both must be multiples of 8.  The page size is 64.  The scores are
 // dot / sqrt(hd), or dot * scale when a scale is given.  With ``sink`` the softmax's denominator holds one more
-// term, a key of score zero without a value: the running maximum starts at 0 and the running sum at 1.
+// term, a key of score zero without a value: the running maximum starts at 0 and the running sum at 1.  ``keep`` (with a
+// window): the first ``keep`` positions of a sequence are seen besides; the blocks of keys that hold them come first.
 #include "common.cuh"
 
 namespace {
@@ -54,7 +55,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache
                     bf16* __restrict__ out, const int* __restrict__ tile_seq, const int* __restrict__ tile_first,
                     const int* __restrict__ seq_start, const int* __restrict__ seq_past,
                     const int* __restrict__ block_table, int table_stride, int n_pages, int nh, int nkv, int hd,
-                    int vd, float scale, int sink, const float* __restrict__ sink_vals, int window, int chunk,
+                    int vd, float scale, int sink, const float* __restrict__ sink_vals, int window, int chunk, int keep,
                     int* __restrict__ status) {
     constexpr int LDS = HDK + 8;                     // row stride in elements: 16 bytes of padding against bank conflicts
     constexpr int LDV = HDV + 8;
@@ -87,7 +88,9 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache
     cp_async_commit();
 
     const int key_lo = first_visible_key(pos0, window, chunk);         // first key any row of the tile sees
-    const int blk_lo = key_lo / BN, blk_hi = pos_last / BN;
+    // blocks of keys: those of the kept first positions that lie ahead of the window's, then the window's
+    const int blk_lo = key_lo / BN, n_kept = min((keep + BN - 1) / BN, blk_lo), n_blk = n_kept + pos_last / BN - blk_lo + 1;
+    auto block_of = [&](int i) { return i < n_kept ? i : blk_lo + i - n_kept; };
 
     auto load_kv = [&](int blk, int buf) {
         int pg = block_table[(size_t)seq * table_stride + blk];
@@ -110,7 +113,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache
         }
         cp_async_commit();
     };
-    load_kv(blk_lo, 0);
+    load_kv(block_of(0), 0);
 
     // ---- query fragments of this warp's 16 rows stay in registers
     cp_async_wait<1>();
@@ -137,10 +140,10 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache
     const int my_first[2] = {first_visible_key(my_pos[0], window, chunk), first_visible_key(my_pos[1], window, chunk)};
     const int warp_first = first_visible_key(pos0 + warp * 16 + 15, window, chunk);   // of the warp's last row
 
-    for (int blk = blk_lo; blk <= blk_hi; blk++) {
-        const int buf = (blk - blk_lo) & 1;
-        if (blk < blk_hi) load_kv(blk + 1, buf ^ 1);
-        if (blk < blk_hi) cp_async_wait<1>(); else cp_async_wait<0>();
+    for (int i = 0; i < n_blk; i++) {
+        const int buf = i & 1, blk = block_of(i);
+        if (i + 1 < n_blk) load_kv(block_of(i + 1), buf ^ 1);
+        if (i + 1 < n_blk) cp_async_wait<1>(); else cp_async_wait<0>();
         __syncthreads();
         const bf16* kb = k_s + buf * BN * LDS;
         const bf16* vb = v_s + buf * BN * LDV;
@@ -174,7 +177,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache
                 const int key = key0 + nb * 8 + tg * 2 + (j & 1);
                 float v = scale > 0.f ? s[nb][j] * scale : s[nb][j] / root;
                 if (edge) {
-                    const bool seen = key <= my_pos[r] && key >= my_first[r];
+                    const bool seen = key <= my_pos[r] && (key >= my_first[r] || key < keep);
                     if (!seen) v = -INFINITY;
                 }
                 s[nb][j] = v;
@@ -254,7 +257,7 @@ attn_prefill_kernel(const bf16* __restrict__ q, const bf16* __restrict__ k_cache
 template <int HDK, int HDV>
 int launch(const bf16* q, const bf16* k, const bf16* v, bf16* out, const int* tile_seq, const int* tile_first,
            const int* seq_start, const int* seq_past, const int* table, int stride, int n_pages, int n_tiles, int nh,
-           int nkv, int hd, int vd, float scale, int sink, const float* sink_vals, int window, int chunk, int* status,
+           int nkv, int hd, int vd, float scale, int sink, const float* sink_vals, int window, int chunk, int keep, int* status,
            cudaStream_t stream) {
     static_assert(BM <= BN, "the queries borrow a key buffer");
     const size_t smem = (size_t)(2 * BN) * ((HDK + 8) + (HDV + 8)) * sizeof(bf16);
@@ -267,7 +270,7 @@ int launch(const bf16* q, const bf16* k, const bf16* v, bf16* out, const int* ti
     dim3 grid(n_tiles, nh);
     attn_prefill_kernel<HDK, HDV><<<grid, THREADS, smem, stream>>>(q, k, v, out, tile_seq, tile_first, seq_start, seq_past,
                                                                    table, stride, n_pages, nh, nkv, hd, vd, scale, sink,
-                                                                   sink_vals, window, chunk, status);
+                                                                   sink_vals, window, chunk, keep, status);
     return esp_launch_status();
 }
 }  // namespace
@@ -278,7 +281,7 @@ int launch(const bf16* q, const bf16* k, const bf16* v, bf16* out, const int* ti
 ESP_API int esp_attn_prefill(const void* q, const void* k_cache, const void* v_cache, void* out, const int* tile_seq,
                              const int* tile_first, const int* seq_start, const int* seq_past, const int* block_table,
                              int table_stride, int n_pages, int page, int n_tiles, int nh, int nkv, int hd, int vd,
-                             float scale, int sink, const float* sink_vals, int window, int chunk, int* status,
+                             float scale, int sink, const float* sink_vals, int window, int chunk, int keep, int* status,
                              cudaStream_t stream) {
     if (n_tiles <= 0) return 0;
     if (vd <= 0) vd = hd;
@@ -287,7 +290,7 @@ ESP_API int esp_attn_prefill(const void* q, const void* k_cache, const void* v_c
 #define ESP_FLASH(HDK_, HDV_)                                                                                              \
     return launch<HDK_, HDV_>((const bf16*)q, (const bf16*)k_cache, (const bf16*)v_cache, (bf16*)out, tile_seq, tile_first, \
                               seq_start, seq_past, block_table, table_stride, n_pages, n_tiles, nh, nkv, hd, vd, scale, sink, \
-                              sink_vals, window, chunk, status, stream)
+                              sink_vals, window, chunk, keep, status, stream)
     if (hd <= 64 && vd <= 64) ESP_FLASH(64, 64);
     if (hd <= 64) ESP_FLASH(64, 128);
     if (vd <= 64) ESP_FLASH(128, 64);

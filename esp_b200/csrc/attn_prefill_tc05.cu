@@ -30,7 +30,11 @@
 // traffic from L2): with 16 products of 128 x 128 x 16 to a block the thread that issues them is busy for
 // most of a block's time.
 //
-// Head sizes 64 and 128.  The page size is 64.  Rows of the tile beyond the sequence's new tokens are
+// ``keep`` (with a window): the first ``keep`` positions of a sequence are seen besides; an item's blocks of keys are then
+// those of the kept positions ahead of the window's blocks, and the window's.
+//
+// Keys and values of up to 128 channels, multiples of 8, are padded with zeros (by the loads) to HD = 64 or 128.  The page
+// size is 64.  Rows of the tile beyond the sequence's new tokens are
 // computed and not stored; keys beyond a row's position are masked before the maximum is taken.
 #include "tc05.cuh"
 
@@ -54,6 +58,8 @@ struct AttnParams {
     int sink;         // the softmax's denominator holds one more term, a key of score zero without a value
     const float* sink_vals;   // with sink: the term is exp(sink_vals[head]) instead (a number per head, not scaled); may be null
     int chunk;        // > 0: a query sees the keys of its own block of ``chunk`` positions (counted from 0) only
+    int keep;         // with a window: the first ``keep`` positions are seen besides
+    int kd, vd;       // channels of a key, of a value
 };
 
 // instruction descriptor: bfloat16 x bfloat16 -> float, M = 128, N = n, A K-major, B K-major or MN-major
@@ -96,7 +102,8 @@ __device__ __forceinline__ void named_sync(int id, int count) {
 
 // the tile of 128 query rows and the head that a block works on
 struct Item {
-    int seq, h, kvh, row0, rows, pos0, pos_last, blk_lo, nb, page_lo;
+    int seq, h, kvh, row0, rows, pos0, pos_last, blk_lo, nb, page_lo, n_kept;
+    __device__ __forceinline__ int block(int j) const { return j < n_kept ? j : blk_lo + j - n_kept; }   // the item's j-th block of keys
 };
 __device__ __forceinline__ Item load_item(const AttnParams& p, int item) {
     Item it;
@@ -112,7 +119,8 @@ __device__ __forceinline__ Item load_item(const AttnParams& p, int item) {
     const int key_lo = first_visible_key(it.pos0, p.window, p.chunk);
     it.blk_lo = key_lo / BN;
     it.page_lo = key_lo / PAGE;                                          // the first page that holds a key any row sees
-    it.nb = it.pos_last / BN - it.blk_lo + 1;
+    it.n_kept = min((p.keep + BN - 1) / BN, it.blk_lo);                  // blocks of kept positions ahead of the window's
+    it.nb = it.n_kept + it.pos_last / BN - it.blk_lo + 1;
     return it;
 }
 
@@ -201,7 +209,7 @@ attn_prefill_tc05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                 }
                 ok = __shfl_sync(0xffffffffu, ok, 0);
                 if (!ok) break;
-                if (lane < HALVES) tma_load_2d(q_s + lane * ATOM_BYTES, &map_q, t.h * HD + lane * 64, t.row0, q_full);
+                if (lane < HALVES) tma_load_3d(q_s + lane * ATOM_BYTES, &map_q, lane * 64, t.h, t.row0, q_full);
                 issued_q = round + 1;
             }
             int rows16 = p.kv_rows;                                      // this lane's page of the 16 blocks at hand
@@ -211,8 +219,8 @@ attn_prefill_tc05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                     // a page past the tile's last key, or ahead of the first key that any of its rows sees (the sequence
                     // may have given it back), is read as zeros (a row past the cache)
                     rows16 = p.kv_rows;
-                    const int page_idx = (t.blk_lo + j) * 2 + lane;
-                    if (page_idx <= t.pos_last / PAGE && page_idx >= t.page_lo) {
+                    const int page_idx = t.block(j + (lane >> 1)) * 2 + (lane & 1);
+                    if (page_idx <= t.pos_last / PAGE && (page_idx >= t.page_lo || page_idx * PAGE < p.keep)) {
                         const int pg = p.block_table[(size_t)t.seq * p.table_stride + page_idx];
                         if (pg >= 0 && pg < p.n_pages) rows16 = (pg * p.nkv + t.kvh) * PAGE;
                         else atomicOr(p.status, ESP_STATUS_BAD_INDEX);
@@ -307,7 +315,7 @@ attn_prefill_tc05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
         // meet at a named barrier of their own (once when all have written, once when all have read).
         const int quad = warp & 3, r = quad * 32 + lane, grp = (warp - 2) / (4 * ROWT), side = ((warp - 2) >> 2) % ROWT;
         const unsigned lane_sel = (unsigned)(quad * 32) << 16;
-        const float sc = 1.4426950408889634f * (p.scale > 0.f ? p.scale : 1.0f / sqrtf((float)HD));
+        const float sc = 1.4426950408889634f * (p.scale > 0.f ? p.scale : 1.0f / sqrtf((float)p.kd));
         constexpr int CW = BN / ROWT;                                    // keys of a block that this thread takes
         constexpr int OW = HD / ROWT;                                    // columns of the group's O that this thread rescales
         constexpr int FW = HD / (GROUPS * ROWT);                         // columns of the result that this thread writes
@@ -329,7 +337,7 @@ attn_prefill_tc05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             const int key_first_last = first_visible_key(t.pos0 + BM - 1, p.window, p.chunk);   // of the tile's last row
             float m_ref = -INFINITY, l_run = 0.f;                         // the maximum that O and l_run are scaled by
             for (int j = grp; j < t.nb && ok; j += GROUPS, n_b++) {
-                const int key0 = (t.blk_lo + j) * BN;
+                const int key0 = t.block(j) * BN;
                 ok = !*abort_flag && mbar_wait(&s_full[grp], n_b & 1);
                 ok = pair_agree(ok, bar_grp, MATES);                      // the threads of a row go on or leave together
                 if (!ok) break;
@@ -340,6 +348,8 @@ attn_prefill_tc05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                 // live columns of this row: c_lo .. c_lo + c_span; one unsigned comparison per element, no branch
                 const int c_lo = key_first - key0 - side * CW;
                 const unsigned c_span = (unsigned)(pos - key_first);
+                // kept first positions among this thread's columns: those below c_kept (0: none)
+                const int c_kept = min(p.keep, pos + 1) - key0 - side * CW;
                 const unsigned s_addr = tm_s + grp * BN + lane_sel + side * CW;
                 float mx = -INFINITY;                                     // of the raw scores: the scale is positive
                 float sv[CW / 32][32];                                    // this thread's scores: read from TMEM once
@@ -348,10 +358,10 @@ attn_prefill_tc05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
                     tc_ld32(s_addr + c * 32, sv[c]);
                     if (edge) {
 #pragma unroll
-                        for (int i = 0; i < 32; i++) {
-                            sv[c][i] = (unsigned)(c * 32 + i - c_lo) <= c_span ? sv[c][i] : -INFINITY;
-                            mx = fmaxf(mx, sv[c][i]);
-                        }
+                        for (int i = 0; i < 32; i++)
+                            if (c * 32 + i >= c_kept) sv[c][i] = (unsigned)(c * 32 + i - c_lo) <= c_span ? sv[c][i] : -INFINITY;
+#pragma unroll
+                        for (int i = 0; i < 32; i++) mx = fmaxf(mx, sv[c][i]);
                     } else {
 #pragma unroll
                         for (int i = 0; i < 32; i++) mx = fmaxf(mx, sv[c][i]);
@@ -455,9 +465,10 @@ attn_prefill_tc05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid
             named_sync(bar_row, ROW_ALL);                                 // all have read the sums: the next item may write
             if (lane == 0) mbar_arrive(o_free);
             if (r < t.rows) {
-                bf16* orow = p.out + ((size_t)(t.row0 + r) * p.nh + t.h) * HD + col0;
+                bf16* orow = p.out + ((size_t)(t.row0 + r) * p.nh + t.h) * p.vd + col0;
 #pragma unroll
                 for (int i = 0; i < FW; i += 8) {
+                    if (col0 + i >= p.vd) break;
                     __nv_bfloat162 b0 = __floats2bfloat162_rn(o[i] * inv, o[i + 1] * inv);
                     __nv_bfloat162 b1 = __floats2bfloat162_rn(o[i + 2] * inv, o[i + 3] * inv);
                     __nv_bfloat162 b2 = __floats2bfloat162_rn(o[i + 4] * inv, o[i + 5] * inv);
@@ -484,8 +495,10 @@ typedef CUresult (*EncodeTiledFn)(CUtensorMap*, CUtensorMapDataType, cuuint32_t,
                                   const cuuint32_t*, const cuuint32_t*, CUtensorMapInterleave, CUtensorMapSwizzle,
                                   CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
 
-// a bfloat16 matrix [rows, cols] (row-major, contiguous) in boxes of box_rows x 64 columns, 128-byte swizzle, zeros outside
-int make_map2d(CUtensorMap* map, const void* base, unsigned long long cols, unsigned long long rows, unsigned box_rows) {
+// a bfloat16 tensor [rows, cols], or with mid > 0 [rows, mid, cols] (contiguous), in boxes of box_rows (x 1) x 64 columns,
+// 128-byte swizzle, zeros outside
+int make_map(CUtensorMap* map, const void* base, unsigned long long cols, unsigned long long mid, unsigned long long rows,
+             unsigned box_rows) {
     static EncodeTiledFn fn = nullptr;
     if (!fn) {
         void* ptr = nullptr;
@@ -495,11 +508,12 @@ int make_map2d(CUtensorMap* map, const void* base, unsigned long long cols, unsi
             return (int)cudaErrorNotSupported;
         fn = reinterpret_cast<EncodeTiledFn>(ptr);
     }
-    const cuuint64_t dims[2] = {cols, rows};
-    const cuuint64_t strides[1] = {cols * 2};
-    const cuuint32_t box[2] = {64, box_rows};
-    const cuuint32_t elem[2] = {1, 1};
-    const CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, const_cast<void*>(base), dims, strides, box, elem,
+    const bool three = mid > 0;
+    const cuuint64_t dims[3] = {cols, three ? mid : rows, rows};
+    const cuuint64_t strides[2] = {cols * 2, cols * (three ? mid : 1) * 2};
+    const cuuint32_t box[3] = {64, three ? 1 : box_rows, box_rows};
+    const cuuint32_t elem[3] = {1, 1, 1};
+    const CUresult r = fn(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, three ? 3 : 2, const_cast<void*>(base), dims, strides, box, elem,
                           CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_128B,
                           CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
     return r == CUDA_SUCCESS ? 0 : (int)cudaErrorInvalidValue;
@@ -538,26 +552,28 @@ int launch(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, 
 
 // q [n_tokens, nh, hd] and out the same shape, bfloat16; tile_seq / tile_first: the tiles of 128 new tokens
 // (sequence, index of the tile's first token among the sequence's new tokens), best listed with the tiles
-// that see the most keys first; hd 64 or 128; pages of 64 positions.
+// that see the most keys first; keys of hd and values of vd channels (0: hd), multiples of 8 up to 128 (out is then
+// [n_tokens, nh, vd]); pages of 64 positions.
 ESP_API int esp_attn_prefill_tc05(const void* q, long long n_tokens, const void* k_cache, const void* v_cache, void* out,
                                   const int* tile_seq, const int* tile_first, const int* seq_start, const int* seq_past,
                                   const int* block_table, int table_stride, int n_pages, int page, int n_tiles, int nh,
-                                  int nkv, int hd, float scale, int sink, const float* sink_vals, int window, int chunk, int* status,
-                                  cudaStream_t stream) {
+                                  int nkv, int hd, int vd, float scale, int sink, const float* sink_vals, int window, int chunk,
+                                  int keep, int* status, cudaStream_t stream) {
     if (n_tiles <= 0) return 0;
-    if (page != PAGE || (hd != 64 && hd != 128) || nkv <= 0 || nh % nkv != 0 || nh > 65535 || n_tokens <= 0)
+    if (vd <= 0) vd = hd;
+    if (page != PAGE || hd <= 0 || hd % 8 != 0 || hd > 128 || vd % 8 != 0 || vd > 128 || keep < 0 || nkv <= 0 || nh % nkv != 0 || nh > 65535 || n_tokens <= 0)
         return (int)cudaErrorInvalidValue;
     const unsigned long long kv_rows = (unsigned long long)n_pages * nkv * PAGE;
     if (kv_rows >= (1ull << 31)) return (int)cudaErrorInvalidValue;
     CUtensorMap mq, mk, mv;
-    int rc = make_map2d(&mq, q, (unsigned long long)nh * hd, (unsigned long long)n_tokens, BM);
+    int rc = make_map(&mq, q, (unsigned long long)hd, (unsigned long long)nh, (unsigned long long)n_tokens, BM);
     if (rc) return rc;
-    rc = make_map2d(&mk, k_cache, (unsigned long long)hd, kv_rows, PAGE);
+    rc = make_map(&mk, k_cache, (unsigned long long)hd, 0, kv_rows, PAGE);
     if (rc) return rc;
-    rc = make_map2d(&mv, v_cache, (unsigned long long)hd, kv_rows, PAGE);
+    rc = make_map(&mv, v_cache, (unsigned long long)vd, 0, kv_rows, PAGE);
     if (rc) return rc;
     AttnParams p{(bf16*)out, tile_seq, tile_first, seq_start, seq_past, block_table, table_stride, n_pages, nh, nkv,
-                 window, (int)kv_rows, n_tiles, 0, status, scale, sink, sink_vals, chunk};
-    if (hd == 64) return launch<64>(mq, mk, mv, p, n_tiles, stream);
+                 window, (int)kv_rows, n_tiles, 0, status, scale, sink, sink_vals, chunk, keep, hd, vd};
+    if (hd <= 64 && vd <= 64) return launch<64>(mq, mk, mv, p, n_tiles, stream);
     return launch<128>(mq, mk, mv, p, n_tiles, stream);
 }

@@ -3,7 +3,8 @@
 // prefill and decode alike and any head size up to 256.
 //
 // The query at absolute position a sees key j iff j <= a and (window == 0 or
-// a - j < window), or, with ``chunk`` > 0, iff j <= a and both lie in the same block of ``chunk`` positions.  score = dot(q, k_j) / sqrt(hd) (divided after the product), or dot(q, k_j) * scale when a scale is
+// a - j < window), or, with ``chunk`` > 0, iff j <= a and both lie in the same block of ``chunk`` positions; the first
+// ``keep`` positions of a sequence are seen besides.  score = dot(q, k_j) / sqrt(hd) (divided after the product), or dot(q, k_j) * scale when a scale is
 // given.  Values may have another size than keys (vd).  With ``sink`` the denominator holds one more term, exp(0 - max):
 // a key of score zero that carries no value; with ``sink_vals`` the term is exp(sink_vals[head] - max), a number per head
 // that is not scaled.  With ``softcap`` > 0 the scaled score s becomes softcap * tanh(s / softcap).  ``maps`` > 1: a key
@@ -26,7 +27,7 @@ __global__ void __launch_bounds__(THREADS)
 attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
                  TO* __restrict__ out, const int* __restrict__ tok_seq, const int* __restrict__ tok_pos,
                  const int* __restrict__ block_table, int table_stride, int n_pages, int page, int nh, int nkv, int hd,
-                 int vd, float scale, int sink, const float* __restrict__ sink_vals, int window, int chunk,
+                 int vd, float scale, int sink, const float* __restrict__ sink_vals, int window, int chunk, int keep,
                  float softcap, int maps, int* __restrict__ status) {
     __shared__ float qs[MAX_HD];
     __shared__ float ps[CHUNK];
@@ -35,7 +36,7 @@ attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T
     const int n = blockIdx.x, h = blockIdx.y, tid = threadIdx.x;
     const int seq = tok_seq[n], pos = tok_pos[n];
     const int kvh = h / (nh / nkv), map = h % maps;
-    const int lo = first_visible_key(pos, window, chunk);
+    const VisibleKeys seen = visible_keys(pos, window, chunk, keep);
     const T* qrow = q + ((size_t)n * nh + h) * hd;
     for (int d = tid; d < hd; d += THREADS) qs[d] = to_f32(qrow[d]);
     const float root = sqrtf((float)hd);
@@ -46,13 +47,19 @@ attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T
     for (int i = 0; i < MAX_HD / THREADS; i++) acc[i] = 0.f;
     __syncthreads();
 
-    for (int c = lo / CHUNK; c <= pos / CHUNK; c++) {
-        const int j0 = max(lo, c * CHUNK), j1 = min(pos, c * CHUNK + CHUNK - 1);
+    for (int c = seen.kept > 0 ? 0 : seen.lo / CHUNK; c <= pos / CHUNK; c++) {
+        if (c * CHUNK >= seen.kept && c < seen.lo / CHUNK) c = seen.lo / CHUNK;     // nothing between the kept keys and the window
+        const int j0 = c * CHUNK < seen.kept ? c * CHUNK : max(seen.lo, c * CHUNK), j1 = min(pos, c * CHUNK + CHUNK - 1);
         const int count = j1 - j0 + 1;
         // scores
         float local_max = -INFINITY;
         for (int t = tid; t < count; t += THREADS) {
             const int j = j0 + t;
+            if (!seen.sees(j)) {                                     // a chunk that holds both kept keys and the window's first
+                pages[t] = -1;
+                ps[t] = -INFINITY;
+                continue;
+            }
             int pg = block_table[(size_t)seq * table_stride + j / page];
             if (pg < 0 || pg >= n_pages) {
                 atomicOr(status, ESP_STATUS_BAD_INDEX);
@@ -111,7 +118,7 @@ attn_simt_kernel(const T* __restrict__ q, const T* __restrict__ k_cache, const T
 ESP_API int esp_attn_simt(const void* q, const void* k_cache, const void* v_cache, void* out, int is_bf16, int out_is_bf16,
                           const int* tok_seq, const int* tok_pos, const int* block_table, int table_stride, int n_pages,
                           int page, int n_tokens, int nh, int nkv, int hd, int vd, float scale, int sink,
-                          const float* sink_vals, int window, int chunk, float softcap, int maps, int* status,
+                          const float* sink_vals, int window, int chunk, int keep, float softcap, int maps, int* status,
                           cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (vd <= 0) vd = hd;
@@ -121,7 +128,7 @@ ESP_API int esp_attn_simt(const void* q, const void* k_cache, const void* v_cach
 #define ESP_SIMT(T, TO)                                                                                                    \
     attn_simt_kernel<T, TO><<<grid, THREADS, 0, stream>>>((const T*)q, (const T*)k_cache, (const T*)v_cache, (TO*)out, tok_seq, \
                                                           tok_pos, block_table, table_stride, n_pages, page, nh, nkv, hd, vd, \
-                                                          scale, sink, sink_vals, window, chunk, softcap, maps, status)
+                                                          scale, sink, sink_vals, window, chunk, keep, softcap, maps, status)
     if (is_bf16 && out_is_bf16) ESP_SIMT(bf16, bf16);
     else if (is_bf16) ESP_SIMT(bf16, float);
     else if (!out_is_bf16) ESP_SIMT(float, float);

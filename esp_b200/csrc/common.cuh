@@ -86,12 +86,36 @@ __device__ __forceinline__ float block_max(float v, float* scratch) {
     return scratch[32];
 }
 
+// A row that a block holds in registers, up to four pieces of four channels a thread (piece threadIdx.x + i * blockDim.x of
+// ``pieces``): takes ``mean`` off every channel and returns the sum of the squares of what is left.
+__device__ __forceinline__ float take_mean(float4 (&v)[4], int pieces, float mean, float* scratch) {
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        if (threadIdx.x + i * blockDim.x >= pieces) continue;
+        v[i].x -= mean, v[i].y -= mean, v[i].z -= mean, v[i].w -= mean;
+        ss = fmaf(v[i].w, v[i].w, fmaf(v[i].z, v[i].z, fmaf(v[i].y, v[i].y, fmaf(v[i].x, v[i].x, ss))));
+    }
+    return block_sum(ss, scratch);
+}
+
 // Which keys a query sees, in every attention kernel of this library: key j from position pos iff first <= j <= pos
 // with first = 0 (every earlier key), pos - window + 1 (the last ``window``), or (chunk > 0) the start of the query's
 // own block of ``chunk`` positions counted from the sequence's start.
 __host__ __device__ __forceinline__ int first_visible_key(int pos, int window, int chunk) {
     if (chunk > 0) return pos - pos % chunk;
     return window > 0 ? (pos - window + 1 > 0 ? pos - window + 1 : 0) : 0;
+}
+
+// The same with the first ``keep`` positions of the sequence seen besides (a window with kept first tokens): the keys
+// [0, kept) and [lo, pos], kept < lo; where the two would meet, lo is 0 and kept is 0.
+struct VisibleKeys {
+    int lo, kept;
+    __host__ __device__ __forceinline__ bool sees(int key) const { return key >= lo || key < kept; }    // of keys up to pos
+};
+__host__ __device__ __forceinline__ VisibleKeys visible_keys(int pos, int window, int chunk, int keep) {
+    const int lo = first_visible_key(pos, window, chunk);
+    return keep >= lo ? VisibleKeys{0, 0} : VisibleKeys{lo, keep};
 }
 
 // Launch-error helper: the C entry points return cudaGetLastError() as an int.

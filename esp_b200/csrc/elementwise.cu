@@ -50,17 +50,19 @@ ESP_API int esp_feed_tokens(int* ids, const int* picks, const int* src, int n, c
     return esp_launch_status();
 }
 
-// ---------------------------------------------------------------- add + RMSNorm
+// ---------------------------------------------------------------- add + RMSNorm or layer norm
 // Row r works on source row s = rows ? rows[r] : r.
 //   v = x[s] + (y ? y[s] * (yscale ? yscale : 1) : 0);  if (write_x) x[s] = v;      (yscale: one factor per channel)
 //   h[r] = v * (1 / sqrt(mean(v^2) + eps)) * gamma       (all in 32-bit)
+// or, LAYER: with the row's mean m, h[r] = (v - m) * (1 / sqrt(mean((v - m)^2) + eps)) * gamma + beta (the mean first, then
+// the squares of the deviations).
 // ``h32`` (may be null) receives the same rows unrounded, for consumers that
 // must work from 32-bit values whatever the activation dtype (the router).
 // The sum of squares is taken per thread in index order and combined by a
 // fixed tree, so a row's result does not depend on the rest of the batch.
-template <typename TH>
+template <typename TH, bool LAYER>
 __global__ void add_rmsnorm_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ yscale,
-                                   const float* __restrict__ gamma,
+                                   const float* __restrict__ gamma, const float* __restrict__ beta,
                                    const int* __restrict__ rows, TH* __restrict__ h, float* __restrict__ h32, int width,
                                    float eps, int write_x) {
     pdl_trigger();
@@ -77,16 +79,26 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ x, const float* __restric
             v += yscale ? yr[i] * yscale[i] : yr[i];
             if (write_x) xr[i] = v;
         }
-        ss = fmaf(v, v, ss);
+        ss = LAYER ? ss + v : fmaf(v, v, ss);
     }
-    const float total = block_sum(ss, scratch);
+    float total = block_sum(ss, scratch), mean = 0.f;
+    if (LAYER) {
+        mean = total / (float)width;
+        ss = 0.f;
+        for (int i = threadIdx.x; i < width; i += blockDim.x) {
+            float v = xr[i];
+            if (yr && !write_x) v += yscale ? yr[i] * yscale[i] : yr[i];
+            ss = fmaf(v - mean, v - mean, ss);
+        }
+        total = block_sum(ss, scratch);
+    }
     const float inv = 1.0f / sqrtf(total / (float)width + eps);
     TH* hr = h + (size_t)r * width;
     float* h32r = h32 ? h32 + (size_t)r * width : nullptr;
     for (int i = threadIdx.x; i < width; i += blockDim.x) {
         float v = xr[i];
         if (yr && !write_x) v += yscale ? yr[i] * yscale[i] : yr[i];
-        const float o = v * inv * gamma[i];
+        const float o = LAYER ? fmaf((v - mean) * inv, gamma[i], beta[i]) : v * inv * gamma[i];
         hr[i] = from_f32<TH>(o);
         if (h32r) h32r[i] = o;
     }
@@ -95,10 +107,11 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ x, const float* __restric
 // Same operation for rows whose width is a multiple of 4 and at most 4 * 4 * 1024: each thread keeps up
 // to four float4 pieces of the row in registers, so x and y are read once and nothing is read back.
 // The sum of squares is taken per thread in piece order and combined by the same fixed tree.
-template <typename TH>
+template <typename TH, bool LAYER>
 __global__ void __launch_bounds__(1024)
 add_rmsnorm_rows_kernel(float* __restrict__ x, const float* __restrict__ y, const float* __restrict__ yscale,
-                        const float* __restrict__ gamma, const int* __restrict__ rows, TH* __restrict__ h, float* __restrict__ h32, int width, float eps,
+                        const float* __restrict__ gamma, const float* __restrict__ beta, const int* __restrict__ rows,
+                        TH* __restrict__ h, float* __restrict__ h32, int width, float eps,
                         int write_x) {
     pdl_trigger();
     pdl_wait();
@@ -124,20 +137,29 @@ add_rmsnorm_rows_kernel(float* __restrict__ x, const float* __restrict__ y, cons
                 v[i].x += a.x; v[i].y += a.y; v[i].z += a.z; v[i].w += a.w;
                 if (write_x) xr[q] = v[i];
             }
-            ss = fmaf(v[i].x, v[i].x, ss);
-            ss = fmaf(v[i].y, v[i].y, ss);
-            ss = fmaf(v[i].z, v[i].z, ss);
-            ss = fmaf(v[i].w, v[i].w, ss);
+            if (LAYER) {
+                ss += (v[i].x + v[i].y) + (v[i].z + v[i].w);
+            } else {
+                ss = fmaf(v[i].x, v[i].x, ss);
+                ss = fmaf(v[i].y, v[i].y, ss);
+                ss = fmaf(v[i].z, v[i].z, ss);
+                ss = fmaf(v[i].w, v[i].w, ss);
+            }
         }
     }
-    const float total = block_sum(ss, scratch);
+    float total = block_sum(ss, scratch);
+    if (LAYER) total = take_mean(v, pieces, total / (float)width, scratch);
     const float inv = 1.0f / sqrtf(total / (float)width + eps);
 #pragma unroll
     for (int i = 0; i < 4; i++) {
         const int q = threadIdx.x + i * blockDim.x;
         if (q < pieces) {
             const float4 gm = reinterpret_cast<const float4*>(gamma)[q];
-            const float o0 = v[i].x * inv * gm.x, o1 = v[i].y * inv * gm.y, o2 = v[i].z * inv * gm.z, o3 = v[i].w * inv * gm.w;
+            float o0 = v[i].x * inv * gm.x, o1 = v[i].y * inv * gm.y, o2 = v[i].z * inv * gm.z, o3 = v[i].w * inv * gm.w;
+            if (LAYER) {
+                const float4 bt = reinterpret_cast<const float4*>(beta)[q];
+                o0 += bt.x, o1 += bt.y, o2 += bt.z, o3 += bt.w;
+            }
             TH* hr = h + (size_t)r * width + 4 * q;
             Vec4<TH>::store(hr, o0, o1, o2, o3);
             if (h32) reinterpret_cast<float4*>(h32 + (size_t)r * width)[q] = make_float4(o0, o1, o2, o3);
@@ -145,26 +167,33 @@ add_rmsnorm_rows_kernel(float* __restrict__ x, const float* __restrict__ y, cons
     }
 }
 
-ESP_API int esp_add_rmsnorm(float* x, const float* y, const float* yscale, const float* gamma, const int* rows, void* h, int h_is_bf16,
-                            float* h32, int n_rows, int width, float eps, int write_x, cudaStream_t stream) {
+// ``beta`` (may be null): the layer norm with this bias instead of the RMS norm.
+ESP_API int esp_add_rmsnorm(float* x, const float* y, const float* yscale, const float* gamma, const float* beta, const int* rows,
+                            void* h, int h_is_bf16, float* h32, int n_rows, int width, float eps, int write_x, cudaStream_t stream) {
     if (n_rows <= 0) return 0;
+#define ESP_ADD_NORM(KERNEL, TH, LAYER)                                                                                        \
+    esp_launch_pdl(ESP_PDL_SMALL, KERNEL<TH, LAYER>, dim3(n_rows), dim3(threads), 0, stream, x, y, yscale, gamma, beta, rows, (TH*)h, \
+                   h32, width, eps, write_x)
+#define ESP_ADD_NORM_T(KERNEL)                                  \
+    do {                                                        \
+        if (h_is_bf16 && beta) ESP_ADD_NORM(KERNEL, bf16, true); \
+        else if (h_is_bf16) ESP_ADD_NORM(KERNEL, bf16, false);   \
+        else if (beta) ESP_ADD_NORM(KERNEL, float, true);        \
+        else ESP_ADD_NORM(KERNEL, float, false);                 \
+    } while (0)
     if (width % 4 == 0 && width <= 16384) {
         int threads = ((width / 4 + 3) / 4 + 31) / 32 * 32;       // up to four pieces per thread
         // one piece per thread while a block can hold them: a row's sum then has the same order whatever else is in
         // the step (the 32-bit path relies on it).  Many rows rounded to bfloat16: four pieces per thread, smaller
         // blocks, more rows in flight per SM.
         if (width / 4 <= 1024 && !(h_is_bf16 && n_rows >= 256)) threads = (width / 4 + 31) / 32 * 32;
-        if (h_is_bf16)
-            esp_launch_pdl(ESP_PDL_SMALL, add_rmsnorm_rows_kernel<bf16>, dim3(n_rows), dim3(threads), 0, stream, x, y, yscale, gamma, rows, (bf16*)h, h32, width, eps, write_x);
-        else
-            esp_launch_pdl(ESP_PDL_SMALL, add_rmsnorm_rows_kernel<float>, dim3(n_rows), dim3(threads), 0, stream, x, y, yscale, gamma, rows, (float*)h, h32, width, eps, write_x);
+        ESP_ADD_NORM_T(add_rmsnorm_rows_kernel);
         return esp_launch_status();
     }
     const int threads = width >= 1024 ? 256 : 128;
-    if (h_is_bf16)
-        esp_launch_pdl(ESP_PDL_SMALL, add_rmsnorm_kernel<bf16>, dim3(n_rows), dim3(threads), 0, stream, x, y, yscale, gamma, rows, (bf16*)h, h32, width, eps, write_x);
-    else
-        esp_launch_pdl(ESP_PDL_SMALL, add_rmsnorm_kernel<float>, dim3(n_rows), dim3(threads), 0, stream, x, y, yscale, gamma, rows, (float*)h, h32, width, eps, write_x);
+    ESP_ADD_NORM_T(add_rmsnorm_kernel);
+#undef ESP_ADD_NORM_T
+#undef ESP_ADD_NORM
     return esp_launch_status();
 }
 

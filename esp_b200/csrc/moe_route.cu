@@ -49,27 +49,30 @@ __device__ __forceinline__ void scores_from_logits(const float* lg, float* ps, i
 
 // What a choice may depend on besides the scores: a number per expert that is added to the score for the choice only
 // (``correction``, may be null), and a limit to the best ``keep`` of ``n_groups`` equal groups of neighbouring experts
-// (a group's score is its largest corrected score; ties go to the lower group; n_groups <= 32, 0 or 1: no limit).
+// (a group's score is the sum of its ``group_top`` largest corrected scores, 1 or 2; ties go to the lower group; n_groups <= 32,
+// 0 or 1: no limit).  ``scale`` multiplies the routing weights.
 struct RouteChoice {
     const float* correction;
     int n_groups;
     int keep;
     const float* bias;      // a number per expert added to its logit (may be null)
+    int group_top;
+    float scale;
 };
 
 // The routing weight of a lane's chosen expert (rank = lane) from its score and the sum of the chosen scores; ``bad`` is
-// set where there is nothing to divide by.
-__device__ __forceinline__ float routing_weight(float my_p, float mass, int flags, int lane, int top_k, bool& bad) {
+// set where there is nothing to divide by.  Scores that are sigmoids may all be tiny: their sum is divided by with 1e-20 added.
+__device__ __forceinline__ float routing_weight(float my_p, float mass, int flags, int lane, int top_k, float scale, bool& bad) {
     if (flags & ROUTE_CHOSEN) {
         const float best = __shfl_sync(0xffffffffu, my_p, 0);             // rank 0 is the largest logit
         const float e = lane < top_k ? expf(my_p - best) : 0.f;
         const float sum = warp_sum(e);
         if (!(sum > 0.f)) bad = true;
-        return e / sum;
+        return e / sum * scale;
     }
-    const float denom = (flags & ROUTE_RENORM) ? mass : 1.0f;
+    const float denom = (flags & ROUTE_RENORM) ? ((flags & ROUTE_SIGMOID) ? mass + 1e-20f : mass) : 1.0f;
     if (!(denom > 0.f)) bad = true;
-    return my_p / denom;
+    return my_p / denom * scale;
 }
 
 // One token's top-k by one warp.  ps[e]: its scores (left as they are when a correction or groups are given, else
@@ -85,9 +88,14 @@ __device__ __forceinline__ float choose_topk(float* ps, float* cs, int n_experts
         __syncwarp();
         if (ch.n_groups > 1) {
             const int per = n_experts / ch.n_groups;
-            float gm = -INFINITY;
+            float gm = -INFINITY, second = -INFINITY;
             if (lane < ch.n_groups)
-                for (int e = lane * per; e < (lane + 1) * per; e++) gm = fmaxf(gm, cs[e]);
+                for (int e = lane * per; e < (lane + 1) * per; e++) {
+                    const float c = cs[e];
+                    second = fmaxf(second, fminf(gm, c));
+                    gm = fmaxf(gm, c);
+                }
+            if (ch.group_top == 2 && per > 1) gm += second;
             int ahead = 0;                                  // groups that come before this lane's
             for (int g = 0; g < ch.n_groups; g++) {
                 const float o = __shfl_sync(0xffffffffu, gm, g);
@@ -254,7 +262,7 @@ router_topk_kernel(const TH* __restrict__ h, const TW* __restrict__ w_router, co
         float my_p = 0.f;
         int my_e = 0;
         const float mass = choose_topk(ps, cs_all + t * n_experts, n_experts, top_k, lane, choice, my_p, my_e, bad);
-        const float wt = routing_weight(my_p, mass, norm_topk, lane, top_k, bad);
+        const float wt = routing_weight(my_p, mass, norm_topk, lane, top_k, choice.scale, bad);
         if (__any_sync(0xffffffffu, bad)) {
             if (lane == 0) atomicOr(status, ESP_STATUS_ROUTER_NONFINITE);
         }
@@ -377,7 +385,7 @@ router_select_kernel(const float* __restrict__ logits, int* __restrict__ topk_id
     float my_p = 0.f;
     int my_e = 0;
     const float mass = choose_topk(ps, ps + n_experts, n_experts, top_k, lane, choice, my_p, my_e, bad);
-    const float wt = routing_weight(my_p, mass, norm_topk, lane, top_k, bad);
+    const float wt = routing_weight(my_p, mass, norm_topk, lane, top_k, choice.scale, bad);
     if (__any_sync(0xffffffffu, bad)) {
         if (lane == 0) atomicOr(status, ESP_STATUS_ROUTER_NONFINITE);
     }
@@ -446,7 +454,7 @@ route_small_kernel(const float* __restrict__ logits, int* __restrict__ topk_ids,
         float my_p = 0.f;
         int my_e = 0;
         const float mass = choose_topk(ps, ps + n_experts, n_experts, top_k, lane, choice, my_p, my_e, bad);
-        const float wt = routing_weight(my_p, mass, norm_topk, lane, top_k, bad);
+        const float wt = routing_weight(my_p, mass, norm_topk, lane, top_k, choice.scale, bad);
         if (__any_sync(0xffffffffu, bad)) {
             if (lane == 0) atomicOr(status, ESP_STATUS_ROUTER_NONFINITE);
         }
@@ -738,12 +746,13 @@ __global__ void moe_combine_kernel(const float* __restrict__ expert_out, const i
 // with s = rows ? rows[r] : r.  Same operations in the same order as the two separate kernels, so the
 // results are the same bits.  Width a multiple of 4, at most 16384.  With gamma_y the combined row is normalised before it
 // is added: y <- y / sqrt(mean(y^2) + eps_y) * gamma_y (POST), and then gamma null: h[r] = v as it is; h null: the add alone.
-template <typename TH, bool POST>
+// LAYER: the norm behind the add is the layer norm, (v - mean(v)) * rsqrt(mean((v - mean(v))^2) + eps) * gamma + beta.
+template <typename TH, bool POST, bool LAYER>
 __global__ void __launch_bounds__(1024)
 moe_combine_add_rmsnorm_kernel(const float* __restrict__ expert_out, const int* __restrict__ topk_ids,
                                const int* __restrict__ inverse, const float* __restrict__ gate,
                                const float* __restrict__ shared, float* __restrict__ x, const float* __restrict__ gamma,
-                               const int* __restrict__ rows, TH* __restrict__ h, float* __restrict__ h32, int width,
+                               const float* __restrict__ beta, const int* __restrict__ rows, TH* __restrict__ h, float* __restrict__ h32, int width,
                                int top_k, float eps, int write_x, int early, const float* __restrict__ topk_w,
                                const float* __restrict__ ident, int n_real, const float* __restrict__ gamma_y, float eps_y) {
     pdl_trigger();
@@ -826,10 +835,14 @@ moe_combine_add_rmsnorm_kernel(const float* __restrict__ expert_out, const int* 
             xv.x += acc.x; xv.y += acc.y; xv.z += acc.z; xv.w += acc.w;
             if (write_x) reinterpret_cast<float4*>(x + t * width)[q] = xv;
             v[i] = xv;
-            ss = fmaf(xv.x, xv.x, ss);
-            ss = fmaf(xv.y, xv.y, ss);
-            ss = fmaf(xv.z, xv.z, ss);
-            ss = fmaf(xv.w, xv.w, ss);
+            if (LAYER) {
+                ss += (xv.x + xv.y) + (xv.z + xv.w);
+            } else {
+                ss = fmaf(xv.x, xv.x, ss);
+                ss = fmaf(xv.y, xv.y, ss);
+                ss = fmaf(xv.z, xv.z, ss);
+                ss = fmaf(xv.w, xv.w, ss);
+            }
         }
     }
     if (POST && !h) return;
@@ -841,14 +854,19 @@ moe_combine_add_rmsnorm_kernel(const float* __restrict__ expert_out, const int* 
         }
         return;
     }
-    const float total = block_sum(ss, scratch);
+    float total = block_sum(ss, scratch);
+    if (LAYER) total = take_mean(v, pieces, total / (float)width, scratch);
     const float inv = 1.0f / sqrtf(total / (float)width + eps);
 #pragma unroll
     for (int i = 0; i < 4; i++) {
         const int q = threadIdx.x + i * blockDim.x;
         if (q < pieces) {
             const float4 gm = reinterpret_cast<const float4*>(gamma)[q];
-            const float o0 = v[i].x * inv * gm.x, o1 = v[i].y * inv * gm.y, o2 = v[i].z * inv * gm.z, o3 = v[i].w * inv * gm.w;
+            float o0 = v[i].x * inv * gm.x, o1 = v[i].y * inv * gm.y, o2 = v[i].z * inv * gm.z, o3 = v[i].w * inv * gm.w;
+            if (LAYER) {
+                const float4 bt = reinterpret_cast<const float4*>(beta)[q];
+                o0 += bt.x, o1 += bt.y, o2 += bt.z, o3 += bt.w;
+            }
             TH* hr = h + (size_t)r * width + 4 * q;
             Vec4<TH>::store(hr, o0, o1, o2, o3);
             if (h32) reinterpret_cast<float4*>(h32 + (size_t)r * width)[q] = make_float4(o0, o1, o2, o3);
@@ -862,13 +880,14 @@ moe_combine_add_rmsnorm_kernel(const float* __restrict__ expert_out, const int* 
 ESP_API int esp_router_topk(const void* h, int h_is_bf16, const void* w_router, const void* w_gate, int w_is_bf16,
                             int* topk_ids, float* topk_w, float* gate, float* probs_out, float* logits, int n_tokens,
                             int width, int n_experts, int top_k, int norm_topk, const float* bias, const float* correction, int n_groups,
-                            int keep_groups, int* status, cudaStream_t stream) {
+                            int keep_groups, int group_top, float scale, int* status, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (top_k > MAX_TOPK || top_k <= 0 || top_k > n_experts) return (int)cudaErrorInvalidValue;
     if (n_groups > 32 || (n_groups > 1 && (n_experts % n_groups != 0 || keep_groups < 1 || keep_groups > n_groups ||
                                            keep_groups * (n_experts / n_groups) < top_k)))
         return (int)cudaErrorInvalidValue;
-    const RouteChoice choice{correction, n_groups, keep_groups, bias};
+    if (n_groups > 1 && group_top != 1 && group_top != 2) return (int)cudaErrorInvalidValue;
+    const RouteChoice choice{correction, n_groups, keep_groups, bias, group_top, scale};
     const int rows = n_experts + (w_gate ? 1 : 0);
     if (logits && !h_is_bf16 && w_is_bf16 && n_tokens >= 64 && width % 128 == 0 && rows <= 72 &&
         (size_t)16 * n_experts * sizeof(float) <= 48 * 1024 && (reinterpret_cast<uintptr_t>(h) & 15) == 0 &&
@@ -926,14 +945,15 @@ ESP_API int esp_route_small(const void* h, int h_is_bf16, const void* w_router, 
                             int width, int n_experts, int top_k, int norm_topk, int* offsets, int* perm_token,
                             float* perm_weight, int* inverse, int* status, unsigned long long* distinct, int* tile_group,
                             int* tile_row0, int* tile_count, int* n_tiles, int max_tiles, const float* bias, const float* correction,
-                            int n_groups, int keep_groups, int n_real, cudaStream_t stream) {
+                            int n_groups, int keep_groups, int group_top, float scale, int n_real, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (top_k > MAX_TOPK || top_k <= 0 || top_k > n_experts || n_tokens > ROUTE_SMALL_MAX) return (int)cudaErrorInvalidValue;
     if (n_real <= 0 || n_real > n_experts || n_groups > 32 ||
         (n_groups > 1 && (n_experts % n_groups != 0 || keep_groups < 1 || keep_groups > n_groups ||
                           keep_groups * (n_experts / n_groups) < top_k)))
         return (int)cudaErrorInvalidValue;
-    const RouteChoice choice{correction, n_groups, keep_groups, bias};
+    if (n_groups > 1 && group_top != 1 && group_top != 2) return (int)cudaErrorInvalidValue;
+    const RouteChoice choice{correction, n_groups, keep_groups, bias, group_top, scale};
     // the tile list (all four or none): one tile per expert with rows (experts from n_real on have none)
     if (tile_group && (!tile_row0 || !tile_count || !n_tiles || max_tiles < (n_real < n_tokens * top_k ? n_real : n_tokens * top_k)))
         return (int)cudaErrorInvalidValue;
@@ -992,12 +1012,13 @@ ESP_API int esp_moe_combine(const float* expert_out, const int* topk_ids, const 
 }
 
 ESP_API int esp_moe_combine_add_rmsnorm(const float* expert_out, const int* topk_ids, const int* inverse, const float* gate,
-                                        const float* shared, float* x, const float* gamma, const int* rows, void* h,
+                                        const float* shared, float* x, const float* gamma, const float* beta, const int* rows, void* h,
                                         int h_is_bf16, float* h32, int n_rows, int width, int top_k, float eps, int write_x,
                                         const float* topk_w, const float* ident, int n_real, const float* gamma_y,
                                         float eps_y, cudaStream_t stream) {
     if (n_rows <= 0) return 0;
-    if (top_k > MAX_TOPK || width % 4 != 0 || width > 16384 || (ident && !topk_w) || (h32 && (!h || !gamma)) || (!gamma_y && (!h || !gamma)))
+    if (top_k > MAX_TOPK || width % 4 != 0 || width > 16384 || (ident && !topk_w) || (h32 && (!h || !gamma)) || (!gamma_y && (!h || !gamma)) ||
+        (beta && (gamma_y || !gamma)))
         return (int)cudaErrorInvalidValue;
     int threads = ((width / 4 + 3) / 4 + 31) / 32 * 32;
     // one piece per thread while a block can hold them: a row's sum then has the same order whatever else is in the
@@ -1005,16 +1026,18 @@ ESP_API int esp_moe_combine_add_rmsnorm(const float* expert_out, const int* topk
     // more rows in flight per SM.
     if (width / 4 <= 1024 && !(h_is_bf16 && n_rows >= 256)) threads = (width / 4 + 31) / 32 * 32;
     const int early = esp_pdl_enabled(ESP_PDL_GROUPED) ? 0 : 1;
-#define ESP_COMBINE(TH, POST)                                                                                                \
-    esp_launch_pdl(ESP_PDL_SMALL, moe_combine_add_rmsnorm_kernel<TH, POST>, dim3(n_rows), dim3(threads), 0, stream, expert_out,  \
-                   topk_ids, inverse, gate, shared, x, gamma, rows, (TH*)h, h32, width, top_k, eps, write_x, early, topk_w,      \
+#define ESP_COMBINE(TH, POST, LAYER)                                                                                              \
+    esp_launch_pdl(ESP_PDL_SMALL, moe_combine_add_rmsnorm_kernel<TH, POST, LAYER>, dim3(n_rows), dim3(threads), 0, stream, expert_out,  \
+                   topk_ids, inverse, gate, shared, x, gamma, beta, rows, (TH*)h, h32, width, top_k, eps, write_x, early, topk_w,      \
                    ident, n_real, gamma_y, eps_y)
     if (h_is_bf16) {
-        if (gamma_y) ESP_COMBINE(bf16, true);
-        else ESP_COMBINE(bf16, false);
+        if (gamma_y) ESP_COMBINE(bf16, true, false);
+        else if (beta) ESP_COMBINE(bf16, false, true);
+        else ESP_COMBINE(bf16, false, false);
     } else {
-        if (gamma_y) ESP_COMBINE(float, true);
-        else ESP_COMBINE(float, false);
+        if (gamma_y) ESP_COMBINE(float, true, false);
+        else if (beta) ESP_COMBINE(float, false, true);
+        else ESP_COMBINE(float, false, false);
     }
 #undef ESP_COMBINE
     return esp_launch_status();

@@ -23,7 +23,7 @@ _SIGNATURES = {
     "esp_embed_gather": [P, c_int, P, P, c_int, c_int, c_int, c_float, P, P],
     "esp_softcap": [P, c_longlong, c_float, P],
     "esp_feed_tokens": [P, P, P, c_int, P],
-    "esp_add_rmsnorm": [P, P, P, P, P, P, c_int, P, c_int, c_int, c_float, c_int, P],
+    "esp_add_rmsnorm": [P, P, P, P, P, P, P, c_int, P, c_int, c_int, c_float, c_int, P],
     "esp_depth_mix": [P, P, P, P, P, c_int, c_int, c_int, P],
     "esp_xielu": [P, P, P, c_int, c_longlong, P],
     "esp_tanh": [P, P, c_int, c_longlong, P],
@@ -47,7 +47,7 @@ _SIGNATURES = {
     "esp_rope_kvwrite": [P, P, P, P, P, P, c_int, c_int, P, P, P, c_int, P, c_int, c_int, c_int, c_int, c_int, c_int,
                          c_int, c_int, P, P],
     "esp_attn_simt": [P, P, P, P, c_int, c_int, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int, P,
-                      c_int, c_int, c_float, c_int, P, P],
+                      c_int, c_int, c_int, c_float, c_int, P, P],
     "esp_headnorm_rope_kvwrite": [P, c_longlong, P, P, c_float, P, P, c_int, P, P, P, P, P, c_int, P, c_int, c_int, c_int, c_int,
                                   c_int, c_int, c_int, c_int, c_int, c_int, P, P],
     "esp_diff_combine": [P, c_float, c_float, c_float, P, c_longlong, P, c_int, c_int, c_int, c_int, P],
@@ -65,7 +65,7 @@ _SIGNATURES = {
     "esp_glu_clamped": [P, P, c_int, c_longlong, c_int, c_float, c_float, c_float, P],
     "esp_weighted_sum": [P, P, P, P, P, c_float, c_float, c_float, c_float, c_longlong, P],
     "esp_cast_cols": [P, c_longlong, P, c_int, c_longlong, c_int, P],
-    "esp_widenorm_rope_kvwrite": [P, P, P, c_float, P, c_int, c_float, P, P, P, P, P, c_int, P, c_int, c_int, c_int, c_int,
+    "esp_widenorm_rope_kvwrite": [P, P, P, P, c_float, P, P, c_int, c_int, c_float, P, P, P, P, P, c_int, P, c_int, c_int, c_int, c_int,
                                   c_int, c_int, c_int, c_int, c_int, P, P],
     "esp_delta_scan": [P, c_longlong, P, c_longlong, P, c_longlong, P, c_longlong, P, P, c_longlong, P, P, P, c_int, c_int,
                        c_int, c_int, c_int, P],
@@ -75,31 +75,32 @@ _SIGNATURES = {
                            c_int, c_int, P],
     "esp_head_scalar_gate": [P, c_int, P, c_longlong, P, c_int, c_int, c_int, c_int, P],
     "esp_heads_to_pages": [P, c_longlong, P, c_longlong, P, P, P, c_int, c_int, c_int, P, P, c_int, c_int, c_int, c_int, c_int, P, P],
-    "esp_pair_rope_unitnorm_kvwrite": [P, P, P, c_int, c_float, c_int, P, c_int, P, P, P, P, P, P, c_int, P, c_int, c_int, c_int,
+    "esp_pair_rope_unitnorm_kvwrite": [P, P, P, P, c_int, c_float, c_int, P, c_int, P, P, P, P, P, P, c_int, P, c_int, c_int, c_int,
                                        c_int, c_int, c_int, c_int, c_int, c_int, P, P],
     "esp_causal_conv": [P, c_longlong, P, P, P, c_longlong, P, P, P, P, c_int, c_int, c_int, c_int, c_int, P],
-    "esp_router_topk": [P, c_int, P, P, c_int, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, P, P, c_int, c_int, P, P],
+    "esp_router_topk": [P, c_int, P, P, c_int, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, P, P, c_int, c_int, c_int, c_float,
+                        P, P],
     "esp_moe_permute": [P, P, c_int, c_int, c_int, P, P, P, P, P, P, P, P, c_int, c_int, P, P, c_int, P],
     "esp_gather_rows": [P, P, P, c_int, c_int, P],
     "esp_route_small": [P, c_int, P, P, c_int, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, P, P, P, P, P, P, P, P, P, P,
-                        c_int, P, P, c_int, c_int, c_int, P],
+                        c_int, P, P, c_int, c_int, c_int, c_float, c_int, P],
     "esp_gemm_tc05": [P, c_longlong, P, c_int, c_int, P, P, c_longlong, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int,
                       c_int, c_int, c_float, c_float, c_float, P, P],
     "esp_wait_probe": [c_int, P, P],
     "esp_moe_combine": [P, P, P, P, P, P, c_int, c_int, c_int, P, P, c_int, P],
     "esp_pick_tokens": [P, c_int, c_int, P, P, P, P, P, P],
-    "esp_moe_combine_add_rmsnorm": [P, P, P, P, P, P, P, P, P, c_int, P, c_int, c_int, c_int, c_float, c_int, P, P, c_int, P, c_float,
+    "esp_moe_combine_add_rmsnorm": [P, P, P, P, P, P, P, P, P, P, c_int, P, c_int, c_int, c_int, c_float, c_int, P, P, c_int, P, c_float,
                                     P],
     "esp_gemm_skinny": [P, c_longlong, P, P, c_longlong, P, P, c_int, c_longlong, P, c_int, c_int, c_int, c_int, c_int,
                         c_int, c_int, P, c_float, c_float, c_float, P],
     "esp_qkv_rope_skinny": [P, c_longlong, P, P, P, P, P, P, c_int, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int,
                             c_int, c_int, c_int, P, P],
     "esp_attn_prefill": [P, P, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float, c_int,
-                         P, c_int, c_int, P, P],
-    "esp_attn_prefill_tc05": [P, c_longlong, P, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
-                              c_int, P, c_int, c_int, P, P],
-    "esp_attn_decode": [P, P, P, P, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
-                        c_int, c_float, c_int, P, c_int, P, P],
+                         P, c_int, c_int, c_int, P, P],
+    "esp_attn_prefill_tc05": [P, c_longlong, P, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
+                              c_int, P, c_int, c_int, c_int, P, P],
+    "esp_attn_decode": [P, P, P, P, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
+                        c_int, c_float, c_int, P, c_int, c_int, P, P],
     "esp_attn_diff_tc05": [P, c_longlong, P, P, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_float,
                            c_float, c_int, c_float, c_float, c_float, P, c_longlong, P, P],
     "esp_attn_decode_diff": [P, P, P, P, P, P, P, P, P, P, P, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_int,
@@ -250,18 +251,19 @@ def feed_tokens(ids, picks, src):
                                            _ptr(src, torch.int32, "src"), ids.shape[0], _stream()), "feed_tokens")
 
 
-def add_rmsnorm(x, y, gamma, h, eps, rows=None, write_x=True, h32=None, yscale=None):
+def add_rmsnorm(x, y, gamma, h, eps, rows=None, write_x=True, h32=None, yscale=None, beta=None):
     """h = rmsnorm(x + y) * gamma with x (+= y when write_x) float32, gamma
     float32, h float32 or bfloat16.  ``rows`` (int32) selects source rows;
     ``h32`` (float32, same shape as h) receives the unrounded rows; ``yscale``
-    (float32 [width]) multiplies y channel by channel before it is added."""
+    (float32 [width]) multiplies y channel by channel before it is added.  ``beta`` (float32 [width]): the layer norm
+    (mean off, then the root of the mean square, gamma and this bias) in place of the RMS norm."""
     n_rows = h.shape[0]
     width = h.shape[1]
     if x.shape[1] != width or gamma.shape[0] != width:
         raise Backend("add_rmsnorm: widths disagree")
     _check(_fn("core", "esp_add_rmsnorm")(
         _ptr(x, torch.float32, "x"), _ptr(y, torch.float32, "y"), _ptr(yscale, torch.float32, "yscale"),
-        _ptr(gamma, torch.float32, "gamma"),
+        _ptr(gamma, torch.float32, "gamma"), _ptr(beta, torch.float32, "beta"),
         _ptr(rows, torch.int32, "rows"), _ptr(h, FLOATS, "h"), _is_bf16(h), _ptr(h32, torch.float32, "h32"), n_rows,
         width, float(eps),
         1 if write_x else 0, _stream()), "add_rmsnorm")
@@ -367,13 +369,14 @@ def _sink_args(sink, nh):
 
 
 def attn_simt(q, k_cache, v_cache, out, tok_seq, tok_pos, block_table, page, nh, nkv, hd, window, status, vd=None,
-              scale=0.0, sink=False, chunk=None, softcap=None, maps=1):
+              scale=0.0, sink=False, chunk=None, softcap=None, maps=1, keep=0):
     """Attention of every token over its sequence's cached keys (32-bit arithmetic).  ``out`` may be float32 whatever the
     cache's dtype.  ``softcap``: scaled scores s become softcap * tanh(s / softcap).  ``maps``: keys that lie side by side
     in a key head's row of the cache; query head h reads the key h % maps of its key head.  ``vd``: size of a value head
     (default: the key size); ``scale`` > 0 multiplies the scores instead of the division by sqrt(hd); ``sink``: the
     softmax's denominator holds one more term exp(0), or exp(sink[head]) when a tensor is given; ``chunk``: a query
-    sees the keys of its own block of that many positions only."""
+    sees the keys of its own block of that many positions only; ``keep`` (with a window): the first ``keep`` positions of a
+    sequence are seen besides."""
     sink_flag, sink_ptr = _sink_args(sink, nh)
     vd = hd if vd is None else vd
     if hd > 256 or vd > 256:
@@ -382,26 +385,31 @@ def attn_simt(q, k_cache, v_cache, out, tok_seq, tok_pos, block_table, page, nh,
         _ptr(q, FLOATS, "q"), _ptr(k_cache, FLOATS), _ptr(v_cache, FLOATS), _ptr(out, FLOATS), _is_bf16(q),
         _is_bf16(out), _ptr(tok_seq, torch.int32), _ptr(tok_pos, torch.int32), _ptr(block_table, torch.int32), block_table.shape[1],
         k_cache.shape[0], page, q.shape[0], nh, nkv, hd, vd, float(scale), sink_flag, sink_ptr, int(window or 0),
-        int(chunk or 0), float(softcap or 0.0), int(maps), _ptr(status, torch.int32), _stream()), "attn_simt")
+        int(chunk or 0), int(keep), float(softcap or 0.0), int(maps), _ptr(status, torch.int32), _stream()), "attn_simt")
 
 
 def _choice_args(choice, n_experts):
-    """(correction pointer, groups, kept groups) of a ``choice`` = (correction float32 [experts] or None, groups, keep)."""
+    """(correction pointer, groups, kept groups, scores summed per group) of a ``choice`` = (correction float32 [experts] or
+    None, groups, keep[, group_top])."""
     if choice is None:
-        return None, 0, 0
-    correction, groups, keep = choice
+        return None, 0, 0, 1
+    correction, groups, keep = choice[:3]
+    group_top = choice[3] if len(choice) > 3 else 1
+    if group_top not in (1, 2):
+        raise Backend(f"router: a group's score is the sum of its one or two largest, not {group_top}")
     if correction is not None and correction.shape[0] != n_experts:
         raise Backend("router: the correction has another length than the router has outputs")
     if groups and groups > 1 and (groups > 32 or n_experts % groups or not 1 <= keep <= groups):
         raise Backend(f"router: {groups} groups (keep {keep}) over {n_experts} experts are not taken")
-    return _ptr(correction, torch.float32, "correction"), int(groups or 0), int(keep or 0)
+    return _ptr(correction, torch.float32, "correction"), int(groups or 0), int(keep or 0), int(group_top)
 
 
 def router_topk(h, w_router, w_gate, topk_ids, topk_w, gate, top_k, norm_topk, status, probs_out=None, logits=None,
-                sigmoid=False, choice=None, bias=None, chosen_softmax=False):
-    """``bias``: float32, a number per expert added to its logit.  ``chosen_softmax``: the experts with the largest logits,
-    weighted by a softmax over those logits alone.  ``choice``: None, or (correction, groups, keep): a number per expert added to its score for the choice only, and
-    a limit of the choice to the best ``keep`` of ``groups`` equal groups of neighbouring experts.  ``logits``: optional float32 scratch [n, experts + 1]; with it, 32-bit activations and bfloat16 weights
+                sigmoid=False, choice=None, bias=None, chosen_softmax=False, scale=1.0):
+    """``scale`` multiplies the weights.  ``bias``: float32, a number per expert added to its logit.  ``chosen_softmax``: the experts with the largest logits,
+    weighted by a softmax over those logits alone.  ``choice``: None, or (correction, groups, keep[, group_top]): a number per expert added to its score for the choice only, and
+    a limit of the choice to the best ``keep`` of ``groups`` equal groups of neighbouring experts (by their largest score, or by
+    the sum of the two largest with group_top 2).  ``logits``: optional float32 scratch [n, experts + 1]; with it, 32-bit activations and bfloat16 weights
     the logits of a step of many tokens are made on the tensor cores (three bfloat16 parts of every
     activation: products exact, sums in float)."""
     n, width = h.shape
@@ -410,7 +418,7 @@ def router_topk(h, w_router, w_gate, topk_ids, topk_w, gate, top_k, norm_topk, s
         raise Backend(f"router: top-k {top_k} is beyond the 32 this kernel takes")
     if (width + 2 * n_experts) * 4 > 200 * 1024:
         raise Backend(f"router: width {width} + experts {n_experts} do not fit the kernel's shared memory")
-    pc, groups, keep = _choice_args(choice, n_experts)
+    pc, groups, keep, group_top = _choice_args(choice, n_experts)
     if w_gate is not None and w_gate.dtype != w_router.dtype:
         raise Backend("router: router and shared-gate weights must share a dtype")
     if logits is not None and logits.numel() < n * (n_experts + 1):
@@ -422,7 +430,7 @@ def router_topk(h, w_router, w_gate, topk_ids, topk_w, gate, top_k, norm_topk, s
         _ptr(topk_ids, torch.int32), _ptr(topk_w, torch.float32), _ptr(gate, torch.float32),
         _ptr(probs_out, torch.float32), _ptr(logits, torch.float32), n, width, n_experts, top_k,
         (1 if norm_topk else 0) | (2 if sigmoid else 0) | (4 if chosen_softmax else 0), _ptr(bias, torch.float32, "bias"), pc,
-        groups, keep, _ptr(status, torch.int32), _stream()), "router_topk")
+        groups, keep, group_top, float(scale), _ptr(status, torch.int32), _stream()), "router_topk")
 
 
 ROUTE_SMALL_TOKENS = 64
@@ -435,8 +443,8 @@ def route_small_fits(width: int, n_experts: int) -> bool:
 
 def route_small(h, w_router, w_gate, logits, topk_ids, topk_w, gate, top_k, norm_topk, offsets, perm_token,
                 perm_weight, inverse, status, probs_out=None, distinct=None, tiles=None, sigmoid=False, choice=None,
-                n_real=None, bias=None, chosen_softmax=False):
-    """``bias``, ``chosen_softmax``: as for router_topk.  ``choice``: as for router_topk.  ``n_real``: experts from this id on have no rows (their pairs get inverse -1).
+                n_real=None, bias=None, chosen_softmax=False, scale=1.0):
+    """``bias``, ``chosen_softmax``, ``scale``: as for router_topk.  ``choice``: as for router_topk.  ``n_real``: experts from this id on have no rows (their pairs get inverse -1).
     Router and permutation for at most ROUTE_SMALL_TOKENS tokens: logits over many blocks, then one
     block for softmax, top-k and the permutation.  ``logits``: float32 scratch [N, E + 1].  ``distinct``:
     an int64 tensor of one element to which the number of experts with at least one token is added.
@@ -445,7 +453,7 @@ def route_small(h, w_router, w_gate, logits, topk_ids, topk_w, gate, top_k, norm
     n_experts = w_router.shape[0]
     if n > ROUTE_SMALL_TOKENS or top_k > 32 or not route_small_fits(width, n_experts):
         raise Backend("route_small: too many tokens or experts for this kernel")
-    pc, groups, keep = _choice_args(choice, n_experts)
+    pc, groups, keep, group_top = _choice_args(choice, n_experts)
     if bias is not None and bias.shape[0] != n_experts:
         raise Backend("route_small: the bias has another length than the router has outputs")
     _check(_fn("core", "esp_route_small")(
@@ -456,7 +464,8 @@ def route_small(h, w_router, w_gate, logits, topk_ids, topk_w, gate, top_k, norm
         _ptr(inverse, torch.int32), _ptr(status, torch.int32), _ptr(distinct, torch.int64),
         _ptr(tiles[0], torch.int32) if tiles else None, _ptr(tiles[1], torch.int32) if tiles else None,
         _ptr(tiles[2], torch.int32) if tiles else None, _ptr(tiles[3], torch.int32) if tiles else None,
-        tiles[0].shape[0] if tiles else 0, _ptr(bias, torch.float32, "bias"), pc, groups, keep, int(n_real if n_real is not None else n_experts), _stream()),
+        tiles[0].shape[0] if tiles else 0, _ptr(bias, torch.float32, "bias"), pc, groups, keep, group_top, float(scale),
+        int(n_real if n_real is not None else n_experts), _stream()),
         "route_small")
 
 
@@ -488,11 +497,11 @@ def moe_combine(expert_out, topk_ids, inverse, gate, shared, y, passing=None):
 
 
 def moe_combine_add_rmsnorm(expert_out, topk_ids, inverse, gate, shared, x, gamma, h, eps, rows=None, write_x=True,
-                            h32=None, passing=None, gamma_y=None, eps_y=0.0):
+                            h32=None, passing=None, gamma_y=None, eps_y=0.0, beta=None):
     """moe_combine followed by add_rmsnorm in one kernel (same operations in the same order): x (+)= combined
     expert outputs, h = rmsnorm(x) * gamma.  Width a multiple of 4, at most 16384.  ``passing``: as for moe_combine.
     ``gamma_y`` (with ``eps_y``): the combined row is normalised, rmsnorm(y) * gamma_y, before it is added.  ``gamma``
-    None: h = x in h's dtype; ``h`` None: the add alone."""
+    None: h = x in h's dtype; ``h`` None: the add alone.  ``beta``: the layer norm with this bias in place of the RMS norm."""
     n_rows, width = h.shape if h is not None else x.shape
     pw, pi, pn = (_ptr(passing[0], torch.float32), _ptr(passing[1], torch.float32, "ident"), int(passing[2])) if passing else (None, None, 0)
     if width % 4 != 0 or width > 16384:
@@ -500,7 +509,7 @@ def moe_combine_add_rmsnorm(expert_out, topk_ids, inverse, gate, shared, x, gamm
     _check(_fn("core", "esp_moe_combine_add_rmsnorm")(
         _ptr(expert_out, torch.float32), _ptr(topk_ids, torch.int32), _ptr(inverse, torch.int32),
         _ptr(gate, torch.float32), _ptr(shared, torch.float32), _ptr(x, torch.float32), _ptr(gamma, torch.float32),
-        _ptr(rows, torch.int32), _ptr(h, FLOATS, "h"), _is_bf16(h) if h is not None else 0, _ptr(h32, torch.float32), n_rows,
+        _ptr(beta, torch.float32), _ptr(rows, torch.int32), _ptr(h, FLOATS, "h"), _is_bf16(h) if h is not None else 0, _ptr(h32, torch.float32), n_rows,
         width, topk_ids.shape[1], float(eps), 1 if write_x else 0, pw, pi, pn, _ptr(gamma_y, torch.float32, "gamma_y"),
         float(eps_y), _stream()), "moe_combine_add_rmsnorm")
 
@@ -630,11 +639,22 @@ def attn_decode_split(n_rows: int, nkv_blocks: int, positions: int, head_dim: in
 ATTN_DECODE_COUNTERS = 65536
 
 
+def attn_decode_fits(hd: int, vd: int) -> bool:
+    """Sizes of a key and a value head that ``attn_decode`` takes."""
+    return hd % 8 == 0 and 0 < hd <= 256 and vd % 8 == 0 and 0 < vd <= 256
+
+
+def attn_decode_tile(hd: int, vd: int) -> int:
+    """The width that ``attn_decode`` pads keys and values to."""
+    return (max(hd, vd) + 63) // 64 * 64
+
+
 def attn_decode(q, k_cache, v_cache, out, part_o, part_ml, counters, tok_seq, tok_pos, block_table, page, nh, nkv, hd,
-                window, split, n_splits, status, seq_past=None, scale=0.0, sink=False, chunk=None):
-    """Split-key attention for few token rows (bfloat16; head sizes 64, 128, 192, 256).  ``split``: key
+                window, split, n_splits, status, seq_past=None, scale=0.0, sink=False, chunk=None, vd=None, keep=0):
+    """Split-key attention for few token rows (bfloat16; keys of hd and values of ``vd`` (default: hd) channels, multiples of
+    8 up to 256; ``keep`` as for attn_simt).  ``split``: key
     positions per block (a multiple of 64); n_splits >= ceil(positions / split).  part_o float32
-    [N, nh, n_splits, hd] and part_ml float32 [N, nh, n_splits, 2] are scratch; ``counters``: int32, at least
+    [N, nh, n_splits, attn_decode_tile(hd, vd)] and part_ml float32 [N, nh, n_splits, 2] are scratch; ``counters``: int32, at least
     N * nh words, all zero (the kernel leaves them zero).  ``seq_past`` (int32 per sequence of the step: the
     positions cached before it): blocks whose keys are all older then load them without waiting for the
     kernel before this one, which writes the step's new keys and values.  ``scale`` > 0 multiplies the scores instead
@@ -645,18 +665,19 @@ def attn_decode(q, k_cache, v_cache, out, part_o, part_ml, counters, tok_seq, to
         raise Backend("attn_decode: too few counters for this many rows and heads")
     if split < 64 or split % 64:
         raise Backend(f"attn_decode: split {split} is not a multiple of 64")
-    if hd not in (64, 128, 192, 256):
-        raise Backend(f"attn_decode: head size {hd} is not one of 64, 128, 192, 256")
+    vd = hd if vd is None else vd
+    if not attn_decode_fits(hd, vd):
+        raise Backend(f"attn_decode: head sizes {hd} / {vd} are not multiples of 8 up to 256")
     n = q.shape[0]
-    if part_o.numel() < n * nh * n_splits * hd or part_ml.numel() < n * nh * n_splits * 2:
+    if part_o.numel() < n * nh * n_splits * attn_decode_tile(hd, vd) or part_ml.numel() < n * nh * n_splits * 2:
         raise Backend("attn_decode: scratch is too small")
     _check(_fn("bf16", "esp_attn_decode")(
         _ptr(q, torch.bfloat16, "q"), _ptr(k_cache, torch.bfloat16), _ptr(v_cache, torch.bfloat16),
         _ptr(out, torch.bfloat16), _ptr(part_o, torch.float32), _ptr(part_ml, torch.float32),
         _ptr(counters, torch.int32), _ptr(tok_seq, torch.int32), _ptr(tok_pos, torch.int32), _ptr(seq_past, torch.int32),
         _ptr(block_table, torch.int32), block_table.shape[1],
-        k_cache.shape[0], page, n, nh, nkv, hd, int(window or 0), split, n_splits, float(scale), sink_flag, sink_ptr,
-        int(chunk or 0), _ptr(status, torch.int32), _stream()), "attn_decode")
+        k_cache.shape[0], page, n, nh, nkv, hd, vd, int(window or 0), split, n_splits, float(scale), sink_flag, sink_ptr,
+        int(chunk or 0), int(keep), _ptr(status, torch.int32), _stream()), "attn_decode")
 
 
 def attn_decode_diff_fits(key_dim: int, value_dim: int, page: int) -> bool:
@@ -761,12 +782,12 @@ def attn_flash_fits(hd, vd=None, page=64) -> bool:
 
 
 def attn_prefill(q, k_cache, v_cache, out, tile_seq, tile_first, seq_start, seq_past, block_table, page, nh, nkv, hd,
-                 window, status, vd=None, scale=0.0, sink=False, chunk=None):
+                 window, status, vd=None, scale=0.0, sink=False, chunk=None, keep=0):
     """Flash-style attention for runs of new tokens (bfloat16; head sizes that are multiples of 8 up to
     128; pages of 64 positions).  tile_seq / tile_first describe the tiles of 64 new tokens.  ``vd``: size of a
     value head (default: the key size); ``scale`` > 0 multiplies the scores instead of the division by sqrt(hd);
     ``sink``: the softmax's denominator holds one more term exp(0), or exp(sink[head]) when a float32 tensor is given;
-    ``chunk``: a query sees the keys of its own block of that many positions only."""
+    ``chunk``: a query sees the keys of its own block of that many positions only; ``keep`` as for attn_simt."""
     sink_flag, sink_ptr = _sink_args(sink, nh)
     vd = hd if vd is None else vd
     if not attn_flash_fits(hd, vd, page):
@@ -776,36 +797,38 @@ def attn_prefill(q, k_cache, v_cache, out, tile_seq, tile_first, seq_start, seq_
         _ptr(out, torch.bfloat16), _ptr(tile_seq, torch.int32), _ptr(tile_first, torch.int32),
         _ptr(seq_start, torch.int32), _ptr(seq_past, torch.int32), _ptr(block_table, torch.int32),
         block_table.shape[1], k_cache.shape[0], page, tile_seq.shape[0], nh, nkv, hd, vd, float(scale), sink_flag, sink_ptr,
-        int(window or 0), int(chunk or 0), _ptr(status, torch.int32), _stream()), "attn_prefill")
+        int(window or 0), int(chunk or 0), int(keep), _ptr(status, torch.int32), _stream()), "attn_prefill")
 
 
 ATTN_TC05_TILE_ROWS = 128      # new tokens of a sequence to a tile of attn_prefill_tc05
 
 
-def attn_prefill_tc05_fits(hd, page) -> bool:
-    """Head sizes and page size that the tensor-memory prefill attention takes."""
-    return hd in (64, 128) and page == 64
+def attn_prefill_tc05_fits(hd, page, vd=None) -> bool:
+    """Head sizes (keys, values) and page size that the tensor-memory prefill attention takes."""
+    vd = hd if vd is None else vd
+    return hd % 8 == 0 and 0 < hd <= 128 and vd % 8 == 0 and 0 < vd <= 128 and page == 64
 
 
 def attn_prefill_tc05(q, k_cache, v_cache, out, tile_seq, tile_first, seq_start, seq_past, block_table, page, nh, nkv, hd,
-                      window, status, scale=0.0, sink=False, chunk=None):
-    """Prefill attention on tcgen05 with accumulators in tensor memory (bfloat16; head size 64 or 128; pages
-    of 64 positions).  Same arguments as attn_prefill, but tile_seq / tile_first list tiles of
+                      window, status, scale=0.0, sink=False, chunk=None, vd=None, keep=0):
+    """Prefill attention on tcgen05 with accumulators in tensor memory (bfloat16; keys of hd and values of ``vd`` (default:
+    hd) channels, multiples of 8 up to 128, padded to 64 or 128; pages of 64 positions; ``keep`` as for attn_simt).  Same arguments as attn_prefill, but tile_seq / tile_first list tiles of
     ATTN_TC05_TILE_ROWS new tokens, best with the tiles that see the most keys first (the order only matters
     for the balance).  ``scale`` > 0 multiplies the scores instead of the division by sqrt(hd); ``sink``: the softmax's
     denominator holds one more term exp(0), or exp(sink[head]) when a float32 tensor is given; ``chunk``: a query sees the
     keys of its own block of that many positions only."""
     sink_flag, sink_ptr = _sink_args(sink, nh)
-    if not attn_prefill_tc05_fits(hd, page):
-        raise Backend(f"attn_prefill_tc05: head size {hd} / page {page} not taken (64 or 128; page 64)")
+    vd = hd if vd is None else vd
+    if not attn_prefill_tc05_fits(hd, page, vd):
+        raise Backend(f"attn_prefill_tc05: head sizes {hd} / {vd} / page {page} not taken (multiples of 8 up to 128; page 64)")
     if not q.is_contiguous() or q.numel() != q.shape[0] * nh * hd:
         raise Backend("attn_prefill_tc05 takes contiguous queries [tokens, heads * head size]")
     _check(_fn("tc05", "esp_attn_prefill_tc05")(
         _ptr(q, torch.bfloat16, "q"), q.shape[0], _ptr(k_cache, torch.bfloat16), _ptr(v_cache, torch.bfloat16),
         _ptr(out, torch.bfloat16), _ptr(tile_seq, torch.int32), _ptr(tile_first, torch.int32),
         _ptr(seq_start, torch.int32), _ptr(seq_past, torch.int32), _ptr(block_table, torch.int32),
-        block_table.shape[1], k_cache.shape[0], page, tile_seq.shape[0], nh, nkv, hd, float(scale), sink_flag, sink_ptr,
-        int(window or 0), int(chunk or 0), _ptr(status, torch.int32), _stream()), "attn_prefill_tc05")
+        block_table.shape[1], k_cache.shape[0], page, tile_seq.shape[0], nh, nkv, hd, vd, float(scale), sink_flag, sink_ptr,
+        int(window or 0), int(chunk or 0), int(keep), _ptr(status, torch.int32), _stream()), "attn_prefill_tc05")
 
 
 def gather_rows(src, rows, out):
@@ -910,6 +933,7 @@ def token_shift_keep(h, prev_state, seq_start, seq_slot, n_seqs: int):
 SCAN_DECAY_BONUS = 0          # d = exp(-exp(g + bias)), the current token weighted by ``bonus``, output before the update
 SCAN_LOWER_SIGMOID = 1        # d = lower + (1 - lower) sigmoid(g + bias), k = 1 - d, q = silu(q), output after the update
 SCAN_SCALAR_DECAY = 2         # with ready=True: g holds one ready-made decay per head and token [rows, heads]; output after the update
+SCAN_FIXED_DECAY = 3          # one decay per head, g [heads] + lower [heads]; q, k, v = SiLU of what is given (ready: as given); output after the update
 SCAN_MAX_KEY_DIM = 256
 
 
@@ -930,11 +954,16 @@ def gated_scan(mode, q, k, g, v, gate_bias, lower, bonus, state, seq_start, seq_
     runs of rows that the sequences bring (seq_start), from and to ``state`` (float32 [slots, >= heads * value_dim *
     key_dim], a head's block laid out [value_dim, key_dim]).  q, k, g: float32 [rows, heads * key_dim]; v: float32
     [rows, heads * value_dim]; out: float32 [rows, heads * value_dim].  All 32-bit.  ``ready``: q, k and g hold the
-    query, the written key and the decay themselves (``gate_prepare`` made them)."""
+    query, the written key and the decay themselves (``gate_prepare`` made them).  SCAN_FIXED_DECAY: g and ``lower`` are
+    float32 [heads], the decay and what 32-bit leaves out of it."""
     if key_dim > SCAN_MAX_KEY_DIM:
         raise Backend(f"gated_scan: {key_dim} key channels per head are beyond the {SCAN_MAX_KEY_DIM} this kernel takes")
     if state.dtype != torch.float32 or state.stride(1) != 1 or state.shape[1] < heads * key_dim * value_dim:
         raise Backend("gated_scan: the state rows are too short or not float32")
+    if mode == SCAN_FIXED_DECAY:
+        if g.numel() != heads or lower is None or lower.numel() != heads:
+            raise Backend("gated_scan: a fixed decay is one number per head, in two parts")
+        g = g.view(1, heads)
     (pq, ldq), (pk, ldk), (pg, ldg), (pv, ldv) = (_rows_ld(t, n) for t, n in ((q, "q"), (k, "k"), (g, "g"), (v, "v")))
     _check(_fn("mixers", "esp_gated_scan")(
         int(mode), 1 if ready else 0, pq, ldq, pk, ldk, pg, ldg, pv, ldv, _ptr(gate_bias, torch.float32, "gate_bias"),
@@ -1222,17 +1251,20 @@ def cast_cols(src, dst):
 
 
 def widenorm_rope_kvwrite(qkv, q_w, k_w, eps, inv_freq, rot, v_scale, tok_seq, tok_pos, q_out, k_cache, v_cache, block_table,
-                          page, nh, nkv, hd, vd, write_kv, status):
+                          page, nh, nkv, hd, vd, write_kv, status, bias=None, neighbour=False, inv_freq_lo=None):
     """Queries and keys normed over their whole projection (weights q_w [nh * hd], k_w [nkv * hd]), the first ``rot``
     channels of every head rotated by position * inv_freq, values times v_scale; queries to q_out, keys and values to the
-    paged cache.  qkv float32 [rows, nh * hd + nkv * hd + nkv * vd]."""
-    if qkv.shape[1] != nh * hd + nkv * hd + nkv * vd:
+    paged cache.  qkv float32 [rows, nh * hd + nkv * hd + nkv * vd].  ``bias`` (float32, of that width) is added first;
+    ``neighbour``: channel 2i of a head turns with channel 2i + 1 (default: i with i + rot / 2); ``inv_freq_lo``: what 32-bit
+    leaves out of the frequencies."""
+    if qkv.shape[1] != nh * hd + nkv * hd + nkv * vd or (bias is not None and bias.shape[0] != qkv.shape[1]):
         raise Backend("widenorm_rope_kvwrite: the projection's width does not fit the head sizes")
     if rot and (inv_freq is None or inv_freq.shape[0] < rot // 2):
         raise Backend("widenorm_rope_kvwrite: too few frequencies")
     _check(_fn("core", "esp_widenorm_rope_kvwrite")(
-        _ptr(qkv, torch.float32, "qkv"), _ptr(q_w, torch.float32, "q_w"), _ptr(k_w, torch.float32, "k_w"), float(eps),
-        _ptr(inv_freq, torch.float32, "inv_freq"), int(rot), float(v_scale), _ptr(tok_seq, torch.int32),
+        _ptr(qkv, torch.float32, "qkv"), _ptr(bias, torch.float32, "bias"), _ptr(q_w, torch.float32, "q_w"),
+        _ptr(k_w, torch.float32, "k_w"), float(eps), _ptr(inv_freq, torch.float32, "inv_freq"),
+        _ptr(inv_freq_lo, torch.float32, "inv_freq_lo"), int(rot), 1 if neighbour else 0, float(v_scale), _ptr(tok_seq, torch.int32),
         _ptr(tok_pos, torch.int32), _ptr(q_out, FLOATS, "q_out"), _ptr(k_cache, q_out.dtype, "k_cache"),
         _ptr(v_cache, q_out.dtype, "v_cache"), _is_bf16(q_out), _ptr(block_table, torch.int32), block_table.shape[1],
         k_cache.shape[0], page, qkv.shape[0], nh, nkv, hd, vd, 1 if write_kv else 0, _ptr(status, torch.int32), _stream()),
@@ -1341,9 +1373,9 @@ def heads_to_pages(k, v, tok_seq, tok_pos, table, k_pool, v_pool, page, heads, k
 
 
 def pair_rope_unitnorm_kvwrite(qkv, bias, inv_freq, rot, eps, unit_norm, v_shared, blend_mode, blend, tok_seq, tok_pos, q_out,
-                               k_cache, v_cache, block_table, page, nh, nkv, hd, vd, write_kv, status):
+                               k_cache, v_cache, block_table, page, nh, nkv, hd, vd, write_kv, status, inv_freq_lo=None):
     """Bias, rotation of neighbouring channel pairs (2i with 2i + 1) of the first ``rot`` channels of every query and key
-    head by position * inv_freq[i], every head then divided by its root mean square (``unit_norm``), values copied to
+    head by position * (inv_freq[i] + inv_freq_lo[i]), every head then divided by its root mean square (``unit_norm``), values copied to
     (blend_mode 1) or blended with (blend_mode 2: (1 - blend) v + blend v_shared, ``blend`` a float32 tensor of one
     element on the device) the float32 rows v_shared [rows, nkv * vd]; queries to q_out, keys and values to the paged
     cache.  qkv float32 [rows, nh * hd + nkv * hd + nkv * vd]."""
@@ -1354,8 +1386,8 @@ def pair_rope_unitnorm_kvwrite(qkv, bias, inv_freq, rot, eps, unit_norm, v_share
     if blend_mode and (v_shared is None or v_shared.numel() < qkv.shape[0] * nkv * vd):
         raise Backend("pair_rope_unitnorm_kvwrite: the shared value rows are missing or too small")
     _check(_fn("core", "esp_pair_rope_unitnorm_kvwrite")(
-        _ptr(qkv, torch.float32, "qkv"), _ptr(bias, torch.float32, "bias"), _ptr(inv_freq, torch.float32, "inv_freq"), int(rot),
-        float(eps), 1 if unit_norm else 0, _ptr(v_shared, torch.float32, "v_shared"), int(blend_mode),
+        _ptr(qkv, torch.float32, "qkv"), _ptr(bias, torch.float32, "bias"), _ptr(inv_freq, torch.float32, "inv_freq"),
+        _ptr(inv_freq_lo, torch.float32, "inv_freq_lo"), int(rot), float(eps), 1 if unit_norm else 0, _ptr(v_shared, torch.float32, "v_shared"), int(blend_mode),
         _ptr(blend, torch.float32, "blend"), _ptr(tok_seq, torch.int32), _ptr(tok_pos, torch.int32), _ptr(q_out, FLOATS, "q_out"),
         _ptr(k_cache, q_out.dtype, "k_cache"), _ptr(v_cache, q_out.dtype, "v_cache"), _is_bf16(q_out),
         _ptr(block_table, torch.int32), block_table.shape[1], k_cache.shape[0], page, qkv.shape[0], nh, nkv, hd, vd,

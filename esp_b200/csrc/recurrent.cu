@@ -115,7 +115,10 @@ constexpr int MAX_K = 16 * KT;  // key channels of a head that the kernel takes
 enum : int {
     GATE_EXP_EXP = 0,       // d = exp(-exp(g + bias));  k, q as given;  o reads S_(t-1) + diag(bonus) k v^T
     GATE_LOWER_SIGMOID = 1, // d = lower + (1 - lower) * sigmoid(g + bias);  k = 1 - d;  q = silu(q);  o reads S_t
-    GATE_SCALAR = 2         // d is one number per head and token, ready made (g: [rows, H]);  k, q as given;  o reads S_t
+    GATE_SCALAR = 2,        // d is one number per head and token, ready made (g: [rows, H]);  k, q as given;  o reads S_t
+    GATE_FIXED = 3          // d is one number per head, g[h] + lower[h] (the second what 32-bit leaves out of the first: the same
+                            // factor over and over would add its rounding up);  q, k, v are SiLUs of what is given (READY: as
+                            // given);  o reads S_t
 };
 
 // The gates, written with explicit operations so that the kernel that makes them ahead of the recurrence and the
@@ -154,6 +157,7 @@ gated_scan_kernel(const float* __restrict__ q, long long ldq, const float* __res
     const int buf_floats = CHUNK * (3 * kp + vt);
     const int b = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * vt;
     const int tid = threadIdx.x, nthreads = blockDim.x;
+    constexpr bool LOADS_K = MODE != GATE_LOWER_SIGMOID || READY, LOADS_D = MODE == GATE_EXP_EXP || MODE == GATE_LOWER_SIGMOID;
     const int part = tid % ks, col = (tid / ks) * CPT;   // neighbouring lanes hold the slices of one pair of columns
     const int vcol = v0 + col;
     bool live[CPT];
@@ -168,7 +172,7 @@ gated_scan_kernel(const float* __restrict__ q, long long ldq, const float* __res
     for (int i = tid; i < ks * KT; i += nthreads) {
         const bool in = i < K;
         c_bias[i] = in && gate_bias ? gate_bias[h * K + i] : 0.f;
-        c_lower[i] = in && lower ? lower[h * K + i] : 0.f;
+        c_lower[i] = in && lower && LOADS_D ? lower[h * K + i] : 0.f;
         c_bonus[i] = in && bonus ? bonus[h * K + i] : 1.f;
     }
     // zero the padding of both buffers once (cp.async never writes it)
@@ -183,13 +187,13 @@ gated_scan_kernel(const float* __restrict__ q, long long ldq, const float* __res
         for (int i = 0; i < KT; i++) S[j][i] = (live[j] && part * KT + i < K) ? srow[(size_t)j * K + i] : 0.f;
 
     // 16-byte copies where every row piece is aligned (the usual case: K, V and the row strides multiples of 4)
-    const bool wide = (K % 4 == 0) && (V % 4 == 0) && (vt % 4 == 0) && (ldq % 4 == 0) && (MODE == GATE_SCALAR || ldg % 4 == 0) &&
-                      (ldv % 4 == 0) && (!(MODE == GATE_EXP_EXP || READY) || ldk % 4 == 0) &&
-                      ((((size_t)q | (size_t)(MODE == GATE_SCALAR ? q : g) | (size_t)v |
-                         (size_t)((MODE == GATE_EXP_EXP || READY) ? k : q)) & 15) == 0);
+    const bool wide = (K % 4 == 0) && (V % 4 == 0) && (vt % 4 == 0) && (ldq % 4 == 0) && (!LOADS_D || ldg % 4 == 0) &&
+                      (ldv % 4 == 0) && (!LOADS_K || ldk % 4 == 0) &&
+                      ((((size_t)q | (size_t)(LOADS_D ? g : q) | (size_t)v | (size_t)(LOADS_K ? k : q)) & 15) == 0);
     float bonus_r[KT];
 #pragma unroll
     for (int i = 0; i < KT; i++) bonus_r[i] = c_bonus[part * KT + i];
+    const float d_fixed = MODE == GATE_FIXED ? g[h] : 0.f, d_rest = MODE == GATE_FIXED ? lower[h] : 0.f;
     auto stage = [&](int buffer, int r0) {
         float* base = smem + buffer * buf_floats;
         const int count = min(CHUNK, row1 - r0);
@@ -199,8 +203,8 @@ gated_scan_kernel(const float* __restrict__ q, long long ldq, const float* __res
                 const int t = i / k4, c = (i - t * k4) * 4;
                 const size_t r = (size_t)(r0 + t);
                 cp_async16(base + t * kp + at(c), q + r * ldq + h * K + c);
-                if (MODE == GATE_EXP_EXP || READY) cp_async16(base + (CHUNK + t) * kp + at(c), k + r * ldk + h * K + c);
-                if (MODE != GATE_SCALAR) cp_async16(base + (2 * CHUNK + t) * kp + at(c), g + r * ldg + h * K + c);
+                if (LOADS_K) cp_async16(base + (CHUNK + t) * kp + at(c), k + r * ldk + h * K + c);
+                if (LOADS_D) cp_async16(base + (2 * CHUNK + t) * kp + at(c), g + r * ldg + h * K + c);
             }
             for (int i = tid; i < count * v4; i += nthreads) {
                 const int t = i / v4, c = (i - t * v4) * 4;
@@ -211,8 +215,8 @@ gated_scan_kernel(const float* __restrict__ q, long long ldq, const float* __res
                 const int t = i / K, c = i - t * K;
                 const size_t r = (size_t)(r0 + t);
                 cp_async4(base + t * kp + at(c), q + r * ldq + h * K + c);
-                if (MODE == GATE_EXP_EXP || READY) cp_async4(base + (CHUNK + t) * kp + at(c), k + r * ldk + h * K + c);
-                if (MODE != GATE_SCALAR) cp_async4(base + (2 * CHUNK + t) * kp + at(c), g + r * ldg + h * K + c);
+                if (LOADS_K) cp_async4(base + (CHUNK + t) * kp + at(c), k + r * ldk + h * K + c);
+                if (LOADS_D) cp_async4(base + (2 * CHUNK + t) * kp + at(c), g + r * ldg + h * K + c);
             }
             for (int i = tid; i < count * vt; i += nthreads) {
                 const int t = i / vt, c = i - t * vt;
@@ -237,6 +241,11 @@ gated_scan_kernel(const float* __restrict__ q, long long ldq, const float* __res
             // gates, in place
             for (int i = tid; i < count * K; i += nthreads) {
                 const int t = i / K, c = i - t * K, p = t * kp + at(c);
+                if (MODE == GATE_FIXED) {
+                    sq[p] = gate_silu(sq[p]);
+                    sk[p] = gate_silu(sk[p]);
+                    continue;
+                }
                 const float raw = __fadd_rn(sd[p], c_bias[c]);
                 if (MODE == GATE_EXP_EXP) {
                     sd[p] = gate_decay(raw);
@@ -247,6 +256,8 @@ gated_scan_kernel(const float* __restrict__ q, long long ldq, const float* __res
                     sq[p] = gate_silu(sq[p]);
                 }
             }
+            if (MODE == GATE_FIXED)
+                for (int i = tid; i < count * vt; i += nthreads) sv[i] = gate_silu(sv[i]);
             __syncthreads();
         }
 #pragma unroll SCAN_UNROLL
@@ -255,7 +266,7 @@ gated_scan_kernel(const float* __restrict__ q, long long ldq, const float* __res
             const float4* tk = reinterpret_cast<const float4*>(sk + t * kp + part * KTP);
             const float4* td = reinterpret_cast<const float4*>(sd + t * kp + part * KTP);
             float vv[CPT], oe[CPT][4];
-            const float d_all = MODE == GATE_SCALAR ? sd[t * kp] : 0.f;
+            const float d_all = MODE == GATE_SCALAR ? sd[t * kp] : d_fixed;
 #pragma unroll
             for (int j = 0; j < CPT; j++) {
                 vv[j] = live[j] ? sv[t * vt + col + j] : 0.f;
@@ -263,7 +274,7 @@ gated_scan_kernel(const float* __restrict__ q, long long ldq, const float* __res
             }
 #pragma unroll
             for (int i4 = 0; i4 < KT / 4; i4++) {
-                const float4 q4 = tq[i4], k4 = tk[i4], d4 = MODE == GATE_SCALAR ? make_float4(d_all, d_all, d_all, d_all) : td[i4];
+                const float4 q4 = tq[i4], k4 = tk[i4], d4 = LOADS_D ? td[i4] : make_float4(d_all, d_all, d_all, d_all);
                 const float qe[4] = {q4.x, q4.y, q4.z, q4.w}, ke[4] = {k4.x, k4.y, k4.z, k4.w}, de[4] = {d4.x, d4.y, d4.z, d4.w};
 #pragma unroll
                 for (int e = 0; e < 4; e++) {
@@ -275,7 +286,7 @@ gated_scan_kernel(const float* __restrict__ q, long long ldq, const float* __res
                             oe[j][e] = fmaf(qe[e], fmaf(bonus_r[i], a, S[j][i]), oe[j][e]);
                             S[j][i] = fmaf(de[e], S[j][i], a);
                         } else {
-                            S[j][i] = fmaf(de[e], S[j][i], a);
+                            S[j][i] = fmaf(de[e], S[j][i], MODE == GATE_FIXED ? fmaf(d_rest, S[j][i], a) : a);
                             oe[j][e] = fmaf(qe[e], S[j][i], oe[j][e]);
                         }
                     }
@@ -371,6 +382,41 @@ __global__ void head_rmsnorm_gate_kernel(const float* __restrict__ o, const floa
             r *= (gate_sigmoid ? 1.0f : z) / (1.0f + expf(-z));
         }
         y[((size_t)n * H + h) * V + i] = from_f32<T>(r);
+    }
+}
+
+// The same for rows of more than 256 channels: a block per (row, head), up to four pieces of four channels a thread in
+// registers.  V and the rows' strides are multiples of four, V is at most 16,384.
+template <typename T>
+__global__ void __launch_bounds__(1024)
+row_rmsnorm_gate_kernel(const float* __restrict__ o, const float* __restrict__ w, int w_head_stride,
+                        const float* __restrict__ gate, long long ldgate, T* __restrict__ y, int H, int V, float eps,
+                        int gate_sigmoid) {
+    pdl_trigger();
+    pdl_wait();
+    __shared__ float scratch[33];
+    const int n = blockIdx.x / H, h = blockIdx.x - n * H, pieces = V / 4;
+    const float4* src = reinterpret_cast<const float4*>(behind_wait(o) + ((size_t)n * H + h) * V);
+    const float4* gsrc = gate ? reinterpret_cast<const float4*>(gate + (size_t)n * ldgate + (size_t)h * V) : nullptr;
+    float4 v[4], z[4];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        const int q = threadIdx.x + i * blockDim.x;
+        if (q >= pieces) continue;
+        v[i] = src[q];
+        if (gate) z[i] = gsrc[q];
+        ss = fmaf(v[i].w, v[i].w, fmaf(v[i].z, v[i].z, fmaf(v[i].y, v[i].y, fmaf(v[i].x, v[i].x, ss))));
+    }
+    const float inv = 1.0f / sqrtf(block_sum(ss, scratch) / (float)V + eps);
+    auto gated = [&](float r, float zz) { return gate ? r * (gate_sigmoid ? 1.0f : zz) / (1.0f + expf(-zz)) : r; };
+#pragma unroll
+    for (int i = 0; i < 4; i++) {
+        const int q = threadIdx.x + i * blockDim.x;
+        if (q >= pieces) continue;
+        const float4 g = reinterpret_cast<const float4*>(w + (size_t)h * w_head_stride)[q];
+        Vec4<T>::store(y + ((size_t)n * H + h) * V + 4 * q, gated(v[i].x * inv * g.x, z[i].x), gated(v[i].y * inv * g.y, z[i].y),
+                       gated(v[i].z * inv * g.z, z[i].z), gated(v[i].w * inv * g.w, z[i].w));
     }
 }
 
@@ -693,6 +739,7 @@ ESP_API int esp_gate_prepare(int mode, const float* q, long long ldq, const floa
 
 // mode: 0 = decay exp(-exp(.)) with an extra weight on the token being read, 1 = lower-bounded sigmoid gate that also writes,
 // 2 (with ready) = one ready-made decay per head and token, g being [rows, H]; q and k as given, the output reads S_t.
+// 3 = one decay per head, g and lower being [H] (see GATE_FIXED).
 // ready: q, k and g already hold the query, the written key and the decay (esp_gate_prepare made them).
 ESP_API int esp_gated_scan(int mode, int ready, const float* q, long long ldq, const float* k, long long ldk, const float* g,
                            long long ldg, const float* v, long long ldv, const float* gate_bias, const float* lower,
@@ -710,7 +757,7 @@ ESP_API int esp_gated_scan(int mode, int ready, const float* q, long long ldq, c
     const int vtiles = (V + vt - 1) / vt;
     const size_t smem = 2 * (size_t)CHUNK * (3 * ks * KTP + vt) * sizeof(float);
     dim3 grid(n_seqs, H, vtiles);
-    if ((mode == GATE_EXP_EXP || ready) && !k) return (int)cudaErrorInvalidValue;
+    if ((mode == GATE_EXP_EXP || mode == GATE_FIXED || ready) && !k) return (int)cudaErrorInvalidValue;
 #define ESP_SCAN(MODE_, READY_)                                                                                              \
     {                                                                                                                       \
         auto kernel = gated_scan_kernel<MODE_, READY_>;                                                                     \
@@ -720,7 +767,10 @@ ESP_API int esp_gated_scan(int mode, int ready, const float* q, long long ldq, c
         esp_launch_pdl(READY_ ? 0 : ESP_PDL_SMALL, kernel, grid, dim3(threads), smem, stream, q, ldq, k, ldk, g, ldg, v, ldv, \
                        gate_bias, lower, bonus, state, state_stride, seq_start, seq_slot, out, H, K, V, ks, vt);            \
     }
+    if (mode == GATE_FIXED && (!g || !lower)) return (int)cudaErrorInvalidValue;
     if (mode == GATE_SCALAR && ready) ESP_SCAN(GATE_SCALAR, true)
+    else if (mode == GATE_FIXED && ready) ESP_SCAN(GATE_FIXED, true)
+    else if (mode == GATE_FIXED) ESP_SCAN(GATE_FIXED, false)
     else if (mode == GATE_EXP_EXP && !ready) ESP_SCAN(GATE_EXP_EXP, false)
     else if (mode == GATE_EXP_EXP) ESP_SCAN(GATE_EXP_EXP, true)
     else if (mode == GATE_LOWER_SIGMOID && !ready) ESP_SCAN(GATE_LOWER_SIGMOID, false)
@@ -735,6 +785,17 @@ ESP_API int esp_head_rmsnorm_gate(const float* o, const float* w, int w_head_str
                                   cudaStream_t stream) {
     if (n_rows <= 0) return 0;
     const long long warps = (long long)n_rows * H;
+    const size_t ptrs = (size_t)o | (size_t)w | (size_t)gate | (size_t)y;
+    if (V > 256 && V % 4 == 0 && V <= 16384 && w_head_stride % 4 == 0 && ldgate % 4 == 0 && (ptrs & 15) == 0) {
+        const int threads = V <= 4096 ? (V / 4 + 31) / 32 * 32 : 1024;
+        if (y_is_bf16)
+            esp_launch_pdl(ESP_PDL_SMALL, row_rmsnorm_gate_kernel<bf16>, dim3((unsigned)warps), dim3(threads), 0, stream, o, w,
+                           w_head_stride, gate, ldgate, (bf16*)y, H, V, eps, gate_sigmoid);
+        else
+            esp_launch_pdl(ESP_PDL_SMALL, row_rmsnorm_gate_kernel<float>, dim3((unsigned)warps), dim3(threads), 0, stream, o, w,
+                           w_head_stride, gate, ldgate, (float*)y, H, V, eps, gate_sigmoid);
+        return esp_launch_status();
+    }
     const int blocks = (int)((warps + 7) / 8);
     if (y_is_bf16)
         esp_launch_pdl(ESP_PDL_SMALL, head_rmsnorm_gate_kernel<bf16>, dim3(blocks), dim3(256), 0, stream, o, w, w_head_stride,

@@ -13,6 +13,18 @@
 // block_table[seq * table_stride + p / PAGE].
 #include "common.cuh"
 
+// Sine and cosine of position * frequency in 32-bit, the frequency given as the sum of two floats: what the product's
+// rounding and the frequency's own leave out (p times 2^-24 of a turn's radians, more than a score's other errors from a
+// few hundred positions on) is put back, to second order.
+__device__ __forceinline__ void angle_sincos(float p, float f, float f_lo, float& sn, float& cs) {
+    const float a = __fmul_rn(p, f), e = fmaf(p, f_lo, fmaf(p, f, -a));
+    float s0, c0;
+    sincosf(a, &s0, &c0);
+    const float h = -0.5f * e * e;
+    sn = fmaf(e, c0, fmaf(h, s0, s0));
+    cs = fmaf(-e, s0, fmaf(h, c0, c0));
+}
+
 template <typename T>
 __global__ void rope_kvwrite_kernel(const float* __restrict__ qkv, const float* __restrict__ bias,
                                     const int* __restrict__ tok_seq,
@@ -261,17 +273,19 @@ ESP_API int esp_qknorm_kvwrite(const float* qkv, const float* bias, const float*
 }
 
 // ---------------------------------------------------------------- norms over the whole projection, partial rotation
-// qkv: [n_tokens, nh*hd + nkv*hd + nkv*vd] float.  The queries of a token, all heads together, are divided by their
+// qkv: [n_tokens, nh*hd + nkv*hd + nkv*vd] float; ``bias`` (same width, may be null) is added first.  The queries of a token, all heads together, are divided by their
 // root mean square over the nh*hd channels (eps inside the root) and multiplied by a weight per channel (q_w, nh*hd
 // numbers); the keys likewise over nkv*hd channels with k_w (null: that side is left as projected).  Then the first
-// ``rot`` channels of every head are rotated, channel i with channel i + rot/2, by the angle position * inv_freq[i]
-// (a 32-bit product; sine and cosine in 32-bit); the other channels pass unchanged.  Values are multiplied by v_scale.
+// ``rot`` channels of every head are rotated, channel i with channel i + rot/2 (NEIGHBOUR: channel 2i with channel 2i + 1),
+// by the angle position * (inv_freq[i] + inv_freq_lo[i]) (angle_sincos; inv_freq_lo may be null); the other channels pass
+// unchanged.  Values are multiplied by v_scale.
 // Queries go to q_out [n_tokens, nh, hd], keys [pages, nkv, PAGE, hd] and values [pages, nkv, PAGE, vd] to the
 // token's place in the paged cache.  One block per token.
-template <typename T>
-__global__ void widenorm_rope_kvwrite_kernel(const float* __restrict__ qkv, const float* __restrict__ q_w,
+template <typename T, bool NEIGHBOUR>
+__global__ void widenorm_rope_kvwrite_kernel(const float* __restrict__ qkv, const float* __restrict__ bias,
+                                             const float* __restrict__ q_w,
                                              const float* __restrict__ k_w, float eps, const float* __restrict__ inv_freq,
-                                             int rot, float v_scale, const int* __restrict__ tok_seq,
+                                             const float* __restrict__ inv_freq_lo, int rot, float v_scale, const int* __restrict__ tok_seq,
                                              const int* __restrict__ tok_pos, T* __restrict__ q_out, T* __restrict__ k_cache,
                                              T* __restrict__ v_cache, const int* __restrict__ block_table, int table_stride,
                                              int n_pages, int page, int nh, int nkv, int hd, int vd, int write_kv,
@@ -293,8 +307,9 @@ __global__ void widenorm_rope_kvwrite_kernel(const float* __restrict__ qkv, cons
     }
     const int in_page = pos % page;
     float ssq = 0.f, ssk = 0.f;
-    for (int e = tid; e < qw; e += blockDim.x) ssq = fmaf(src[e], src[e], ssq);
-    for (int e = tid; e < kw; e += blockDim.x) ssk = fmaf(src[qw + e], src[qw + e], ssk);
+    auto at = [&](int e) { return src[e] + (bias ? bias[e] : 0.f); };
+    for (int e = tid; e < qw; e += blockDim.x) ssq = fmaf(at(e), at(e), ssq);
+    for (int e = qw + tid; e < qw + kw; e += blockDim.x) ssk = fmaf(at(e), at(e), ssk);
     const float inv_q = q_w ? 1.0f / sqrtf(block_sum(ssq, scratch) / (float)qw + eps) : 1.0f;
     const float inv_k = k_w ? 1.0f / sqrtf(block_sum(ssk, scratch) / (float)kw + eps) : 1.0f;
     const int half = rot / 2;
@@ -302,27 +317,30 @@ __global__ void widenorm_rope_kvwrite_kernel(const float* __restrict__ qkv, cons
     // the row's angles are the same for every head: their cosines and sines are made once (dynamic shared memory:
     // rot floats), from the same expression a head of its own would evaluate
     extern __shared__ float rot_cs[];
-    for (int c = tid; c < half; c += blockDim.x) sincosf(p * inv_freq[c], &rot_cs[half + c], &rot_cs[c]);
+    for (int c = tid; c < half; c += blockDim.x)
+        angle_sincos(p, inv_freq[c], inv_freq_lo ? inv_freq_lo[c] : 0.f, rot_cs[half + c], rot_cs[c]);
     __syncthreads();
     for (int e = tid; e < qw + kw; e += blockDim.x) {
         const bool is_q = e < qw;
         const int local = is_q ? e : e - qw;
         const int head = local / hd, c = local - head * hd;
-        if (c >= half && c < rot) continue;               // the second half of a pair is written with the first
+        const bool turns = c < rot;
+        if (turns && (NEIGHBOUR ? (c & 1) : c >= half)) continue;          // the second channel of a pair is written with the first
+        const int far = NEIGHBOUR ? 1 : half, pair = NEIGHBOUR ? c >> 1 : c;
         const float* w = is_q ? q_w : k_w;
         const float inv = is_q ? inv_q : inv_k;
         T* dst;
         if (is_q) dst = q_out + ((size_t)n * nh + head) * hd;
         else if (page_id >= 0) dst = k_cache + (((size_t)page_id * nkv + head) * page + in_page) * hd;
         else continue;
-        float a = src[e];
+        float a = at(e);
         if (w) a = a * inv * w[local];
-        if (c < half) {
-            float b = src[e + half];
-            if (w) b = b * inv * w[local + half];
-            const float cs = rot_cs[c], sn = rot_cs[half + c];
+        if (turns) {
+            float b = at(e + far);
+            if (w) b = b * inv * w[local + far];
+            const float cs = rot_cs[pair], sn = rot_cs[half + pair];
             dst[c] = from_f32<T>(a * cs - b * sn);
-            dst[c + half] = from_f32<T>(b * cs + a * sn);
+            dst[c + far] = from_f32<T>(b * cs + a * sn);
         } else {
             dst[c] = from_f32<T>(a);
         }
@@ -330,21 +348,23 @@ __global__ void widenorm_rope_kvwrite_kernel(const float* __restrict__ qkv, cons
     if (page_id >= 0) {
         for (int e = tid; e < vw; e += blockDim.x) {
             const int head = e / vd, c = e - head * vd;
-            v_cache[(((size_t)page_id * nkv + head) * page + in_page) * vd + c] = from_f32<T>(src[qw + kw + e] * v_scale);
+            v_cache[(((size_t)page_id * nkv + head) * page + in_page) * vd + c] = from_f32<T>(at(qw + kw + e) * v_scale);
         }
     }
 }
 
-// The same for head sizes, value sizes and half a rotation of whole pieces of four channels, and aligned buffers.  The
+// The same for head sizes and value sizes (and, where the halves of a rotation are partners, half a rotation) of whole
+// pieces of four channels, and aligned buffers.  The
 // row's query and key part is read once, in 16-byte loads, into shared memory (the sums of squares are taken on the
 // way, both reduced in one exchange).  A thread then makes four
 // neighbouring channels and, where they are rotated, their four partners, and stores each as one piece.  Per element the
 // arithmetic is that of the kernel above; only the order in which the squares are added differs.
 // Dynamic shared memory: (nh * hd + nkv * hd + rot) floats.
-template <typename T>
+template <typename T, bool NEIGHBOUR>
 __global__ void __launch_bounds__(256)
-widenorm_rope_kvwrite_vec_kernel(const float* __restrict__ qkv, const float* __restrict__ q_w,
-                                 const float* __restrict__ k_w, float eps, const float* __restrict__ inv_freq, int rot,
+widenorm_rope_kvwrite_vec_kernel(const float* __restrict__ qkv, const float* __restrict__ bias, const float* __restrict__ q_w,
+                                 const float* __restrict__ k_w, float eps, const float* __restrict__ inv_freq,
+                                 const float* __restrict__ inv_freq_lo, int rot,
                                  float v_scale, const int* __restrict__ tok_seq, const int* __restrict__ tok_pos,
                                  T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache,
                                  const int* __restrict__ block_table, int table_stride, int n_pages, int page, int nh,
@@ -359,7 +379,8 @@ widenorm_rope_kvwrite_vec_kernel(const float* __restrict__ qkv, const float* __r
     pdl_wait();
     const int pos = tok_pos[n], seq = tok_seq[n];
     const float p = (float)pos;
-    for (int c = tid; c < half; c += blockDim.x) sincosf(p * inv_freq[c], &rot_cs[half + c], &rot_cs[c]);
+    for (int c = tid; c < half; c += blockDim.x)
+        angle_sincos(p, inv_freq[c], inv_freq_lo ? inv_freq_lo[c] : 0.f, rot_cs[half + c], rot_cs[c]);
     int page_id = -1;
     if (write_kv) {
         page_id = block_table[(size_t)seq * table_stride + pos / page];
@@ -369,10 +390,18 @@ widenorm_rope_kvwrite_vec_kernel(const float* __restrict__ qkv, const float* __r
         }
     }
     const int in_page = pos % page;
-    const float* src = qkv + (size_t)n * (qw + kw + vw);
+    const float* src = behind_wait(qkv) + (size_t)n * (qw + kw + vw);
+    auto piece = [&](int e) {
+        float4 v = *reinterpret_cast<const float4*>(src + e);
+        if (bias) {
+            const float4 b = *reinterpret_cast<const float4*>(bias + e);
+            v.x += b.x, v.y += b.y, v.z += b.z, v.w += b.w;
+        }
+        return v;
+    };
     float ssq = 0.f, ssk = 0.f;
     for (int e = 4 * tid; e < qw + kw; e += 4 * blockDim.x) {
-        const float4 v = *reinterpret_cast<const float4*>(src + e);
+        const float4 v = piece(e);
         *reinterpret_cast<float4*>(row + e) = v;
         const float s4 = fmaf(v.w, v.w, fmaf(v.z, v.z, fmaf(v.y, v.y, v.x * v.x)));
         if (e < qw) ssq += s4; else ssk += s4;
@@ -388,7 +417,7 @@ widenorm_rope_kvwrite_vec_kernel(const float* __restrict__ qkv, const float* __r
         const bool is_q = e < qw;
         const int local = is_q ? e : e - qw;
         const int head = local / hd, c = local - head * hd;
-        if (c >= half && c < rot) continue;               // written with the first halves of their pairs
+        if (!NEIGHBOUR && c >= half && c < rot) continue;   // written with the first halves of their pairs
         const float* w = is_q ? q_w : k_w;
         const float inv = is_q ? inv_q : inv_k;
         T* dst;
@@ -401,7 +430,19 @@ widenorm_rope_kvwrite_vec_kernel(const float* __restrict__ qkv, const float* __r
             const float4 w4 = *reinterpret_cast<const float4*>(w + local);
             a[0] = a[0] * inv * w4.x, a[1] = a[1] * inv * w4.y, a[2] = a[2] * inv * w4.z, a[3] = a[3] * inv * w4.w;
         }
-        if (c < half) {
+        if (NEIGHBOUR) {
+            if (c < rot) {
+                const float cs = rot_cs[c >> 1], sn = rot_cs[half + (c >> 1)], u = a[0];
+                a[0] = u * cs - a[1] * sn;
+                a[1] = a[1] * cs + u * sn;
+            }
+            if (c + 2 < rot) {
+                const float cs = rot_cs[(c >> 1) + 1], sn = rot_cs[half + (c >> 1) + 1], u = a[2];
+                a[2] = u * cs - a[3] * sn;
+                a[3] = a[3] * cs + u * sn;
+            }
+            Vec4<T>::store(dst + c, a[0], a[1], a[2], a[3]);
+        } else if (c < half) {
             const float4 b4 = *reinterpret_cast<const float4*>(row + e + half);
             float b[4] = {b4.x, b4.y, b4.z, b4.w};
             if (w) {
@@ -424,52 +465,50 @@ widenorm_rope_kvwrite_vec_kernel(const float* __restrict__ qkv, const float* __r
     if (page_id >= 0) {
         for (int e = 4 * tid; e < vw; e += 4 * blockDim.x) {
             const int head = e / vd, c = e - head * vd;
-            const float4 v = *reinterpret_cast<const float4*>(src + qw + kw + e);
+            const float4 v = piece(qw + kw + e);
             Vec4<T>::store(v_cache + (((size_t)page_id * nkv + head) * page + in_page) * vd + c, v.x * v_scale, v.y * v_scale,
                            v.z * v_scale, v.w * v_scale);
         }
     }
 }
 
-ESP_API int esp_widenorm_rope_kvwrite(const float* qkv, const float* q_w, const float* k_w, float eps, const float* inv_freq,
-                                      int rot, float v_scale, const int* tok_seq, const int* tok_pos, void* q_out,
-                                      void* k_cache, void* v_cache, int is_bf16, const int* block_table, int table_stride,
-                                      int n_pages, int page, int n_tokens, int nh, int nkv, int hd, int vd, int write_kv,
-                                      int* status, cudaStream_t stream) {
+// ``neighbour``: channel 2i of a head is rotated with channel 2i + 1 instead of channel i with channel i + rot/2.
+ESP_API int esp_widenorm_rope_kvwrite(const float* qkv, const float* bias, const float* q_w, const float* k_w, float eps,
+                                      const float* inv_freq, const float* inv_freq_lo, int rot, int neighbour, float v_scale,
+                                      const int* tok_seq, const int* tok_pos, void* q_out, void* k_cache, void* v_cache,
+                                      int is_bf16, const int* block_table, int table_stride, int n_pages, int page, int n_tokens,
+                                      int nh, int nkv, int hd, int vd, int write_kv, int* status, cudaStream_t stream) {
     if (n_tokens <= 0) return 0;
     if (hd <= 0 || vd <= 0 || nkv <= 0 || nh <= 0 || page <= 0 || rot < 0 || rot > hd || rot % 2 != 0 || (rot > 0 && !inv_freq))
         return (int)cudaErrorInvalidValue;
     const int threads = (nh + nkv) * hd >= 2048 ? 256 : 128;
     // which form runs depends on the sizes and the buffers' alignment alone, never on the rows of a step
     const size_t row_bytes = (size_t)((nh + nkv) * hd + rot) * sizeof(float);
-    const size_t ptrs = (size_t)qkv | (size_t)q_w | (size_t)k_w | (size_t)q_out | (size_t)k_cache | (size_t)v_cache;
-    if (hd % 4 == 0 && vd % 4 == 0 && rot % 8 == 0 && (ptrs & 15) == 0 && row_bytes <= 40 * 1024) {
-        if (is_bf16)
-            esp_launch_pdl(ESP_PDL_SMALL, widenorm_rope_kvwrite_vec_kernel<bf16>, dim3(n_tokens), dim3(threads), row_bytes, stream,
-                           qkv, q_w, k_w, eps, inv_freq, rot, v_scale, tok_seq, tok_pos, (bf16*)q_out, (bf16*)k_cache,
-                           (bf16*)v_cache, block_table, table_stride, n_pages, page, nh, nkv, hd, vd, write_kv, status);
-        else
-            esp_launch_pdl(ESP_PDL_SMALL, widenorm_rope_kvwrite_vec_kernel<float>, dim3(n_tokens), dim3(threads), row_bytes, stream,
-                           qkv, q_w, k_w, eps, inv_freq, rot, v_scale, tok_seq, tok_pos, (float*)q_out, (float*)k_cache,
-                           (float*)v_cache, block_table, table_stride, n_pages, page, nh, nkv, hd, vd, write_kv, status);
-        return esp_launch_status();
-    }
-    if (is_bf16)
-        esp_launch_pdl(ESP_PDL_SMALL, widenorm_rope_kvwrite_kernel<bf16>, dim3(n_tokens), dim3(threads), rot * sizeof(float), stream, qkv, q_w, k_w,
-                       eps, inv_freq, rot, v_scale, tok_seq, tok_pos, (bf16*)q_out, (bf16*)k_cache, (bf16*)v_cache, block_table,
-                       table_stride, n_pages, page, nh, nkv, hd, vd, write_kv, status);
-    else
-        esp_launch_pdl(ESP_PDL_SMALL, widenorm_rope_kvwrite_kernel<float>, dim3(n_tokens), dim3(threads), rot * sizeof(float), stream, qkv, q_w, k_w,
-                       eps, inv_freq, rot, v_scale, tok_seq, tok_pos, (float*)q_out, (float*)k_cache, (float*)v_cache,
-                       block_table, table_stride, n_pages, page, nh, nkv, hd, vd, write_kv, status);
+    const size_t ptrs = (size_t)qkv | (size_t)bias | (size_t)q_w | (size_t)k_w | (size_t)q_out | (size_t)k_cache | (size_t)v_cache;
+    const bool vec = hd % 4 == 0 && vd % 4 == 0 && (neighbour || rot % 8 == 0) && (ptrs & 15) == 0 && row_bytes <= 40 * 1024;
+#define ESP_WIDENORM(KERNEL, T, NB)                                                                                          \
+    esp_launch_pdl(ESP_PDL_SMALL, KERNEL<T, NB>, dim3(n_tokens), dim3(threads), vec ? row_bytes : rot * sizeof(float), stream,    \
+                   qkv, bias, q_w, k_w, eps, inv_freq, inv_freq_lo, rot, v_scale, tok_seq, tok_pos, (T*)q_out, (T*)k_cache,       \
+                   (T*)v_cache, block_table, table_stride, n_pages, page, nh, nkv, hd, vd, write_kv, status)
+#define ESP_WIDENORM_T(T)                                                                      \
+    do {                                                                                       \
+        if (vec && neighbour) ESP_WIDENORM(widenorm_rope_kvwrite_vec_kernel, T, true);         \
+        else if (vec) ESP_WIDENORM(widenorm_rope_kvwrite_vec_kernel, T, false);                \
+        else if (neighbour) ESP_WIDENORM(widenorm_rope_kvwrite_kernel, T, true);               \
+        else ESP_WIDENORM(widenorm_rope_kvwrite_kernel, T, false);                             \
+    } while (0)
+    if (is_bf16) ESP_WIDENORM_T(bf16);
+    else ESP_WIDENORM_T(float);
+#undef ESP_WIDENORM_T
+#undef ESP_WIDENORM
     return esp_launch_status();
 }
 
 // ---------------------------------------------------------------- neighbour-pair rotation, unit root mean square per head,
 // values blended with those of an earlier layer
 // qkv: [n_tokens, nh*hd + nkv*hd + nkv*vd] float, bias (may be null) of the same width.  Of the first ``rot`` channels of
-// every query and key head, channel 2i is rotated with channel 2i + 1 by the angle position * inv_freq[i] (a 32-bit
-// product; sine and cosine in 32-bit); the other channels pass unchanged.  With ``unit_norm`` every head is then divided
+// every query and key head, channel 2i is rotated with channel 2i + 1 by the angle position * (inv_freq[i] + inv_freq_lo[i])
+// (angle_sincos; inv_freq_lo may be null); the other channels pass unchanged.  With ``unit_norm`` every head is then divided
 // by its root mean square over hd (eps inside the root; no weight).  Values: blend_mode 1 copies the row's values
 // (bias added, unrounded) to v_shared [n_tokens, nkv*vd]; blend_mode 2 replaces them by (1 - lambda) v + lambda v_shared
 // with lambda read from the device.  Queries go to q_out [n_tokens, nh, hd], keys [pages, nkv, PAGE, hd] and values
@@ -486,7 +525,8 @@ __device__ __forceinline__ void store_pair(bf16* dst, float a, float b) {
 // and stores it as one; else channel by channel.  Which form runs depends on the sizes and the buffers' alignment alone.
 template <typename T, bool PAIRS>
 __global__ void pair_rope_unitnorm_kvwrite_kernel(const float* __restrict__ qkv, const float* __restrict__ bias,
-                                                  const float* __restrict__ inv_freq, int rot, float eps, int unit_norm,
+                                                  const float* __restrict__ inv_freq,
+                                                  const float* __restrict__ inv_freq_lo, int rot, float eps, int unit_norm,
                                                   float* __restrict__ v_shared, int blend_mode,
                                                   const float* __restrict__ lambda, const int* __restrict__ tok_seq,
                                                   const int* __restrict__ tok_pos, T* __restrict__ q_out,
@@ -514,7 +554,8 @@ __global__ void pair_rope_unitnorm_kvwrite_kernel(const float* __restrict__ qkv,
     const float p = (float)pos;
     const int half = rot / 2;
     // the row's angles are the same for every head: their cosines and sines are made once
-    for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(p * inv_freq[i], &rope_cs[half + i], &rope_cs[i]);
+    for (int i = threadIdx.x; i < half; i += blockDim.x)
+        angle_sincos(p, inv_freq[i], inv_freq_lo ? inv_freq_lo[i] : 0.f, rope_cs[half + i], rope_cs[i]);
     __syncthreads();
     constexpr int PER = PAIR_ROPE_MAX_HD / 64;             // pairs of channels a lane holds
     for (int head = warp; head < nh + 2 * nkv; head += nwarp) {
@@ -607,8 +648,8 @@ __global__ void pair_rope_unitnorm_kvwrite_kernel(const float* __restrict__ qkv,
 }
 }  // namespace
 
-ESP_API int esp_pair_rope_unitnorm_kvwrite(const float* qkv, const float* bias, const float* inv_freq, int rot, float eps,
-                                           int unit_norm, float* v_shared, int blend_mode, const float* lambda,
+ESP_API int esp_pair_rope_unitnorm_kvwrite(const float* qkv, const float* bias, const float* inv_freq,
+                                           const float* inv_freq_lo, int rot, float eps, int unit_norm, float* v_shared, int blend_mode, const float* lambda,
                                            const int* tok_seq, const int* tok_pos, void* q_out, void* k_cache, void* v_cache,
                                            int is_bf16, const int* block_table, int table_stride, int n_pages, int page,
                                            int n_tokens, int nh, int nkv, int hd, int vd, int write_kv, int* status,
@@ -625,8 +666,8 @@ ESP_API int esp_pair_rope_unitnorm_kvwrite(const float* qkv, const float* bias, 
     const bool pairs = hd % 2 == 0 && vd % 2 == 0 && (ptrs & 7) == 0;
 #define ESP_PAIR_ROPE(T, PAIRS)                                                                                              \
     esp_launch_pdl(ESP_PDL_SMALL, pair_rope_unitnorm_kvwrite_kernel<T, PAIRS>, dim3(n_tokens), dim3(threads), smem, stream, qkv,  \
-                   bias, inv_freq, rot, eps, unit_norm, v_shared, blend_mode, lambda, tok_seq, tok_pos, (T*)q_out, (T*)k_cache,    \
-                   (T*)v_cache, block_table, table_stride, n_pages, page, nh, nkv, hd, vd, write_kv, status)
+                   bias, inv_freq, inv_freq_lo, rot, eps, unit_norm, v_shared, blend_mode, lambda, tok_seq, tok_pos, (T*)q_out,    \
+                   (T*)k_cache, (T*)v_cache, block_table, table_stride, n_pages, page, nh, nkv, hd, vd, write_kv, status)
     if (is_bf16) {
         if (pairs) ESP_PAIR_ROPE(bf16, true);
         else ESP_PAIR_ROPE(bf16, false);
@@ -649,17 +690,6 @@ ESP_API int esp_pair_rope_unitnorm_kvwrite(const float* qkv, const float* bias, 
 // in the paged cache.  One block per token; a row's queries and keys are staged in shared memory.
 // VEC 4: sizes are whole pieces of four channels and the buffers aligned to them; VEC 1: any sizes.  Which form runs
 // depends on the sizes and the alignment alone.  Dynamic shared memory: (staged channels + rotated runs + rot) floats.
-
-// Sine and cosine of position * frequency in 32-bit, the frequency given as the sum of two floats: what the product's
-// rounding and the frequency's own leave out (p times 2^-24 of a turn's radians, more than a score's other errors from a
-// few hundred positions on) is put back to first order.
-__device__ __forceinline__ void angle_sincos(float p, float f, float f_lo, float& sn, float& cs) {
-    const float a = __fmul_rn(p, f), e = fmaf(p, f_lo, fmaf(p, f, -a));
-    float s0, c0;
-    sincosf(a, &s0, &c0);
-    sn = fmaf(e, c0, s0);
-    cs = fmaf(-e, s0, c0);
-}
 
 template <typename T, int VEC>
 __global__ void __launch_bounds__(256)

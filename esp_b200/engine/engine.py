@@ -370,7 +370,7 @@ class Engine:
                 # the keys the sequence's last new token sees: every kernel streams a sequence's visible keys once
                 last = p + t
                 span = layout.window if layout.window is not None else layout.chunk
-                seen += last if span is None else min(last, span + t - 1)
+                seen += last if span is None else min(last, span + t - 1 + layout.keep_first)
             c["kv_bytes_read"] += seen * per_key
 
     def profile_step(self, entries: list):

@@ -20,13 +20,12 @@ DECODE_ROWS = 128      # steps with at most this many token rows use the split-k
 # which kernel a step of n token rows gets, the index lists it needs, and the launch.  Shared by the parts below.
 def scaled_kernel_for(rt, key_dim: int, value_dim: int, scale: float, n: int, page: int = PAGE) -> str:
     if rt.dtype == torch.bfloat16 and page == PAGE:
-        same = key_dim == value_dim and scale > 0
-        if same and key_dim in (64, 128, 192, 256) and n <= DECODE_ROWS:
+        if scale > 0 and ops.attn_decode_fits(key_dim, value_dim) and n <= DECODE_ROWS:
             return "split"         # few rows: the keys are split over blocks
-        if same and ops.attn_prefill_tc05_fits(key_dim, page):
+        if scale > 0 and ops.attn_prefill_tc05_fits(key_dim, page, value_dim):
             return "tc05"          # many rows: scores and weighted values in tensor memory
         if ops.attn_flash_fits(key_dim, value_dim):
-            return "flash"         # keys and values of different sizes, any multiples of 8 up to 128
+            return "flash"         # a scale that is not positive
     return "plain"
 
 
@@ -46,8 +45,11 @@ def scaled_tiles(kind: str, step) -> dict:
             f"attention.tiles{rows}.first": np.asarray([t[1] for t in tiles], dtype=np.int32)}
 
 
-def scaled_attend(rt, kind, q, o, ctx, layer, num_heads, num_kv_heads, key_dim, value_dim, scale, sink, window=None, chunk=None):
-    """``sink``: False, True (a term exp(0)) or a float32 tensor with a number per head (a term exp(sink_h))."""
+def scaled_attend(rt, kind, q, o, ctx, layer, num_heads, num_kv_heads, key_dim, value_dim, scale, sink, window=None, chunk=None,
+                  keep=0):
+    """``sink``: False, True (a term exp(0)) or a float32 tensor with a number per head (a term exp(sink_h)).  ``keep``
+    (with a window): the sequence's first ``keep`` positions are seen besides."""
+    keep = keep if window else 0
     n = q.shape[0]
     table = ctx.block_tables[layer.group]
     tile_seq = tile_first = None
@@ -62,25 +64,28 @@ def scaled_attend(rt, kind, q, o, ctx, layer, num_heads, num_kv_heads, key_dim, 
         kv_blocks = num_kv_heads * ((group + 15) // 16)
         # a layer with a window or a mask of blocks reads at most that many keys (+ a page) of each row
         seen = window or chunk
-        span = min(positions, seen + layer.page) if seen else positions
-        split = ops.attn_decode_split(n, kv_blocks, span, key_dim, rt.sm_count)
+        span = min(positions, seen + keep + layer.page) if seen else positions
+        tile = ops.attn_decode_tile(key_dim, value_dim)
+        split = ops.attn_decode_split(n, kv_blocks, span, tile, rt.sm_count)
         n_splits = (positions + split - 1) // split
-        part_o = rt.ws.get("attn_part_o", (n, num_heads, n_splits, key_dim), torch.float32)
+        part_o = rt.ws.get("attn_part_o", (n, num_heads, n_splits, tile), torch.float32)
         part_ml = rt.ws.get("attn_part_ml", (n, num_heads, n_splits, 2), torch.float32)
         if getattr(rt, "attn_counters", None) is None:
             rt.attn_counters = torch.zeros(ops.ATTN_DECODE_COUNTERS, dtype=torch.int32, device=rt.device)
         ops.attn_decode(q, layer.k, layer.v, o, part_o, part_ml, rt.attn_counters, ctx.tok_seq, ctx.tok_pos, table, layer.page,
                         num_heads, num_kv_heads, key_dim, window, split, n_splits, rt.status,
-                        seq_past=ctx.seq_past if layer.writes else None, scale=scale, sink=sink, chunk=chunk)
+                        seq_past=ctx.seq_past if layer.writes else None, scale=scale, sink=sink, chunk=chunk, vd=value_dim, keep=keep)
     elif kind == "tc05":
         ops.attn_prefill_tc05(q, layer.k, layer.v, o, tile_seq, tile_first, ctx.seq_start, ctx.seq_past, table, layer.page,
-                              num_heads, num_kv_heads, key_dim, window, rt.status, scale=scale, sink=sink, chunk=chunk)
+                              num_heads, num_kv_heads, key_dim, window, rt.status, scale=scale, sink=sink, chunk=chunk, vd=value_dim,
+                              keep=keep)
     elif kind == "flash":
         ops.attn_prefill(q, layer.k, layer.v, o, tile_seq, tile_first, ctx.seq_start, ctx.seq_past, table, layer.page,
-                         num_heads, num_kv_heads, key_dim, window, rt.status, vd=value_dim, scale=scale, sink=sink, chunk=chunk)
+                         num_heads, num_kv_heads, key_dim, window, rt.status, vd=value_dim, scale=scale, sink=sink, chunk=chunk,
+                         keep=keep)
     else:
         ops.attn_simt(q, layer.k, layer.v, o, ctx.tok_seq, ctx.tok_pos, table, layer.page, num_heads, num_kv_heads,
-                      key_dim, window, rt.status, vd=value_dim, scale=scale, sink=sink, chunk=chunk)
+                      key_dim, window, rt.status, vd=value_dim, scale=scale, sink=sink, chunk=chunk, keep=keep)
 
 
 class Attention(Part):
@@ -157,7 +162,7 @@ class Attention(Part):
         if rt.dtype == torch.bfloat16:
             if s.head_dim in (64, 128, 192, 256) and n <= DECODE_ROWS and page == PAGE:
                 return "split"         # few rows: split the keys over blocks so that the cache streams at full width
-            if ops.attn_prefill_tc05_fits(s.head_dim, page):
+            if s.head_dim in (64, 128) and ops.attn_prefill_tc05_fits(s.head_dim, page):
                 return "tc05"          # many rows, head size 64 or 128: scores and weighted values in tensor memory
             if s.head_dim <= 128 and page == 64:
                 return "flash"
@@ -342,10 +347,10 @@ class NormedAttention(Part):
 
 class WideNormAttention(Part):
     """Causal softmax attention over the paged cache whose query and key norms run over the whole projection (see
-    ``WideNormAttentionSpec``): packed q/k/v projection; one kernel norms queries and keys over all their heads at
+    ``WideNormAttentionSpec``): packed q/k/v projection; one kernel adds the biases, norms queries and keys over all their heads at
     once, rotates the first channels of every head and stores keys (normed and rotated) and values in the cache;
     the attention kernels take the scores' scale as given, a mask of blocks counted from the sequence's start
-    (``chunk``) or a window, and a learned sink per head.  Query head i reads key/value head
+    (``chunk``) or a window with kept first positions, and a learned sink per head.  Query head i reads key/value head
     i // (num_heads / num_kv_heads)."""
 
     graph_safe = True
@@ -364,21 +369,25 @@ class WideNormAttention(Part):
         self.v_width = s.num_kv_heads * s.value_dim
         self.o_width = s.num_heads * s.value_dim
         self.qkv_width = self.q_width + self.k_width + self.v_width
+        if s.keep_first and s.window is None:
+            raise Unsupported("mask", "kept first positions without a window")
         self.position = None
+        self.neighbour = getattr(s.position, "kind", None) == "rope_neighbour_pairs"
         if s.position is not None:
-            if getattr(s.position, "factor", None) is not None:
+            if not self.neighbour and getattr(s.position, "factor", None) is not None:
                 raise Unsupported("rot", "interpolated frequencies on an attention layer with norms over the whole projection")
             key = ("position", s.position)            # layers with the same encoding share one part (and its frequencies)
             if key not in rt.shared_parts:
                 rt.shared_parts[key] = build("position", s.position, rt)
             self.position = rt.shared_parts[key]
-        self.w_qkv = self.w_o = self.q_norm = self.k_norm = self.sink = None
+        self.w_qkv = self.b_qkv = self.w_o = self.q_norm = self.k_norm = self.sink = None
 
     def children(self):
         return [self.position] if self.position is not None else []
 
-    def _n(self, which):
-        return self.spec.prefix + getattr(self.spec.names, which)
+    def _n(self, which, bias=False):
+        n = self.spec.names
+        return self.spec.prefix + getattr(n, which) + (n.bias if bias else "")
 
     def param_specs(self):
         s = self.spec
@@ -388,6 +397,9 @@ class WideNormAttention(Part):
                  ParamSpec(self._n("o"), (s.hidden, self.o_width), "matrix"),
                  ParamSpec(self._n("q_norm"), (self.q_width,), "norm_scale"),
                  ParamSpec(self._n("k_norm"), (self.k_width,), "norm_scale")]
+        if s.qkv_bias:
+            specs += [ParamSpec(self._n("q", True), (self.q_width,), "bias"), ParamSpec(self._n("k", True), (self.k_width,), "bias"),
+                      ParamSpec(self._n("v", True), (self.v_width,), "bias")]
         if s.learned_sink:
             specs.append(ParamSpec(self._n("sink"), (s.num_heads,), "attention_sink", init=(0.0, 1.0)))
         return specs
@@ -402,6 +414,10 @@ class WideNormAttention(Part):
         a, b = self.q_width, self.q_width + self.k_width
         views = {names[0]: self.w_qkv[:a], names[1]: self.w_qkv[a:b], names[2]: self.w_qkv[b:], self._n("o"): self.w_o,
                  self._n("q_norm"): self.q_norm, self._n("k_norm"): self.k_norm}
+        if s.qkv_bias:
+            self.b_qkv = torch.empty(self.qkv_width, dtype=torch.float32, device=dev)
+            views.update({self._n("q", True): self.b_qkv[:a], self._n("k", True): self.b_qkv[a:b],
+                          self._n("v", True): self.b_qkv[b:]})
         if s.learned_sink:
             self.sink = torch.empty(s.num_heads, dtype=torch.float32, device=dev)
             views[self._n("sink")] = self.sink
@@ -410,7 +426,7 @@ class WideNormAttention(Part):
     def kv_layout(self):
         s = self.spec
         return KvLayout(s.num_kv_heads, s.key_dim, s.window, value_dim=s.value_dim if s.value_dim != s.key_dim else None,
-                        chunk=s.chunk)
+                        chunk=s.chunk, keep_first=s.keep_first)
 
     def state_spec(self):
         return None
@@ -438,10 +454,11 @@ class WideNormAttention(Part):
         ops.widenorm_rope_kvwrite(qkv, self.q_norm, self.k_norm, s.eps, pos.inv_freq if pos is not None else None,
                                   pos.spec.rotary_dim if pos is not None else 0, 1.0, ctx.tok_seq, ctx.tok_pos, q, layer.k,
                                   layer.v, table, layer.page, s.num_heads, s.num_kv_heads, s.key_dim, s.value_dim, layer.writes,
-                                  rt.status)
+                                  rt.status, bias=self.b_qkv, neighbour=self.neighbour,
+                                  inv_freq_lo=pos.inv_freq_lo if pos is not None else None)
         o = rt.ws.get("attn_o", (n, self.o_width), rt.dtype)
         scaled_attend(rt, self.kernel_for(n, layer.page), q, o, ctx, layer, s.num_heads, s.num_kv_heads, s.key_dim, s.value_dim,
-                      s.scale, self.sink if s.learned_sink else False, window=s.window, chunk=s.chunk)
+                      s.scale, self.sink if s.learned_sink else False, window=s.window, chunk=s.chunk, keep=s.keep_first)
         y = rt.ws.get("mixer_out", (n, s.hidden), torch.float32)
         linear(rt, o, self.w_o, y)
         return y
@@ -559,7 +576,7 @@ class UnitNormAttention(Part):
                                        pos.spec.rotary_dim if pos is not None else 0, s.eps, s.unit_heads, shared_v,
                                        {None: 0, "first": 1, "blend": 2}[s.value_blend], self.blend, ctx.tok_seq, ctx.tok_pos, q,
                                        layer.k, layer.v, table, layer.page, s.num_heads, s.num_kv_heads, s.key_dim, s.value_dim,
-                                       layer.writes, rt.status)
+                                       layer.writes, rt.status, inv_freq_lo=pos.inv_freq_lo if pos is not None else None)
         o = rt.ws.get("attn_o", (n, self.o_width), rt.dtype)
         scaled_attend(rt, self.kernel_for(n, layer.page), q, o, ctx, layer, s.num_heads, s.num_kv_heads, s.key_dim, s.value_dim,
                       s.scale, self.sink if s.learned_sink else False, window=s.window)

@@ -208,6 +208,53 @@ class OutputNormBlock(Part):
         return pending
 
 
+class ParallelResidualBlock(Part):
+    """x += mixer(h) + ffn(h) with h = norm(x).  Neither sublayer waits for the other: the mixer runs on a second stream
+    beside the feed-forward (in a captured step: a parallel branch of the graph), and the norm that reads x next adds
+    both results, in one launch with a sparse feed-forward's ordered sum of its experts."""
+
+    graph_safe = True
+
+    def __init__(self, spec, rt):
+        self.spec, self.rt = spec, rt
+        self.norm = build("norm", spec.norm, rt)
+        self.mixer = build("mixer", spec.mixer, rt)
+        self.ffn = build("ffn", spec.ffn, rt)
+
+    def children(self):
+        return [p for p in (self.norm, self.mixer, self.ffn) if p is not None]
+
+    def forward(self, x, pending, ctx, layer):
+        rt = self.rt
+        h = rt.ws.get("block_h", tuple(x.shape), rt.dtype)
+        h32 = None
+        if rt.dtype != torch.float32 and getattr(self.ffn, "wants_f32_input", False):
+            h32 = rt.ws.get("block_h32", tuple(x.shape), torch.float32)
+        self.norm.forward(x, plain_delta(self.norm, pending), h, h32=h32)
+        if self.ffn is None:
+            pending = self.mixer.forward(h, ctx, layer)
+        else:
+            side = rt.side_stream
+            if side is not None:
+                main = torch.cuda.current_stream()
+                side.wait_stream(main)
+                with torch.cuda.stream(side):
+                    mixed = plain_delta(None, self.mixer.forward(h, ctx, layer))
+            else:
+                mixed = plain_delta(None, self.mixer.forward(h, ctx, layer))
+            pending = self.ffn.forward(h, ctx, h32=h32)
+            if side is not None:
+                main.wait_stream(side)
+            if not getattr(pending, "take_along", lambda rows: False)(mixed):
+                pending = plain_delta(None, pending).add_(mixed)
+        if "residual_trace" in ctx.aux:
+            # debugging aid (see ScaledDepthMixBlock._trace): the add is done here so that x is the layer's result
+            x.add_(plain_delta(None, pending))
+            ctx.aux["residual_trace"].append(x.clone())
+            return None
+        return pending
+
+
 class DeferredStreamWrite:
     """The write of a sublayer into the copies of the residual stream, on its way to whoever reads them next: the
     next layer's first read, or the model's last norm (which then sees the sum of the copies).  Either does the
@@ -316,4 +363,5 @@ register("block", "prenorm_residual", PreNormResidualBlock)
 register("block", "hyper_connections", HyperConnectionBlock)
 register("block", "sandwich_residual", SandwichBlock)
 register("block", "output_norm_residual", OutputNormBlock)
+register("block", "parallel_residual", ParallelResidualBlock)
 register("block", "prenorm_scaled_depthmix", ScaledDepthMixBlock)

@@ -31,6 +31,17 @@ class DeferredMoeCombine:
                                     rows=rows, write_x=write_x, h32=h32, passing=self.passing,
                                     gamma_y=post[0] if post else None, eps_y=post[1] if post else 0.0)
 
+    def fused_add_layernorm(self, x, gamma, beta, h, eps, rows, write_x, h32):
+        ops.moe_combine_add_rmsnorm(self.expert_out, self.ids, self.inverse, self.gate, self.shared, x, gamma, h, eps,
+                                    rows=rows, write_x=write_x, h32=h32, passing=self.passing, beta=beta)
+
+    def take_along(self, rows) -> bool:
+        """Adds ``rows`` (float32, one per token) to the sum of the experts, where nothing else rides there yet."""
+        if self.shared is not None:
+            return False
+        self.shared, self.gate = rows, None
+        return True
+
 
 # Steps with at least AHEAD_ROWS rows start the shared expert's first product on a second stream before the
 # router, on all SMs but ROUTING_SMS: the router and the permutation are a chain of short launches that leaves
@@ -179,7 +190,8 @@ class MoeSwiGluShared(Part):
     (crates/esp/src/infer/decoder/moe.rs:135-256).  Options of the spec: router outputs without an expert behind
     them (a chosen one returns the block's input times its weight), a correction per output that counts for the
     choice only, a choice limited to the best groups of neighbouring outputs, a bias on the logits, weights that are a
-    softmax over the chosen logits alone, gated units with clamped branches, no shared expert or one without a gate."""
+    softmax over the chosen logits alone, scores that are sigmoids of the logits, a factor on the weights, gated units with
+    clamped branches, no shared expert or one without a gate."""
 
     graph_safe = True
 
@@ -280,7 +292,9 @@ class MoeSwiGluShared(Part):
         n, k, E, Im, H = h.shape[0], s.top_k, s.num_experts, s.expert_intermediate, s.hidden
         R = self.n_outputs                       # router outputs: experts with weights, then those without
         has_shared = s.shared_intermediate is not None
-        choice = (self.correction, s.groups, s.keep_groups) if (self.correction is not None or s.groups > 1) else None
+        choice = None
+        if self.correction is not None or s.groups > 1:
+            choice = (self.correction, s.groups, s.keep_groups, s.group_top)
         ws = rt.ws
         ids = ws.get("moe_ids", (n, k), torch.int32)
         wts = ws.get("moe_w", (n, k), torch.float32)
@@ -332,11 +346,12 @@ class MoeSwiGluShared(Part):
             logits = ws.get("moe_logits", (n, R + 1), torch.float32)
             ops.route_small(router_in, self.w_router, self.w_shared_gate, logits, ids, wts, gate, k, s.norm_topk,
                             offsets, perm_token, perm_weight, inverse, rt.status, probs, distinct=self.expert_reads,
-                            tiles=tiles, choice=choice, n_real=E, bias=self.router_bias, chosen_softmax=s.chosen_softmax)
+                            tiles=tiles, choice=choice, n_real=E, bias=self.router_bias, chosen_softmax=s.chosen_softmax,
+                            sigmoid=s.sigmoid_scores, scale=s.weight_scale)
         else:
             ops.router_topk(router_in, self.w_router, self.w_shared_gate, ids, wts, gate, k, s.norm_topk, rt.status,
                             probs, logits=ws.get("moe_logits", (n, R + 1), torch.float32), choice=choice, bias=self.router_bias,
-                            chosen_softmax=s.chosen_softmax)
+                            chosen_softmax=s.chosen_softmax, sigmoid=s.sigmoid_scores, scale=s.weight_scale)
             ops.moe_permute(ids, wts, E, offsets, perm_token, perm_weight, inverse, rt.status, tiles=tiles,
                             distinct=self.expert_reads, n_ids=R)
         if rt.record_routing:

@@ -1,4 +1,4 @@
-"""RMSNorm fused with the residual add that precedes it."""
+"""RMS norm and layer norm, fused with the residual add that precedes them."""
 from __future__ import annotations
 
 import torch
@@ -72,6 +72,34 @@ class OffsetRmsNorm(RmsNorm):
             self.weight.add_(1.0)
 
 
+class LayerNorm(RmsNorm):
+    """h = (v - mean(v)) / sqrt(mean((v - mean(v))^2) + eps) * weight + bias with v = x + delta, in 32-bit."""
+
+    def __init__(self, spec, rt):
+        super().__init__(spec, rt)
+        self.bias = None
+
+    def param_specs(self):
+        return super().param_specs() + [ParamSpec(self.spec.bias, (self.spec.width,), "norm_bias", init=(0.0, 0.1))]
+
+    def allocate(self, stored, rt):
+        views = super().allocate(stored, rt)
+        self.bias = torch.empty(self.spec.width, dtype=torch.float32, device=rt.device)
+        views[self.spec.bias] = self.bias
+        return views
+
+    def forward(self, x, delta, h, rows=None, write_x=True, h32=None, delta_scale=None):
+        if hasattr(delta, "fused_add_layernorm") and delta_scale is None:
+            # the producer left its last step (an ordered sum) to be done here, in the same launch
+            delta.fused_add_layernorm(x, self.weight, self.bias, h, self.spec.eps, rows, write_x, h32)
+            return h
+        if hasattr(delta, "materialize"):
+            delta = delta.materialize()
+        ops.add_rmsnorm(x, delta, self.weight, h, self.spec.eps, rows=rows, write_x=write_x, h32=h32,
+                        yscale=delta_scale if delta is not None else None, beta=self.bias)
+        return h
+
+
 class DeferredPostNorm:
     """A sublayer's result on its way into the residual stream through a norm of its own: x += norm(y).  The norm that
     reads x next does that add and its own normalisation in one launch (``fused_add_rmsnorm``); anything else gets the
@@ -108,3 +136,4 @@ class DeferredPostNorm:
 register("norm", "rmsnorm", RmsNorm)
 register("norm", "rmsnorm_scalar", ScalarRmsNorm)
 register("norm", "rmsnorm_offset", OffsetRmsNorm)
+register("norm", "layernorm", LayerNorm)

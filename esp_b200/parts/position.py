@@ -108,7 +108,21 @@ class RopeScaled(Part):
             self.inv_freq_lo = torch.from_numpy((f - hi).astype(np.float32)).to(self.rt.device).contiguous()
 
 
+class RopeNeighbourPairs(RopeScaled):
+    """The rotation of neighbouring channels (see ``NeighbourRopeSpec``): the frequencies, slow ones slowed by their
+    wavelength; which channels form a pair is the kernel's business.  No factor on cosines and sines."""
+
+    def exact_frequencies(self):
+        sp = self.spec
+        f = np.power(float(sp.theta), -2.0 * np.arange(sp.rotary_dim // 2, dtype=np.float64) / sp.rotary_dim)
+        if sp.factor is not None:
+            turns = sp.original * f / (2.0 * np.pi)          # of a pair within the original length: original / wavelength
+            s = (turns - sp.low) / (sp.high - sp.low)
+            f = np.where(turns > sp.high, f, np.where(turns < sp.low, f / sp.factor, (1.0 - s) * f / sp.factor + s * f))
+        return f, 1.0
+
+
 register("position", "rope_split_half", RopeSplitHalf)
 register("position", "rope_split_half_scaled", RopeScaled)
-register("position", "rope_neighbour_pairs", RopeScaled)     # the same frequencies; which channels form a pair is the kernel's business
+register("position", "rope_neighbour_pairs", RopeNeighbourPairs)
 register("position", "none", NoPosition)

@@ -1,7 +1,7 @@
 """Mixers with a recurrent state of fixed size per sequence: two forms of the gated outer-product recurrence
 S_t = diag(d_t) S_(t-1) + k_t v_t^T per head.  A head's matrix S is float32 and belongs to the sequence: it sits in
 the cache's per-slot state rows, is zeroed when the slot is opened, and every step continues from what the step before
-left there, whatever run of tokens it brings.  Both run on ``ops.gated_scan``, which makes the gates from the projections' raw outputs."""
+left there, whatever run of tokens it brings.  They run on ``ops.gated_scan``, which makes the gates from the projections' raw outputs."""
 from __future__ import annotations
 
 import numpy as np
@@ -354,7 +354,77 @@ class GatedDiagonalRecurrence(Part):
         return out
 
 
+class FixedDecayAttention(Part):
+    """Linear attention with one fixed decay per head (see ``FixedDecayAttentionSpec``).  One packed product makes q, k, v and
+    the output gate; the recurrence takes the SiLUs of the first three as it stages its rows; the heads' output is normed
+    as one row and multiplied by the sigmoid gate in one kernel; then W_o.  Per slot the state holds S as [heads, value
+    channels, key channels] floats."""
+
+    graph_safe = True
+
+    def __init__(self, spec, rt):
+        self.spec, self.rt = spec, rt
+        s = spec
+        _check_dims(s.kind, s.key_dim)
+        if len(s.decay) != s.num_heads:
+            raise Unsupported(s.kind + ".decay", f"{len(s.decay)} decays for {s.num_heads} heads")
+        self.kw, self.vw = s.num_heads * s.key_dim, s.num_heads * s.value_dim
+        self.at_v, self.at_gate = 2 * self.kw, 2 * self.kw + self.vw
+        self.w_in = self.w_o = self.norm_w = self.decay = self.decay_rest = None
+
+    def _n(self, which):
+        return self.spec.prefix + getattr(self.spec.names, which)
+
+    def param_specs(self):
+        s = self.spec
+        return [ParamSpec(self._n("q"), (self.kw, s.hidden), "matrix"), ParamSpec(self._n("k"), (self.kw, s.hidden), "matrix"),
+                ParamSpec(self._n("v"), (self.vw, s.hidden), "matrix"), ParamSpec(self._n("gate"), (self.vw, s.hidden), "matrix"),
+                ParamSpec(self._n("norm"), (self.vw,), "norm_scale"), ParamSpec(self._n("o"), (s.hidden, self.vw), "matrix")]
+
+    def allocate(self, stored, rt):
+        s, dev = self.spec, rt.device
+        names = [self._n(t) for t in ("q", "k", "v", "gate")]
+        self.w_in = torch.empty((self.at_gate + self.vw, s.hidden), dtype=rt.matrix_dtype([stored[n] for n in names]), device=dev)
+        self.w_o = torch.empty((s.hidden, self.vw), dtype=rt.matrix_dtype([stored[self._n("o")]]), device=dev)
+        self.norm_w = torch.empty(self.vw, dtype=torch.float32, device=dev)
+        views, at = {}, 0
+        for n, size in zip(names, (self.kw, self.kw, self.vw, self.vw)):
+            views[n] = self.w_in[at:at + size]
+            at += size
+        views.update({self._n("o"): self.w_o, self._n("norm"): self.norm_w})
+        return views
+
+    def finalize(self):
+        if self.decay is None and self.w_in is not None:
+            exact = np.asarray(self.spec.decay, dtype=np.float64)
+            top = exact.astype(np.float32)
+            self.decay = torch.from_numpy(top).to(self.rt.device)
+            self.decay_rest = torch.from_numpy((exact - top).astype(np.float32)).to(self.rt.device)
+
+    def kv_layout(self):
+        return None
+
+    def state_spec(self):
+        return StateSpec((self.spec.num_heads * self.spec.value_dim * self.spec.key_dim,), torch.float32)
+
+    def forward(self, h, ctx, layer):
+        s, rt = self.spec, self.rt
+        n = h.shape[0]
+        proj = rt.ws.get("lightning_proj", (n, self.at_gate + self.vw), torch.float32)
+        linear(rt, h, self.w_in, proj)
+        o = rt.ws.get("rec_out", (n, self.vw), torch.float32)
+        ops.gated_scan(ops.SCAN_FIXED_DECAY, proj[:, :self.kw], proj[:, self.kw:self.at_v], self.decay,
+                       proj[:, self.at_v:self.at_gate], None, self.decay_rest, None, layer.state, ctx.seq_start, ctx.seq_slot, o,
+                       ctx.n_seqs, s.num_heads, s.key_dim, s.value_dim)
+        y = rt.ws.get("rec_normed", (n, self.vw), rt.dtype)
+        ops.head_rmsnorm_gate(o, self.norm_w, 0, proj[:, self.at_gate:], y, 1, self.vw, s.eps, gate_sigmoid=True)
+        out = rt.ws.get("mixer_out", (n, s.hidden), torch.float32)
+        linear(rt, y, self.w_o, out)
+        return out
+
+
 register("mixer", "hgrn2", LowerBoundRecurrence)
+register("mixer", "lightning", FixedDecayAttention)
 register("mixer", "mlstm", MatrixMemory)
 register("mixer", "rglru", GatedDiagonalRecurrence)
 register("mixer", "wkv", DecayBonusRecurrence)

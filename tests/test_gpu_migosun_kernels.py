@@ -183,7 +183,7 @@ def test_norm_over_the_whole_projection_then_rotation_of_the_first_channels(H, G
     k_want = plain.rms(qkv[:, H * K:H * K + G * K].double(), eps) * k_w.double()
     if rot:
         # the frequencies as the kernel gets them (32-bit), the angle in 32-bit too: compare with that angle exactly
-        ang = (pos.float()[:, None] * inv_freq[None, :]).double()
+        ang = pos.double()[:, None] * inv_freq.double()[None, :]          # the product is exact, the frequency 32-bit
         def turn(x, heads):
             x = x.view(n, heads, K)
             a, b = x[..., :rot // 2], x[..., rot // 2:rot]

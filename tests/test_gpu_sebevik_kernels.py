@@ -163,7 +163,7 @@ def test_rotation_of_neighbours_then_unit_heads_and_blended_values(H, G, K, V, r
     def turn(t):
         if not rot:
             return t
-        ang = (pos.float()[:, None] * inv_freq[None, :]).double()      # the angle as the kernel takes it: a 32-bit product
+        ang = pos.double()[:, None] * inv_freq.double()[None, :]          # the product is exact, the frequency 32-bit
         c, s = torch.cos(ang)[:, None], torch.sin(ang)[:, None]
         out = t.clone()
         a, b = t[..., 0:rot:2], t[..., 1:rot:2]
