@@ -556,6 +556,29 @@ def satavik_config(width, ff, layers, vocab, chunk):
             "layers": out}
 
 
+# --design galirax: the decoder whose mixer and feed-forward read one norm side by side, with attention over every key,
+# windowed attention that keeps the first tokens in sight, and linear attention with a fixed decay per head, beside the Qwen2
+# MoE decoder of the same width, depth, heads and expert sizes with experts in every layer (the closest model this library
+# has: grouped attention, a router over gated experts).  Four experts a token here, two and a shared one as wide as two
+# there: as many weights at work per token.
+GALIRAX_TOP = 4
+
+
+def galirax_config(width, ff, layers, vocab, window):
+    heads = width // 128
+    att = {"heads": heads, "kv_heads": max(1, heads // 4), "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "rot": {"dims": 128, "base": 1e6}}
+    scaled = dict(att, rot=dict(att["rot"], scaling={"factor": 8.0, "low": 1.0, "high": 4.0, "original": 8192}))
+    kept = dict(att, mask={"size": window, "keep_first": 4})
+    pattern = [{"type": "attention", "mixer": scaled}, {"type": "attention_2", "mixer": kept},
+               {"type": "lightning", "mixer": {"heads": heads, "dim": 128, "vdim": 128,
+                                               "decay": [1 - 2.0 ** -(3 + 6 * h / heads) for h in range(heads)]}},
+               {"type": "attention_2", "mixer": kept}]
+    moe = {"kind": "moe", "router": {"experts": VUMEDRA_EXPERTS, "top": GALIRAX_TOP, "scale": 2.5, "groups": {"count": 4, "keep": 2}},
+           "expert": {"ff": ff // 4}}
+    out = [dict(pattern[i % 4], mixer=dict(pattern[i % 4]["mixer"]), mlp=dict(moe)) for i in range(layers)]
+    return {"architecture": "Galirax", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "logit_softcap": 30.0, "layers": out}
+
+
 def measure_design(torch, raw, prefill_tokens, batches, context, steps, warmup, clocks):
     """Prefill of one prompt and decode steps of a model with random weights: tokens per second, and device time
     by kind of kernel for one eager prefill and one eager decode step (library products count with the kernel
@@ -612,9 +635,9 @@ def bench_design(torch, a, pk):
     sizes = {"w1024": (1024, 2816, 8), "w2048": (2048, 5632, 8), "w4096": (4096, 11008, 8)}
     picked = [s for s in a.design_sizes.split(",") if s]
     vocab, window = 32768, 4096
-    vumedra, migosun, sebevik, satavik = (a.design == d for d in ("vumedra", "migosun", "sebevik", "satavik"))
+    vumedra, migosun, sebevik, satavik, galirax = (a.design == d for d in ("vumedra", "migosun", "sebevik", "satavik", "galirax"))
     beside = ("Qwen2 MoE decoder of equal width, depth, heads, dense and expert sizes" if vumedra or sebevik else
-              "Qwen2 MoE decoder of equal width, depth, heads and expert sizes, experts in every layer" if satavik else
+              "Qwen2 MoE decoder of equal width, depth, heads and expert sizes, experts in every layer" if satavik or galirax else
               "Zusepel decoder of equal width, depth and feed-forward width" if migosun else
               "dense Qwen2 decoder of equal width, depth and feed-forward width")
     result = {"design": a.design, "beside": beside, "dtype": "bf16",
@@ -630,13 +653,13 @@ def bench_design(torch, a, pk):
             mine, other = vumedra_config(width, ff, layers, vocab), sparse_qwen2_config(width, ff, layers, vocab)
         elif sebevik:
             mine, other = sebevik_config(width, ff, layers, vocab, window), sparse_qwen2_config(width, ff, layers, vocab)
-        elif satavik:
-            mine = satavik_config(width, ff, layers, vocab, window)
+        elif satavik or galirax:
+            mine = (satavik_config if satavik else galirax_config)(width, ff, layers, vocab, window)
             other = dict(sparse_qwen2_config(width, ff, layers, vocab), mlp_only_layers=[])
         else:
             mine, other = zusepel_config(width, ff, layers, vocab, window), dense_qwen2_config(width, ff, layers, vocab)
         entry[a.design] = measure_design(torch, mine, a.prefill_tokens, (1, 8), a.context, a.steps, a.warmup, clocks)
-        entry["zusepel" if migosun else "qwen2_moe" if vumedra or sebevik or satavik else "qwen2_dense"] = measure_design(
+        entry["zusepel" if migosun else "qwen2_moe" if vumedra or sebevik or satavik or galirax else "qwen2_dense"] = measure_design(
             torch, other, a.prefill_tokens, (1, 8), a.context, a.steps, a.warmup, clocks)
         result["sizes"][name] = entry
     result["clocks"] = clocks.summary()
@@ -646,10 +669,10 @@ def bench_design(torch, a, pk):
 
 def main() -> int:
     ap = argparse.ArgumentParser()
-    ap.add_argument("--design", default=None, choices=["zusepel", "vumedra", "migosun", "sebevik", "satavik"],
+    ap.add_argument("--design", default=None, choices=["zusepel", "vumedra", "migosun", "sebevik", "satavik", "galirax"],
                     help="instead of the default workload: prefill and decode of this design at a few layer sizes, beside "
                          "the closest other decoder of equal size (the dense Qwen2 for zusepel, the Qwen2 with routed "
-                         "experts for vumedra, sebevik and satavik, zusepel for migosun)")
+                         "experts for vumedra, sebevik, satavik and galirax, zusepel for migosun)")
     ap.add_argument("--design-sizes", default="w1024,w2048", help="with --design: which of w1024, w2048, w4096")
     ap.add_argument("--gpus", type=int, default=1)
     ap.add_argument("--steps", type=int, default=32)

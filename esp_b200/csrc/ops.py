@@ -32,6 +32,8 @@ _SIGNATURES = {
     "esp_gate_prepare": [c_int, P, c_longlong, P, c_longlong, P, P, P, P, P, c_longlong, c_int, P],
     "esp_gated_scan": [c_int, c_int, P, c_longlong, P, c_longlong, P, c_longlong, P, c_longlong, P, P, P, P, c_longlong, P, P, P,
                        c_int, c_int, c_int, c_int, P],
+    "esp_linear_attn_chunks": [P, P, P, c_longlong, P, P, P, P, P, P, P, c_int, P, c_longlong, P, c_int, c_int, c_int, c_int, c_int,
+                               P],
     "esp_head_rmsnorm_gate": [P, P, c_int, P, c_longlong, P, c_int, c_int, c_int, c_int, c_float, c_int, P],
     "esp_latent_kv_store": [P, P, P, c_float, c_int, P, P, P, c_int, c_int, c_int, P, c_int, c_int, c_int, c_int, c_float, P,
                             P],
@@ -970,6 +972,34 @@ def gated_scan(mode, q, k, g, v, gate_bias, lower, bonus, state, seq_start, seq_
         _ptr(lower, torch.float32, "lower"), _ptr(bonus, torch.float32, "bonus"), state.data_ptr(), state.stride(0),
         _ptr(seq_start, torch.int32), _ptr(seq_slot, torch.int32), _ptr(out, torch.float32, "out"), int(n_seqs), heads,
         key_dim, value_dim, _stream()), "gated_scan")
+
+
+LINEAR_CHUNK = 64            # tokens of a chunk of linear_attn_chunks
+
+
+def linear_attn_chunks_fits(key_dim: int, value_dim: int) -> bool:
+    """Sizes of a head that ``linear_attn_chunks`` takes."""
+    return key_dim % 4 == 0 and 0 < key_dim <= 256 and value_dim % 4 == 0 and value_dim > 0
+
+
+def linear_attn_chunks(q, k, v, chunk_seq, chunk_first, chunk_start, seq_start, seq_slot, powers, scratch, state, out, n_seqs,
+                       heads, key_dim, value_dim):
+    """What ``gated_scan(SCAN_FIXED_DECAY, ...)`` computes, for runs of many tokens, in chunks of LINEAR_CHUNK tokens on the
+    tensor cores (products of bfloat16 operands, states and decays 32-bit).  q, k, v: float32 views of rows of one stride,
+    before their SiLU; chunk_seq / chunk_first: the chunks in order of the sequences, chunk_start int32 [n_seqs + 1] their
+    ranges; powers float32 [heads, LINEAR_CHUNK + 1]; scratch float32, whole chunks of heads * value_dim * key_dim: as many
+    chunks as it holds are worked on at once."""
+    per = heads * key_dim * value_dim
+    (pq, ld), (pk, ldk), (pv, ldv) = _rows_ld(q, "q"), _rows_ld(k, "k"), _rows_ld(v, "v")
+    if not linear_attn_chunks_fits(key_dim, value_dim) or ldk != ld or ldv != ld or scratch.numel() < per:
+        raise Backend(f"linear_attn_chunks: head sizes {key_dim} / {value_dim}, strides or scratch not taken")
+    if state.dtype != torch.float32 or state.stride(1) != 1 or state.shape[1] < per or tuple(powers.shape) != (heads, LINEAR_CHUNK + 1):
+        raise Backend("linear_attn_chunks: the state rows are too short or the powers have another shape")
+    _check(_fn("bf16", "esp_linear_attn_chunks")(
+        pq, pk, pv, ld, _ptr(chunk_seq, torch.int32), _ptr(chunk_first, torch.int32), _ptr(chunk_start, torch.int32),
+        _ptr(seq_start, torch.int32), _ptr(seq_slot, torch.int32), _ptr(powers, torch.float32, "powers"),
+        _ptr(scratch, torch.float32, "scratch"), scratch.numel() // per, state.data_ptr(), state.stride(0),
+        _ptr(out, torch.float32, "out"), chunk_seq.shape[0], int(n_seqs), heads, key_dim, value_dim, _stream()), "linear_attn_chunks")
 
 
 def head_rmsnorm_gate(o, weight, weight_head_stride, gate, y, heads, value_dim, eps, gate_sigmoid=False):

@@ -17,6 +17,10 @@ from .linear import SKINNY_ROWS, linear
 # Steps with more rows than this per sequence make the gates in a parallel pass ahead of the recurrence; shorter
 # ones (decoding) let the recurrence make them as it stages its rows.  Both give the same bits.
 GATES_AHEAD_ROWS = 8
+# Steps with more rows than this per sequence run linear attention with a fixed decay in chunks on the tensor cores
+# (bfloat16); the states of up to CHUNK_SCRATCH_FLOATS / (heads x key x value channels) chunks are made at once.
+CHUNKED_ROWS = 16
+CHUNK_SCRATCH_FLOATS = 64 << 20
 
 
 def _check_dims(kind, key_dim):
@@ -357,8 +361,9 @@ class GatedDiagonalRecurrence(Part):
 class FixedDecayAttention(Part):
     """Linear attention with one fixed decay per head (see ``FixedDecayAttentionSpec``).  One packed product makes q, k, v and
     the output gate; the recurrence takes the SiLUs of the first three as it stages its rows; the heads' output is normed
-    as one row and multiplied by the sigmoid gate in one kernel; then W_o.  Per slot the state holds S as [heads, value
-    channels, key channels] floats."""
+    as one row and multiplied by the sigmoid gate in one kernel; then W_o.  In bfloat16, steps of many tokens run the
+    recurrence in chunks on the tensor cores; short ones, and all of the 32-bit engine's, token by token.  Per slot the
+    state holds S as [heads, value channels, key channels] floats."""
 
     graph_safe = True
 
@@ -370,7 +375,7 @@ class FixedDecayAttention(Part):
             raise Unsupported(s.kind + ".decay", f"{len(s.decay)} decays for {s.num_heads} heads")
         self.kw, self.vw = s.num_heads * s.key_dim, s.num_heads * s.value_dim
         self.at_v, self.at_gate = 2 * self.kw, 2 * self.kw + self.vw
-        self.w_in = self.w_o = self.norm_w = self.decay = self.decay_rest = None
+        self.w_in = self.w_o = self.norm_w = self.decay = self.decay_rest = self.powers = None
 
     def _n(self, which):
         return self.spec.prefix + getattr(self.spec.names, which)
@@ -400,6 +405,8 @@ class FixedDecayAttention(Part):
             top = exact.astype(np.float32)
             self.decay = torch.from_numpy(top).to(self.rt.device)
             self.decay_rest = torch.from_numpy((exact - top).astype(np.float32)).to(self.rt.device)
+            powers = exact[:, None] ** np.arange(ops.LINEAR_CHUNK + 1)
+            self.powers = torch.from_numpy(powers.astype(np.float32)).to(self.rt.device)
 
     def kv_layout(self):
         return None
@@ -407,15 +414,43 @@ class FixedDecayAttention(Part):
     def state_spec(self):
         return StateSpec((self.spec.num_heads * self.spec.value_dim * self.spec.key_dim,), torch.float32)
 
+    # -- the chunks of new tokens, for steps of many rows ------------------------------------
+    def step_arrays_key(self):
+        return ("linear_chunks", self.rt.dtype)
+
+    def step_arrays(self, step):
+        if self.rt.dtype != torch.bfloat16 or step.n_tokens <= CHUNKED_ROWS * step.n_seqs:
+            return {}
+        size = ops.LINEAR_CHUNK
+        chunks = [(i, f) for i, t in enumerate(step.news) for f in range(0, t, size)]
+        starts = np.concatenate([[0], np.cumsum([(t + size - 1) // size for t in step.news])])
+        return {"linear.chunks.seq": np.asarray([c[0] for c in chunks], dtype=np.int32),
+                "linear.chunks.first": np.asarray([c[1] for c in chunks], dtype=np.int32),
+                "linear.chunks.start": starts.astype(np.int32)}
+
     def forward(self, h, ctx, layer):
         s, rt = self.spec, self.rt
         n = h.shape[0]
         proj = rt.ws.get("lightning_proj", (n, self.at_gate + self.vw), torch.float32)
         linear(rt, h, self.w_in, proj)
         o = rt.ws.get("rec_out", (n, self.vw), torch.float32)
+        chunk_seq = ctx.arrays.get("linear.chunks.seq")
+        if chunk_seq is not None and ops.linear_attn_chunks_fits(s.key_dim, s.value_dim):
+            per = s.num_heads * s.key_dim * s.value_dim
+            at_once = min(chunk_seq.shape[0], max(1, CHUNK_SCRATCH_FLOATS // per))
+            scratch = rt.ws.get("linear_chunks", (at_once * per,), torch.float32)
+            ops.linear_attn_chunks(proj[:, :self.kw], proj[:, self.kw:self.at_v], proj[:, self.at_v:self.at_gate], chunk_seq,
+                                   ctx.arrays["linear.chunks.first"], ctx.arrays["linear.chunks.start"], ctx.seq_start, ctx.seq_slot,
+                                   self.powers, scratch, layer.state, o, ctx.n_seqs, s.num_heads, s.key_dim, s.value_dim)
+            return self._finish(proj, o)
         ops.gated_scan(ops.SCAN_FIXED_DECAY, proj[:, :self.kw], proj[:, self.kw:self.at_v], self.decay,
                        proj[:, self.at_v:self.at_gate], None, self.decay_rest, None, layer.state, ctx.seq_start, ctx.seq_slot, o,
                        ctx.n_seqs, s.num_heads, s.key_dim, s.value_dim)
+        return self._finish(proj, o)
+
+    def _finish(self, proj, o):
+        s, rt = self.spec, self.rt
+        n = o.shape[0]
         y = rt.ws.get("rec_normed", (n, self.vw), rt.dtype)
         ops.head_rmsnorm_gate(o, self.norm_w, 0, proj[:, self.at_gate:], y, 1, self.vw, s.eps, gate_sigmoid=True)
         out = rt.ws.get("mixer_out", (n, s.hidden), torch.float32)

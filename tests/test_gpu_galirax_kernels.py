@@ -347,3 +347,69 @@ def test_norm_of_all_heads_as_one_row_with_a_sigmoid_gate(rows, width, dtype):
     y = torch.zeros(rows, width, dtype=dtype, device=DEV)
     ops.head_rmsnorm_gate(dev(o), dev(w), 0, dev(gate)[:, :width], y, 1, width, 1e-5, gate_sigmoid=True)
     assert (y.double().cpu() - want).abs().max() < (1e-5 if dtype == torch.float32 else 3e-2)
+
+
+@pytest.mark.parametrize("H, K, V, decay", [(3, 16, 24, [0.2, 0.97, 0.9999]), (2, 44, 100, [0.0, 1.0]), (1, 256, 40, [0.995]),
+                                            (2, 128, 128, [0.9, 0.9995]), (1, 64, 8, [0.5])])
+@pytest.mark.parametrize("cuts", [[300], [64, 1, 63, 65, 107], [17, 283], [2, 3, 128, 167]])
+@pytest.mark.parametrize("at_once", [1, 3, 100])
+def test_chunks_on_the_tensor_cores_over_any_cutting(H, K, V, decay, cuts, at_once):
+    """Three sequences in slots 3, 0 and 2 (the second brings a tenth of the tokens of the others, down to one), every cutting,
+    with room for one chunk's states, three and all of them.  What the state holds is made of values rounded to 8 bits and of
+    keys that are not; the outputs of rounded queries, keys and values."""
+    g = torch.Generator().manual_seed(K + V)
+    shares = [[n, max(1, n // 10), n] for n in cuts]
+    totals = [sum(s[i] for s in shares) for i in range(3)]
+    seqs = [lightning_inputs(t, H, K, V, g) for t in totals]
+    start = torch.randn(3, H, K, V, generator=g, dtype=torch.float64) * 3
+    state, slots = torch.zeros(5, H * V * K + 4, device=DEV), [3, 0, 2]
+    for slot, s0 in zip(slots, start):
+        state[slot, :H * V * K] = dev(s0.transpose(1, 2).reshape(-1).float())
+    powers = dev(torch.from_numpy((np.asarray(decay)[:, None] ** np.arange(ops.LINEAR_CHUNK + 1)).astype(np.float32)))
+    scratch = torch.full((at_once * H * K * V,), float("nan"), device=DEV)
+    outs, at = [[], [], []], [0, 0, 0]
+    for news in shares:
+        starts = [0, news[0], news[0] + news[1], sum(news)]
+        rows = torch.cat([torch.cat([seqs[i][j][at[i]:at[i] + news[i]] for i in range(3)]) for j in range(3)], dim=1)
+        rows = dev(torch.cat([rows, torch.full((starts[-1], 4), 7.0)], dim=1))
+        chunks = [(i, f) for i, t in enumerate(news) for f in range(0, t, ops.LINEAR_CHUNK)]
+        ranges = np.concatenate([[0], np.cumsum([-(-t // ops.LINEAR_CHUNK) for t in news])])
+        o = torch.full((starts[-1], H * V), float("nan"), device=DEV)
+        ops.linear_attn_chunks(rows[:, :H * K], rows[:, H * K:2 * H * K], rows[:, 2 * H * K:2 * H * K + H * V], i32([c[0] for c in chunks]),
+                               i32([c[1] for c in chunks]), i32(ranges), i32(starts), i32(slots), powers, scratch, state, o, 3, H, K, V)
+        for i in range(3):
+            outs[i].append(o[starts[i]:starts[i + 1]].cpu())
+            at[i] += news[i]
+    rounded = lambda t: t.to(torch.bfloat16).double()
+    for i, slot in enumerate(slots):
+        q, k, v = (plain.silu(t.double()).view(totals[i], H, -1) for t in seqs[i])
+        d = torch.tensor(decay, dtype=torch.float64)
+        _, S = plain.decayed_sums(q, k, rounded(v), d, start[i])
+        end = state[slot, :H * V * K].cpu().double().view(H, V, K).transpose(1, 2)
+        for h in range(H):
+            assert (end[h] - S[h]).abs().max() < 3e-5 * S[h].abs().max(), h
+        want, _ = plain.decayed_sums(rounded(q), k, rounded(v), d, start[i])
+        got = torch.cat(outs[i]).double().view(totals[i], H, V)
+        for h in range(H):
+            assert (got[:, h] - want[:, h]).abs().max() < 6e-3 * want[:, h].abs().max(), h
+    assert float(state[1].abs().max()) == 0 and float(state[:, H * V * K:].abs().max()) == 0
+
+
+def test_a_key_far_back_is_read_through_the_chunks():
+    """One token among 1,500 has a key that the last query alone points at: it is read through twenty-three chunks' states."""
+    H, K, V, T, decay = 1, 64, 64, 1500, [0.9995]
+    g = torch.Generator().manual_seed(4)
+    q, k, v = (torch.randn(T, n, generator=g) * 0.2 for n in (K, K, V))
+    k[3], q[-1] = torch.where(torch.rand(K, generator=g) < 0.5, 8.0, -30.0), 0.0
+    q[-1] = torch.where(k[3] > 0, 8.0, -30.0)
+    v[3] = 10 * torch.rand(V, generator=g)
+    rows = dev(torch.cat([q, k, v], dim=1))
+    firsts = list(range(0, T, ops.LINEAR_CHUNK))
+    powers = dev(torch.from_numpy((np.asarray(decay)[:, None] ** np.arange(ops.LINEAR_CHUNK + 1)).astype(np.float32)))
+    state, o = torch.zeros(1, K * V, device=DEV), torch.zeros(T, V, device=DEV)
+    ops.linear_attn_chunks(rows[:, :K], rows[:, K:2 * K], rows[:, 2 * K:], i32([0] * len(firsts)), i32(firsts), i32([0, len(firsts)]),
+                           i32([0, T]), i32([0]), powers, torch.zeros(len(firsts) * K * V, device=DEV), state, o, 1, H, K, V)
+    want, _ = lightning_want(q, k, v, H, decay, None)
+    alone, _ = lightning_want(q[-1:], k[3:4], v[3:4], H, [1.0], None)
+    assert (want[-1] - alone[0] * decay[0] ** (T - 4)).abs().max() < 0.2 * want[-1].abs().max()      # the probe stands out
+    assert (o[-1].double().cpu() - want[-1]).abs().max() < 6e-3 * want[-1].abs().max()
