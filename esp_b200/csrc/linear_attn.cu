@@ -1,4 +1,5 @@
-// Linear attention with one fixed decay per head over runs of many tokens, in chunks on the tensor cores.
+// Linear attention with one fixed decay per head (bfloat16 engine): runs of many tokens in chunks on the tensor cores, runs of
+// few tokens (decoding) token by token with the state in registers.
 //
 //     S_t = d S_(t-1) + k_t v_t^T,   o_t = S_t^T q_t      per head; q, k, v = SiLU of the projections (float rows)
 //
@@ -72,22 +73,33 @@ __device__ __forceinline__ Chunk chunk_at(const ChunkList& l, int c) {
     return Chunk{l.seq_start[s] + first, min(C, l.seq_start[s + 1] - l.seq_start[s] - first)};
 }
 
-// rows of a chunk, ``width`` channels from column ``col`` on, SiLU taken, to shared memory [C][ld] as bfloat16 (rows past
-// the chunk and channels past ``width`` up to ``padded``: zeros).  scale (may be null): a factor per row; lo (may be
-// null): what rounding left out, as a second tile.
-__device__ __forceinline__ void stage(const float* src, long long stride, int row0, int count, int width, int padded, bf16* hi,
-                                      bf16* lo, int ld, const float* scale) {
-    const int pieces = padded / 4;
-    for (int i = threadIdx.x; i < C * pieces; i += THREADS) {
-        const int r = i / pieces, c = (i - r * pieces) * 4;
-        float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
-        if (r < count && c < width) v = silu4(*reinterpret_cast<const float4*>(src + (size_t)(row0 + r) * stride + c));
-        if (scale) {
-            const float f = scale[r];
-            v.x *= f, v.y *= f, v.z *= f, v.w *= f;
+// 64 rows of ``width`` channels, ``stride`` numbers apart, to shared memory [64][LD] as bfloat16 (rows from ``count`` on and
+// channels past ``width`` up to W: zeros).  ACT: their SiLU.  scale (may be null): a factor per row; lo (may be null): what
+// rounding left out, as a second tile.  A thread's loads go out several at a time.
+template <int W, int LD, bool ACT>
+__device__ __forceinline__ void stage(const float* src, long long stride, int count, int width, bf16* hi, bf16* lo, const float* scale) {
+    constexpr int PIECES = W / 4, PER = 64 * PIECES / THREADS, BATCH = PER < 8 ? PER : 8;
+    static_assert(64 * PIECES % THREADS == 0 && PER % BATCH == 0, "every thread stages the same number of pieces");
+#pragma unroll
+    for (int j0 = 0; j0 < PER; j0 += BATCH) {
+        float4 v[BATCH];
+#pragma unroll
+        for (int j = 0; j < BATCH; j++) {
+            const int i = threadIdx.x + (j0 + j) * THREADS, r = i / PIECES, c = (i % PIECES) * 4;
+            v[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+            if (r < count && c < width) v[j] = *reinterpret_cast<const float4*>(src + (size_t)r * stride + c);
         }
-        Vec4<bf16>::store(hi + r * ld + c, v.x, v.y, v.z, v.w);
-        if (lo) Vec4<bf16>::store(lo + r * ld + c, low_part(v.x), low_part(v.y), low_part(v.z), low_part(v.w));
+#pragma unroll
+        for (int j = 0; j < BATCH; j++) {
+            const int i = threadIdx.x + (j0 + j) * THREADS, r = i / PIECES, c = (i % PIECES) * 4;
+            float4 s = ACT ? silu4(v[j]) : v[j];          // the SiLU of zero is zero
+            if (scale) {
+                const float f = scale[r];
+                s.x *= f, s.y *= f, s.z *= f, s.w *= f;
+            }
+            Vec4<bf16>::store(hi + r * LD + c, s.x, s.y, s.z, s.w);
+            if (lo) Vec4<bf16>::store(lo + r * LD + c, low_part(s.x), low_part(s.y), low_part(s.z), low_part(s.w));
+        }
     }
 }
 
@@ -106,8 +118,8 @@ linear_chunk_updates_kernel(const float* __restrict__ k, const float* __restrict
     const Chunk ch = chunk_at(list, chunk0 + blockIdx.x);
     if (threadIdx.x < C) fade[threadIdx.x] = threadIdx.x < ch.count ? powers[h * (C + 1) + ch.count - 1 - threadIdx.x] : 0.f;
     __syncthreads();
-    stage(k + (size_t)h * K, ld, ch.row0, ch.count, K, KP, k_hi, k_lo, LDK, fade);
-    stage(v + (size_t)h * V + v0, ld, ch.row0, ch.count, min(VT, V - v0), VT, v_s, nullptr, LDV, nullptr);
+    stage<KP, LDK, true>(k + (size_t)ch.row0 * ld + h * K, ld, ch.count, K, k_hi, k_lo, fade);
+    stage<VT, LDV, true>(v + (size_t)ch.row0 * ld + h * V + v0, ld, ch.count, V - v0, v_s, nullptr, nullptr);
     __syncthreads();
     const int m0 = (warp & 3) * 16, n0 = (warp >> 2) * (KP / 2);
     float acc[NB][4];
@@ -195,8 +207,8 @@ linear_chunk_outputs_kernel(const float* __restrict__ q, const float* __restrict
     const int g = lane >> 2, tg = lane & 3;
     const Chunk ch = chunk_at(list, chunk0 + blockIdx.x);
     if (threadIdx.x <= C) pw[threadIdx.x] = powers[h * (C + 1) + threadIdx.x];
-    stage(q + (size_t)h * K, ld, ch.row0, ch.count, K, KP, q_s, nullptr, LDK, nullptr);
-    stage(k + (size_t)h * K, ld, ch.row0, ch.count, K, KP, s_hi, nullptr, LDK, nullptr);
+    stage<KP, LDK, true>(q + (size_t)ch.row0 * ld + h * K, ld, ch.count, K, q_s, nullptr, nullptr);
+    stage<KP, LDK, true>(k + (size_t)ch.row0 * ld + h * K, ld, ch.count, K, s_hi, nullptr, nullptr);
     __syncthreads();
     const int m0 = (warp & 3) * 16, n0 = (warp >> 2) * 32;   // a warp's share of a 64 x 64 tile: 16 tokens x 32 columns
     const int ta = m0 + g, tb = ta + 8;                      // the lane's two tokens
@@ -230,15 +242,8 @@ linear_chunk_outputs_kernel(const float* __restrict__ q, const float* __restrict
     const float* S = scratch + ((size_t)blockIdx.x * H + h) * V * K;
     for (int v0 = 0; v0 < V; v0 += VT) {
         __syncthreads();                            // the keys (or the tile before) have been read, the scores are written
-        constexpr int PIECES = KP / 4;
-        for (int i = threadIdx.x; i < VT * PIECES; i += THREADS) {
-            const int r = i / PIECES, c = (i - r * PIECES) * 4;
-            float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
-            if (v0 + r < V && c < K) s = *reinterpret_cast<const float4*>(S + (size_t)(v0 + r) * K + c);
-            Vec4<bf16>::store(s_hi + r * LDK + c, s.x, s.y, s.z, s.w);
-            Vec4<bf16>::store(s_lo + r * LDK + c, low_part(s.x), low_part(s.y), low_part(s.z), low_part(s.w));
-        }
-        stage(v + (size_t)h * V + v0, ld, ch.row0, ch.count, min(VT, V - v0), VT, v_s, nullptr, LDV, nullptr);
+        stage<KP, LDK, false>(S + (size_t)v0 * K, K, V - v0, K, s_hi, s_lo, nullptr);
+        stage<VT, LDV, true>(v + (size_t)ch.row0 * ld + h * V + v0, ld, ch.count, V - v0, v_s, nullptr, nullptr);
         __syncthreads();
         clear();
 #pragma unroll
@@ -281,6 +286,66 @@ linear_chunk_outputs_kernel(const float* __restrict__ q, const float* __restrict
             if (tb < ch.count) *reinterpret_cast<float2*>(o + (size_t)tb * H * V) = make_float2(acc[b][2], acc[b][3]);
         }
     }
+}
+
+// ---- runs of few tokens: grid (sequences, heads, value tiles).  A warp owns STEP_ROWS value channels of a head, a lane four
+// key channels of each (KL times); the state stays in registers over the run.  It was written by an earlier step, so its loads
+// do not wait for the kernel before this one.
+constexpr int STEP_ROWS = 4, STEP_WARPS = 4;
+template <int KL>
+__global__ void __launch_bounds__(32 * STEP_WARPS)
+linear_steps_kernel(const float* __restrict__ q, const float* __restrict__ k, const float* __restrict__ v, long long ld,
+                    const float* __restrict__ decay, const float* __restrict__ rest, float* __restrict__ state,
+                    long long state_stride, const int* __restrict__ seq_start, const int* __restrict__ seq_slot,
+                    float* __restrict__ out, int K, int V) {
+    pdl_trigger();
+    const int b = blockIdx.x, h = blockIdx.y, H = gridDim.y, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    const int v0 = (blockIdx.z * STEP_WARPS + warp) * STEP_ROWS;
+    const int row0 = seq_start[b], row1 = seq_start[b + 1];
+    const float d = decay[h], d_rest = rest[h];
+    float* own = state + (size_t)seq_slot[b] * state_stride + (size_t)h * V * K + (size_t)v0 * K + lane * 4;
+    const float4 none = make_float4(0.f, 0.f, 0.f, 0.f);
+    float4 S[STEP_ROWS][KL];
+#pragma unroll
+    for (int r = 0; r < STEP_ROWS; r++)
+#pragma unroll
+        for (int l = 0; l < KL; l++)
+            S[r][l] = v0 + r < V && lane * 4 + l * 128 < K ? *reinterpret_cast<const float4*>(own + r * K + l * 128) : none;
+    pdl_wait();
+    const float* q_now = behind_wait(q);
+    const float* k_now = behind_wait(k);
+    const float* v_now = behind_wait(v);
+    for (int t = row0; t < row1; t++) {
+        float4 qv[KL], kv[KL];
+#pragma unroll
+        for (int l = 0; l < KL; l++) {
+            const int c = lane * 4 + l * 128;
+            qv[l] = c < K ? silu4(*reinterpret_cast<const float4*>(q_now + t * ld + h * K + c)) : none;
+            kv[l] = c < K ? silu4(*reinterpret_cast<const float4*>(k_now + t * ld + h * K + c)) : none;
+        }
+        float o[STEP_ROWS];
+#pragma unroll
+        for (int r = 0; r < STEP_ROWS; r++) {
+            const float val = v0 + r < V ? silu(v_now[t * ld + h * V + v0 + r]) : 0.f;
+            o[r] = 0.f;
+#pragma unroll
+            for (int l = 0; l < KL; l++) {
+                float4& s = S[r][l];
+                s.x = fmaf(d, s.x, fmaf(d_rest, s.x, kv[l].x * val)), s.y = fmaf(d, s.y, fmaf(d_rest, s.y, kv[l].y * val));
+                s.z = fmaf(d, s.z, fmaf(d_rest, s.z, kv[l].z * val)), s.w = fmaf(d, s.w, fmaf(d_rest, s.w, kv[l].w * val));
+                o[r] = fmaf(s.w, qv[l].w, fmaf(s.z, qv[l].z, fmaf(s.y, qv[l].y, fmaf(s.x, qv[l].x, o[r]))));
+            }
+        }
+#pragma unroll
+        for (int r = 0; r < STEP_ROWS; r++) o[r] = warp_sum(o[r]);
+        if (lane < STEP_ROWS && v0 + lane < V) out[(size_t)t * H * V + h * V + v0 + lane] = lane == 0 ? o[0] : lane == 1 ? o[1] : lane == 2 ? o[2] : o[3];
+    }
+    static_assert(STEP_ROWS == 4, "a lane each writes the outputs");
+#pragma unroll
+    for (int r = 0; r < STEP_ROWS; r++)
+#pragma unroll
+        for (int l = 0; l < KL; l++)
+            if (v0 + r < V && lane * 4 + l * 128 < K) *reinterpret_cast<float4*>(own + r * K + l * 128) = S[r][l];
 }
 
 template <int KP>
@@ -333,4 +398,22 @@ ESP_API int esp_linear_attn_chunks(const float* q, const float* k, const float* 
     if (K <= 128) ESP_CHUNKS(128);
     ESP_CHUNKS(256);
 #undef ESP_CHUNKS
+}
+
+// The same for runs of few tokens.  decay, rest [H]: the decay and what 32-bit leaves out of it.  Sizes as above.
+ESP_API int esp_linear_attn_steps(const float* q, const float* k, const float* v, long long ld, const float* decay, const float* rest,
+                                  float* state, long long state_stride, const int* seq_start, const int* seq_slot, float* out,
+                                  int n_seqs, int H, int K, int V, cudaStream_t stream) {
+    if (n_seqs <= 0) return 0;
+    const size_t ptrs = (size_t)q | (size_t)k | (size_t)v | (size_t)state;
+    if (K <= 0 || V <= 0 || K > 256 || K % 4 || V % 4 || ld % 4 || state_stride % 4 || (ptrs & 15) || H <= 0 || H > 65535)
+        return (int)cudaErrorInvalidValue;
+    const dim3 grid(n_seqs, H, (V + STEP_ROWS * STEP_WARPS - 1) / (STEP_ROWS * STEP_WARPS));
+    if (K <= 128)
+        esp_launch_pdl(ESP_PDL_SMALL, linear_steps_kernel<1>, grid, dim3(32 * STEP_WARPS), 0, stream, q, k, v, ld, decay, rest, state,
+                       state_stride, seq_start, seq_slot, out, K, V);
+    else
+        esp_launch_pdl(ESP_PDL_SMALL, linear_steps_kernel<2>, grid, dim3(32 * STEP_WARPS), 0, stream, q, k, v, ld, decay, rest, state,
+                       state_stride, seq_start, seq_slot, out, K, V);
+    return esp_launch_status();
 }

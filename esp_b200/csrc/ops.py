@@ -34,6 +34,7 @@ _SIGNATURES = {
                        c_int, c_int, c_int, c_int, P],
     "esp_linear_attn_chunks": [P, P, P, c_longlong, P, P, P, P, P, P, P, c_int, P, c_longlong, P, c_int, c_int, c_int, c_int, c_int,
                                P],
+    "esp_linear_attn_steps": [P, P, P, c_longlong, P, P, P, c_longlong, P, P, P, c_int, c_int, c_int, c_int, P],
     "esp_head_rmsnorm_gate": [P, P, c_int, P, c_longlong, P, c_int, c_int, c_int, c_int, c_float, c_int, P],
     "esp_latent_kv_store": [P, P, P, c_float, c_int, P, P, P, c_int, c_int, c_int, P, c_int, c_int, c_int, c_int, c_float, P,
                             P],
@@ -978,7 +979,7 @@ LINEAR_CHUNK = 64            # tokens of a chunk of linear_attn_chunks
 
 
 def linear_attn_chunks_fits(key_dim: int, value_dim: int) -> bool:
-    """Sizes of a head that ``linear_attn_chunks`` takes."""
+    """Sizes of a head that ``linear_attn_chunks`` and ``linear_attn_steps`` take."""
     return key_dim % 4 == 0 and 0 < key_dim <= 256 and value_dim % 4 == 0 and value_dim > 0
 
 
@@ -1000,6 +1001,20 @@ def linear_attn_chunks(q, k, v, chunk_seq, chunk_first, chunk_start, seq_start, 
         _ptr(seq_start, torch.int32), _ptr(seq_slot, torch.int32), _ptr(powers, torch.float32, "powers"),
         _ptr(scratch, torch.float32, "scratch"), scratch.numel() // per, state.data_ptr(), state.stride(0),
         _ptr(out, torch.float32, "out"), chunk_seq.shape[0], int(n_seqs), heads, key_dim, value_dim, _stream()), "linear_attn_chunks")
+
+
+def linear_attn_steps(q, k, v, decay, rest, state, seq_start, seq_slot, out, n_seqs, heads, key_dim, value_dim):
+    """What ``gated_scan(SCAN_FIXED_DECAY, ...)`` computes, for runs of few tokens: the state in registers, four key channels a
+    lane.  q, k, v as for ``linear_attn_chunks``; decay, rest: float32 [heads]."""
+    (pq, ld), (pk, ldk), (pv, ldv) = _rows_ld(q, "q"), _rows_ld(k, "k"), _rows_ld(v, "v")
+    if not linear_attn_chunks_fits(key_dim, value_dim) or ldk != ld or ldv != ld or decay.numel() != heads or rest.numel() != heads:
+        raise Backend(f"linear_attn_steps: head sizes {key_dim} / {value_dim} or strides not taken")
+    if state.dtype != torch.float32 or state.stride(1) != 1 or state.shape[1] < heads * key_dim * value_dim:
+        raise Backend("linear_attn_steps: the state rows are too short or not float32")
+    _check(_fn("bf16", "esp_linear_attn_steps")(
+        pq, pk, pv, ld, _ptr(decay, torch.float32, "decay"), _ptr(rest, torch.float32, "rest"), state.data_ptr(), state.stride(0),
+        _ptr(seq_start, torch.int32), _ptr(seq_slot, torch.int32), _ptr(out, torch.float32, "out"), int(n_seqs), heads, key_dim,
+        value_dim, _stream()), "linear_attn_steps")
 
 
 def head_rmsnorm_gate(o, weight, weight_head_stride, gate, y, heads, value_dim, eps, gate_sigmoid=False):

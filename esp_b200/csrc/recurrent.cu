@@ -787,7 +787,9 @@ ESP_API int esp_head_rmsnorm_gate(const float* o, const float* w, int w_head_str
     const long long warps = (long long)n_rows * H;
     const size_t ptrs = (size_t)o | (size_t)w | (size_t)gate | (size_t)y;
     if (V > 256 && V % 4 == 0 && V <= 16384 && w_head_stride % 4 == 0 && ldgate % 4 == 0 && (ptrs & 15) == 0) {
-        const int threads = V <= 4096 ? (V / 4 + 31) / 32 * 32 : 1024;
+        // one piece a thread while a block can hold them; many rows rounded to bfloat16: up to four, more rows in flight per SM
+        const int per = V > 4096 || (y_is_bf16 && n_rows >= 256) ? 4 : 1;
+        const int threads = ((V / 4 + per - 1) / per + 31) / 32 * 32;
         if (y_is_bf16)
             esp_launch_pdl(ESP_PDL_SMALL, row_rmsnorm_gate_kernel<bf16>, dim3((unsigned)warps), dim3(threads), 0, stream, o, w,
                            w_head_stride, gate, ldgate, (bf16*)y, H, V, eps, gate_sigmoid);

@@ -353,14 +353,14 @@ __global__ void widenorm_rope_kvwrite_kernel(const float* __restrict__ qkv, cons
     }
 }
 
-// The same for head sizes and value sizes (and, where the halves of a rotation are partners, half a rotation) of whole
-// pieces of four channels, and aligned buffers.  The
+// The same, halves of a rotation being partners, for head sizes, value sizes and half a rotation of whole pieces of four
+// channels, and aligned buffers.  The
 // row's query and key part is read once, in 16-byte loads, into shared memory (the sums of squares are taken on the
 // way, both reduced in one exchange).  A thread then makes four
 // neighbouring channels and, where they are rotated, their four partners, and stores each as one piece.  Per element the
 // arithmetic is that of the kernel above; only the order in which the squares are added differs.
 // Dynamic shared memory: (nh * hd + nkv * hd + rot) floats.
-template <typename T, bool NEIGHBOUR>
+template <typename T>
 __global__ void __launch_bounds__(256)
 widenorm_rope_kvwrite_vec_kernel(const float* __restrict__ qkv, const float* __restrict__ bias, const float* __restrict__ q_w,
                                  const float* __restrict__ k_w, float eps, const float* __restrict__ inv_freq,
@@ -417,7 +417,7 @@ widenorm_rope_kvwrite_vec_kernel(const float* __restrict__ qkv, const float* __r
         const bool is_q = e < qw;
         const int local = is_q ? e : e - qw;
         const int head = local / hd, c = local - head * hd;
-        if (!NEIGHBOUR && c >= half && c < rot) continue;   // written with the first halves of their pairs
+        if (c >= half && c < rot) continue;               // written with the first halves of their pairs
         const float* w = is_q ? q_w : k_w;
         const float inv = is_q ? inv_q : inv_k;
         T* dst;
@@ -430,19 +430,7 @@ widenorm_rope_kvwrite_vec_kernel(const float* __restrict__ qkv, const float* __r
             const float4 w4 = *reinterpret_cast<const float4*>(w + local);
             a[0] = a[0] * inv * w4.x, a[1] = a[1] * inv * w4.y, a[2] = a[2] * inv * w4.z, a[3] = a[3] * inv * w4.w;
         }
-        if (NEIGHBOUR) {
-            if (c < rot) {
-                const float cs = rot_cs[c >> 1], sn = rot_cs[half + (c >> 1)], u = a[0];
-                a[0] = u * cs - a[1] * sn;
-                a[1] = a[1] * cs + u * sn;
-            }
-            if (c + 2 < rot) {
-                const float cs = rot_cs[(c >> 1) + 1], sn = rot_cs[half + (c >> 1) + 1], u = a[2];
-                a[2] = u * cs - a[3] * sn;
-                a[3] = a[3] * cs + u * sn;
-            }
-            Vec4<T>::store(dst + c, a[0], a[1], a[2], a[3]);
-        } else if (c < half) {
+        if (c < half) {
             const float4 b4 = *reinterpret_cast<const float4*>(row + e + half);
             float b[4] = {b4.x, b4.y, b4.z, b4.w};
             if (w) {
@@ -472,6 +460,119 @@ widenorm_rope_kvwrite_vec_kernel(const float* __restrict__ qkv, const float* __r
     }
 }
 
+// Neighbour pairs lie in one piece of four channels, so a row needs no exchange but its norms' sums: a thread keeps up to
+// NP pieces of the row (queries, keys and values alike) in registers, all loads in flight at once.  Head and value sizes of
+// whole pieces, aligned buffers, rows of up to 4096 * NP channels.  q_w and k_w null: no norms.  Positions and page tables
+// were written before the step's first kernel: with few rows what hangs on them precedes the wait, with many the row's loads
+// come first and the angles are made while they are on their way.  Dynamic shared memory: rot floats.
+constexpr int NEIGHBOUR_PIECES = 4;
+template <typename T, int NP>
+__global__ void __launch_bounds__(1024)
+neighbour_rope_row_kernel(const float* __restrict__ qkv, const float* __restrict__ bias, const float* __restrict__ q_w,
+                          const float* __restrict__ k_w, float eps, const float* __restrict__ inv_freq,
+                          const float* __restrict__ inv_freq_lo, int rot, float v_scale, const int* __restrict__ tok_seq,
+                          const int* __restrict__ tok_pos, T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache,
+                          const int* __restrict__ block_table, int table_stride, int n_pages, int page, int nh, int nkv, int hd,
+                          int vd, int write_kv, int* __restrict__ status) {
+    pdl_trigger();
+    extern __shared__ __align__(16) float angle_cs[];     // [rot / 2] cosines, then [rot / 2] sines of this row's angles
+    __shared__ float part[2][32];
+    const int n = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nwarp = blockDim.x >> 5;
+    const int qw = nh * hd, kw = nkv * hd, all = qw + kw + nkv * vd, half = rot / 2;
+    float4 x[NP];
+    auto load_row = [&] {
+        pdl_wait();
+        const float* src = behind_wait(qkv) + (size_t)n * all;
+#pragma unroll
+        for (int i = 0; i < NP; i++) {
+            const int e = 4 * (tid + i * blockDim.x);
+            x[i] = e < all ? *reinterpret_cast<const float4*>(src + e) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+    };
+    const bool row_first = gridDim.x > 64;
+    if (row_first) load_row();
+    const int pos = tok_pos[n], seq = tok_seq[n];
+    for (int c = tid; c < half; c += blockDim.x)
+        angle_sincos((float)pos, inv_freq[c], inv_freq_lo ? inv_freq_lo[c] : 0.f, angle_cs[half + c], angle_cs[c]);
+    int page_id = -1;
+    if (write_kv) {
+        page_id = block_table[(size_t)seq * table_stride + pos / page];
+        if (page_id < 0 || page_id >= n_pages) {
+            if (tid == 0) atomicOr(status, ESP_STATUS_BAD_INDEX);
+            page_id = -1;
+        }
+    }
+    const int in_page = pos % page;
+    if (!row_first) load_row();
+    float ssq = 0.f, ssk = 0.f;
+#pragma unroll
+    for (int i = 0; i < NP; i++) {
+        const int e = 4 * (tid + i * blockDim.x);
+        if (e >= all) continue;
+        if (bias) {
+            const float4 b = *reinterpret_cast<const float4*>(bias + e);
+            x[i].x += b.x, x[i].y += b.y, x[i].z += b.z, x[i].w += b.w;
+        }
+        const float s4 = fmaf(x[i].w, x[i].w, fmaf(x[i].z, x[i].z, fmaf(x[i].y, x[i].y, x[i].x * x[i].x)));
+        if (e < qw) ssq += s4;
+        else if (e < qw + kw) ssk += s4;
+    }
+    float inv_q = 1.f, inv_k = 1.f;
+    if (q_w || k_w) {
+        ssq = warp_sum(ssq), ssk = warp_sum(ssk);
+        if (lane == 0) part[0][warp] = ssq, part[1][warp] = ssk;
+    }
+    __syncthreads();                                      // the angles and the sums are there
+    if (q_w || k_w) {
+        float tq = 0.f, tk = 0.f;
+        for (int i = 0; i < nwarp; i++) tq += part[0][i], tk += part[1][i];
+        if (q_w) inv_q = 1.0f / sqrtf(tq / (float)qw + eps);
+        if (k_w) inv_k = 1.0f / sqrtf(tk / (float)kw + eps);
+    }
+#pragma unroll
+    for (int i = 0; i < NP; i++) {
+        const int e = 4 * (tid + i * blockDim.x);
+        if (e >= all) continue;
+        float a[4] = {x[i].x, x[i].y, x[i].z, x[i].w};
+        if (e >= qw + kw) {
+            if (page_id < 0) continue;
+            const int local = e - qw - kw, head = local / vd, c = local - head * vd;
+            Vec4<T>::store(v_cache + (((size_t)page_id * nkv + head) * page + in_page) * vd + c, a[0] * v_scale, a[1] * v_scale,
+                           a[2] * v_scale, a[3] * v_scale);
+            continue;
+        }
+        const bool is_q = e < qw;
+        const int local = is_q ? e : e - qw, head = local / hd, c = local - head * hd;
+        const float* w = is_q ? q_w : k_w;
+        if (w) {
+            const float inv = is_q ? inv_q : inv_k;
+            const float4 w4 = *reinterpret_cast<const float4*>(w + local);
+            a[0] = a[0] * inv * w4.x, a[1] = a[1] * inv * w4.y, a[2] = a[2] * inv * w4.z, a[3] = a[3] * inv * w4.w;
+        }
+#pragma unroll
+        for (int j = 0; j < 4; j += 2)
+            if (c + j < rot) {
+                const float cs = angle_cs[(c + j) >> 1], sn = angle_cs[half + ((c + j) >> 1)], u = a[j];
+                a[j] = u * cs - a[j + 1] * sn;
+                a[j + 1] = a[j + 1] * cs + u * sn;
+            }
+        T* dst;
+        if (is_q) dst = q_out + (size_t)n * qw + local;
+        else if (page_id >= 0) dst = k_cache + (((size_t)page_id * nkv + head) * page + in_page) * hd + c;
+        else continue;
+        Vec4<T>::store(dst, a[0], a[1], a[2], a[3]);
+    }
+}
+
+// Threads of a row's block: about two pieces each (the same for every step, so that a row's sums have one order); 0 where
+// the kernel does not take the sizes.
+static int neighbour_row_threads(int nh, int nkv, int hd, int vd, size_t ptrs) {
+    const int pieces = ((nh + nkv) * hd + nkv * vd) / 4;
+    if (hd % 4 || vd % 4 || (ptrs & 15) || pieces > 1024 * NEIGHBOUR_PIECES) return 0;
+    const int two = (pieces + 1) / 2;
+    return two >= 1024 ? 1024 : (two + 31) / 32 * 32;
+}
+
 // ``neighbour``: channel 2i of a head is rotated with channel 2i + 1 instead of channel i with channel i + rot/2.
 ESP_API int esp_widenorm_rope_kvwrite(const float* qkv, const float* bias, const float* q_w, const float* k_w, float eps,
                                       const float* inv_freq, const float* inv_freq_lo, int rot, int neighbour, float v_scale,
@@ -485,17 +586,22 @@ ESP_API int esp_widenorm_rope_kvwrite(const float* qkv, const float* bias, const
     // which form runs depends on the sizes and the buffers' alignment alone, never on the rows of a step
     const size_t row_bytes = (size_t)((nh + nkv) * hd + rot) * sizeof(float);
     const size_t ptrs = (size_t)qkv | (size_t)bias | (size_t)q_w | (size_t)k_w | (size_t)q_out | (size_t)k_cache | (size_t)v_cache;
-    const bool vec = hd % 4 == 0 && vd % 4 == 0 && (neighbour || rot % 8 == 0) && (ptrs & 15) == 0 && row_bytes <= 40 * 1024;
-#define ESP_WIDENORM(KERNEL, T, NB)                                                                                          \
-    esp_launch_pdl(ESP_PDL_SMALL, KERNEL<T, NB>, dim3(n_tokens), dim3(threads), vec ? row_bytes : rot * sizeof(float), stream,    \
-                   qkv, bias, q_w, k_w, eps, inv_freq, inv_freq_lo, rot, v_scale, tok_seq, tok_pos, (T*)q_out, (T*)k_cache,       \
-                   (T*)v_cache, block_table, table_stride, n_pages, page, nh, nkv, hd, vd, write_kv, status)
-#define ESP_WIDENORM_T(T)                                                                      \
-    do {                                                                                       \
-        if (vec && neighbour) ESP_WIDENORM(widenorm_rope_kvwrite_vec_kernel, T, true);         \
-        else if (vec) ESP_WIDENORM(widenorm_rope_kvwrite_vec_kernel, T, false);                \
-        else if (neighbour) ESP_WIDENORM(widenorm_rope_kvwrite_kernel, T, true);               \
-        else ESP_WIDENORM(widenorm_rope_kvwrite_kernel, T, false);                             \
+    const int row_threads = neighbour ? neighbour_row_threads(nh, nkv, hd, vd, ptrs) : 0;
+    const int row_pieces = row_threads ? (((nh + nkv) * hd + nkv * vd) / 4 + row_threads - 1) / row_threads : 0;
+    const bool vec = !neighbour && hd % 4 == 0 && vd % 4 == 0 && rot % 8 == 0 && (ptrs & 15) == 0 && row_bytes <= 40 * 1024;
+#define ESP_WIDENORM(KERNEL, THREADS, SMEM)                                                                                   \
+    esp_launch_pdl(ESP_PDL_SMALL, KERNEL, dim3(n_tokens), dim3(THREADS), SMEM, stream, qkv, bias, q_w, k_w, eps, inv_freq, inv_freq_lo, \
+                   rot, v_scale, tok_seq, tok_pos, (decltype(q_at))q_out, (decltype(q_at))k_cache, (decltype(q_at))v_cache, block_table, \
+                   table_stride, n_pages, page, nh, nkv, hd, vd, write_kv, status)
+#define ESP_WIDENORM_T(T)                                                                                             \
+    do {                                                                                                              \
+        T* q_at = nullptr;                                                                                            \
+        if (row_threads && row_pieces <= 2) ESP_WIDENORM((neighbour_rope_row_kernel<T, 2>), row_threads, rot * sizeof(float));   \
+        else if (row_threads) ESP_WIDENORM((neighbour_rope_row_kernel<T, NEIGHBOUR_PIECES>), row_threads, rot * sizeof(float));  \
+        else if (vec) ESP_WIDENORM(widenorm_rope_kvwrite_vec_kernel<T>, threads, row_bytes);                           \
+        else if (neighbour) ESP_WIDENORM((widenorm_rope_kvwrite_kernel<T, true>), threads, rot * sizeof(float));       \
+        else ESP_WIDENORM((widenorm_rope_kvwrite_kernel<T, false>), threads, rot * sizeof(float));                     \
+        (void)q_at;                                                                                                   \
     } while (0)
     if (is_bf16) ESP_WIDENORM_T(bf16);
     else ESP_WIDENORM_T(float);
@@ -664,6 +770,20 @@ ESP_API int esp_pair_rope_unitnorm_kvwrite(const float* qkv, const float* bias, 
     const size_t smem = (size_t)rot * sizeof(float);
     const size_t ptrs = (size_t)qkv | (size_t)bias | (size_t)v_shared | (size_t)q_out | (size_t)k_cache | (size_t)v_cache;
     const bool pairs = hd % 2 == 0 && vd % 2 == 0 && (ptrs & 7) == 0;
+    const int row_threads = unit_norm || blend_mode ? 0 : neighbour_row_threads(nh, nkv, hd, vd, ptrs);
+    if (row_threads) {
+        const int row_pieces = (((nh + nkv) * hd + nkv * vd) / 4 + row_threads - 1) / row_threads;
+#define ESP_PAIR_ROW(T, NP)                                                                                                  \
+    esp_launch_pdl(ESP_PDL_SMALL, neighbour_rope_row_kernel<T, NP>, dim3(n_tokens), dim3(row_threads), smem, stream, qkv, bias, nullptr,  \
+                   nullptr, eps, inv_freq, inv_freq_lo, rot, 1.0f, tok_seq, tok_pos, (T*)q_out, (T*)k_cache, (T*)v_cache,          \
+                   block_table, table_stride, n_pages, page, nh, nkv, hd, vd, write_kv, status)
+        if (is_bf16 && row_pieces <= 2) ESP_PAIR_ROW(bf16, 2);
+        else if (is_bf16) ESP_PAIR_ROW(bf16, NEIGHBOUR_PIECES);
+        else if (row_pieces <= 2) ESP_PAIR_ROW(float, 2);
+        else ESP_PAIR_ROW(float, NEIGHBOUR_PIECES);
+#undef ESP_PAIR_ROW
+        return esp_launch_status();
+    }
 #define ESP_PAIR_ROPE(T, PAIRS)                                                                                              \
     esp_launch_pdl(ESP_PDL_SMALL, pair_rope_unitnorm_kvwrite_kernel<T, PAIRS>, dim3(n_tokens), dim3(threads), smem, stream, qkv,  \
                    bias, inv_freq, inv_freq_lo, rot, eps, unit_norm, v_shared, blend_mode, lambda, tok_seq, tok_pos, (T*)q_out,    \

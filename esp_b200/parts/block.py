@@ -208,8 +208,16 @@ class OutputNormBlock(Part):
         return pending
 
 
+# Which steps run a mixer on a second stream beside the feed-forward: few rows (decode steps, which are replayed from captured
+# graphs: two chains of short launches side by side) and much work (rows x width), where one's kernels leave room that the
+# other's fill.  In between the host's extra calls cost more than the overlap gains (eight layers, 2,048 tokens: width 1,024
+# 1.71 -> 2.10 ms, width 2,048 2.91 -> 2.63 ms).
+BESIDE_ROWS = 64
+BESIDE_WORK = 3 << 20
+
+
 class ParallelResidualBlock(Part):
-    """x += mixer(h) + ffn(h) with h = norm(x).  Neither sublayer waits for the other: the mixer runs on a second stream
+    """x += mixer(h) + ffn(h) with h = norm(x).  Neither sublayer waits for the other: the mixer may run on a second stream
     beside the feed-forward (in a captured step: a parallel branch of the graph), and the norm that reads x next adds
     both results, in one launch with a sparse feed-forward's ordered sum of its experts."""
 
@@ -234,7 +242,8 @@ class ParallelResidualBlock(Part):
         if self.ffn is None:
             pending = self.mixer.forward(h, ctx, layer)
         else:
-            side = rt.side_stream
+            n = x.shape[0]
+            side = rt.side_stream if n <= BESIDE_ROWS or n * x.shape[1] >= BESIDE_WORK else None
             if side is not None:
                 main = torch.cuda.current_stream()
                 side.wait_stream(main)

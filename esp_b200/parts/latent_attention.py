@@ -132,7 +132,7 @@ class LatentAttention(Part):
     def _unfolded_fits(self) -> bool:
         s = self.spec
         return (self.rt.dtype == torch.bfloat16 and s.own_kv and s.rot_dim == 0 and s.window is None and s.scale > 0
-                and s.nope_dim == s.value_dim and ops.attn_prefill_tc05_fits(s.nope_dim, PAGE) and s.kv_rank % 8 == 0
+                and s.nope_dim == s.value_dim and s.nope_dim in (64, 128) and ops.attn_prefill_tc05_fits(s.nope_dim, PAGE) and s.kv_rank % 8 == 0
                 and self.w_uk is not None and self.w_uk.dtype == torch.bfloat16 and self.w_uv.dtype == torch.bfloat16)
 
     def step_arrays_key(self):

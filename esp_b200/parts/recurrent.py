@@ -362,7 +362,7 @@ class FixedDecayAttention(Part):
     """Linear attention with one fixed decay per head (see ``FixedDecayAttentionSpec``).  One packed product makes q, k, v and
     the output gate; the recurrence takes the SiLUs of the first three as it stages its rows; the heads' output is normed
     as one row and multiplied by the sigmoid gate in one kernel; then W_o.  In bfloat16, steps of many tokens run the
-    recurrence in chunks on the tensor cores; short ones, and all of the 32-bit engine's, token by token.  Per slot the
+    recurrence in chunks on the tensor cores; short ones, and all of the 32-bit engine's, go token by token.  Per slot the
     state holds S as [heads, value channels, key channels] floats."""
 
     graph_safe = True
@@ -435,22 +435,20 @@ class FixedDecayAttention(Part):
         linear(rt, h, self.w_in, proj)
         o = rt.ws.get("rec_out", (n, self.vw), torch.float32)
         chunk_seq = ctx.arrays.get("linear.chunks.seq")
-        if chunk_seq is not None and ops.linear_attn_chunks_fits(s.key_dim, s.value_dim):
+        q, k, v = proj[:, :self.kw], proj[:, self.kw:self.at_v], proj[:, self.at_v:self.at_gate]
+        if rt.dtype != torch.bfloat16 or not ops.linear_attn_chunks_fits(s.key_dim, s.value_dim):
+            ops.gated_scan(ops.SCAN_FIXED_DECAY, q, k, self.decay, v, None, self.decay_rest, None, layer.state, ctx.seq_start,
+                           ctx.seq_slot, o, ctx.n_seqs, s.num_heads, s.key_dim, s.value_dim)
+        elif chunk_seq is None:
+            ops.linear_attn_steps(q, k, v, self.decay, self.decay_rest, layer.state, ctx.seq_start, ctx.seq_slot, o, ctx.n_seqs,
+                                  s.num_heads, s.key_dim, s.value_dim)
+        else:
             per = s.num_heads * s.key_dim * s.value_dim
             at_once = min(chunk_seq.shape[0], max(1, CHUNK_SCRATCH_FLOATS // per))
             scratch = rt.ws.get("linear_chunks", (at_once * per,), torch.float32)
-            ops.linear_attn_chunks(proj[:, :self.kw], proj[:, self.kw:self.at_v], proj[:, self.at_v:self.at_gate], chunk_seq,
-                                   ctx.arrays["linear.chunks.first"], ctx.arrays["linear.chunks.start"], ctx.seq_start, ctx.seq_slot,
-                                   self.powers, scratch, layer.state, o, ctx.n_seqs, s.num_heads, s.key_dim, s.value_dim)
-            return self._finish(proj, o)
-        ops.gated_scan(ops.SCAN_FIXED_DECAY, proj[:, :self.kw], proj[:, self.kw:self.at_v], self.decay,
-                       proj[:, self.at_v:self.at_gate], None, self.decay_rest, None, layer.state, ctx.seq_start, ctx.seq_slot, o,
-                       ctx.n_seqs, s.num_heads, s.key_dim, s.value_dim)
-        return self._finish(proj, o)
-
-    def _finish(self, proj, o):
-        s, rt = self.spec, self.rt
-        n = o.shape[0]
+            ops.linear_attn_chunks(q, k, v, chunk_seq, ctx.arrays["linear.chunks.first"], ctx.arrays["linear.chunks.start"],
+                                   ctx.seq_start, ctx.seq_slot, self.powers, scratch, layer.state, o, ctx.n_seqs, s.num_heads,
+                                   s.key_dim, s.value_dim)
         y = rt.ws.get("rec_normed", (n, self.vw), rt.dtype)
         ops.head_rmsnorm_gate(o, self.norm_w, 0, proj[:, self.at_gate:], y, 1, self.vw, s.eps, gate_sigmoid=True)
         out = rt.ws.get("mixer_out", (n, s.hidden), torch.float32)
