@@ -18,13 +18,13 @@ pytestmark = pytest.mark.gpu
 
 def draw(rng):
     pick = lambda *xs: xs[int(rng.integers(0, len(xs)))]
-    width = pick(64, 72, 100, 128, 160, 320)
+    width = pick(64, 70, 72, 100, 128, 160, 320)
     layers = []
     for i in range(int(rng.integers(2, 6))):
         kind = pick("attention", "attention_2", "attention_2", "lightning")
         if kind == "lightning":
             heads = pick(1, 2, 3, 5)
-            mixer = {"heads": heads, "dim": pick(8, 16, 20, 48, 64, 128), "vdim": pick(8, 16, 24, 40, 64, 96),
+            mixer = {"heads": heads, "dim": pick(8, 16, 18, 20, 48, 64, 128), "vdim": pick(8, 10, 16, 24, 40, 64, 96),
                      "decay": [float(1 - 10 ** -rng.uniform(0.2, 3.5)) for _ in range(heads)]}
         else:
             kv, dim = pick(1, 1, 2, 3), pick(8, 16, 20, 24, 32, 48, 64, 80, 112, 128)
