@@ -612,8 +612,8 @@ class HyperConnectionBlockSpec:
 class NeighbourRopeSpec:
     """Rotary encoding over neighbouring channels: of the first ``rotary_dim`` channels of a head, channel 2i is
     rotated with channel 2i + 1 by the angle position * f_i, f_i = theta^(-2i / rotary_dim).  With ``factor`` slow frequencies
-    are slowed further by their wavelength l = 2 pi / f: f stays where l < original / high, is divided by the factor where
-    l > original / low, and in between is (1 - s) f / factor + s f with s = (original / l - low) / (high - low)."""
+    are slowed: with t = original f / (2 pi) turns within the original length, f stays for t > high, becomes f / factor for
+    t < low, and in between moves linearly in t from the one to the other."""
     rotary_dim: int
     theta: float
     factor: Optional[float] = None

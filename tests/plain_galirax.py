@@ -36,9 +36,9 @@ def layer_norm(x, w, b, eps):
 
 # ---------------------------------------------------------------------------------------------------------
 def frequencies(rot):
-    """float64 [dims / 2]: base^(-2i/dims), slow ones slowed further when the configuration scales them: with the
-    wavelength l = 2 pi / f a frequency is kept below original / high, divided by the factor above original / low, and
-    in between is (1 - s) f / factor + s f with s = (original / l - low) / (high - low)."""
+    """float64 [dims / 2]: base^(-2i/dims).  With scaling, a channel pair whose period (in positions) is shorter than
+    original / high keeps its frequency, one whose period is longer than original / low has it divided by the factor, and
+    between the two the frequency is a blend that is linear in original / period."""
     i = torch.arange(rot["dims"] // 2, dtype=torch.float64)
     f = float(rot["base"]) ** (-2.0 * i / rot["dims"])
     sc = rot.get("scaling")
@@ -46,14 +46,14 @@ def frequencies(rot):
         return f
     out = []
     for v in f.tolist():
-        l = 2 * math.pi / v
-        if l < sc["original"] / sc["high"]:
+        period, slow = 2 * math.pi / v, v / sc["factor"]
+        if period < sc["original"] / sc["high"]:
             out.append(v)
-        elif l > sc["original"] / sc["low"]:
-            out.append(v / sc["factor"])
+        elif period > sc["original"] / sc["low"]:
+            out.append(slow)
         else:
-            s = (sc["original"] / l - sc["low"]) / (sc["high"] - sc["low"])
-            out.append((1 - s) * v / sc["factor"] + s * v)
+            share = (sc["original"] / period - sc["low"]) / (sc["high"] - sc["low"])
+            out.append(slow + share * (v - slow))
     return torch.tensor(out, dtype=torch.float64)
 
 
